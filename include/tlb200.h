@@ -36,7 +36,8 @@ typedef enum { TLB_F32 = 0, TLB_F64 = 1, TLB_F16 = 2, TLB_BF16 = 3, TLB_I32 = 4,
 
 /* GGML type ids as stored in GGUF (crates/tl_runtime/src/quantized.rs:10-22) */
 typedef enum { TLB_GGML_F32 = 0, TLB_GGML_F16 = 1, TLB_GGML_Q4_0 = 2, TLB_GGML_Q4_1 = 3, TLB_GGML_Q5_0 = 6, TLB_GGML_Q5_1 = 7,
-               TLB_GGML_Q8_0 = 8, TLB_GGML_Q8_1 = 9, TLB_GGML_Q4_K = 12, TLB_GGML_Q6_K = 14 } tlb_ggml_type;
+               TLB_GGML_Q8_0 = 8, TLB_GGML_Q8_1 = 9, TLB_GGML_Q4_K = 12, TLB_GGML_Q6_K = 14,
+               TLB_GGML_I32 = 26, TLB_GGML_BF16 = 30 } tlb_ggml_type;
 
 typedef struct tlb_tensor tlb_tensor;     /* CudaTensor handle (crates/tl_cuda/src/tensor.rs:39-99) */
 typedef struct tlb_qtensor tlb_qtensor;   /* QTensor (crates/tl_runtime/src/quantized.rs:29-40) */
@@ -197,6 +198,12 @@ tlb_status tlb_gguf_load_str(tlb_map **out, const tlb_string *path);
  * block layout with a row-major shape (what gguf.rs:129-190 builds per tensor). */
 tlb_status tlb_map_new(tlb_map **out);
 tlb_status tlb_map_add(tlb_map *m, const char *name, tlb_ggml_type type, const int64_t *shape, int rank, const void *bytes, size_t nbytes);
+/* A model folder: config.json (kept in the map, see tlb_map_set_config) and model.safetensors (BF16, F16, F32, I32 tensors).
+ * No counterpart in the reference, which loads GGUF only.  A session on such a map runs the design config.json names. */
+tlb_status tlb_model_load(tlb_map **out, const char *dir);
+/* The description of the model whose tensors the map holds, as the text of a config.json: checked against the registry of
+ * designs (TLB_ERR_TYPE for an unknown one) and from then on the map's model, instead of GGUF metadata. */
+tlb_status tlb_map_set_config(tlb_map *m, const char *config_json);
 tlb_status tlb_map_free(tlb_map *m);                                                      /* tensor_map.rs tl_tensor_map_free */
 int64_t    tlb_map_count(const tlb_map *m);
 const char *tlb_map_name(const tlb_map *m, int64_t i);
@@ -289,6 +296,10 @@ typedef struct {
     /* sequences the session holds (0 or 1: one).  Every sequence has its own cache rows and position; sequence 0 is the
      * one the single-sequence entry points (tlb_decoder_step, _generate, _prefill, _kv_write) work on. */
     int32_t batch;
+    /* models described by a config.json: 1: every product in 32-bit floats and f32 caches and activations; 0: bf16 operands with
+     * 32-bit accumulation, f16 caches.  (kv_f16 is the Llama chain's field and is not looked at for these models; the size
+     * fields above come from the description.) */
+    int32_t f32;
 } tlb_decoder_cfg;
 
 /* Fills the model sizes of *cfg from the GGUF metadata of a loaded file (<arch>.block_count, .embedding_length, ...;
@@ -342,6 +353,12 @@ tlb_status tlb_decoder_generate(tlb_decoder *d, int32_t first_token, int32_t sta
  * tlb_decoder_logits / tlb_decoder_hidden then describe that last token.  Prompts of 16 tokens or fewer, and
  * shapes the GEMM does not take, run token by token through the fused chain. */
 tlb_status tlb_decoder_prefill(tlb_decoder *d, const int32_t *tokens, int32_t n, int32_t pos0, int32_t rope_pos0, int32_t rope_step, int32_t *next);
+/* The same pass over n tokens, with the logits of several of them instead of one greedy token: want[i] is an offset among the n
+ * tokens, logits_out (host) receives [n_want, vocab]; n_want may be 0.  seq: 0, or a sequence of a batch session. */
+tlb_status tlb_decoder_prefill_logits(tlb_decoder *d, int32_t seq, const int32_t *tokens, int32_t n, int32_t pos0, const int32_t *want, int32_t n_want, float *logits_out);
+/* Forgets a sequence: its next token is at position 0.  (A session checks that a recurrent model continues where its state
+ * stands; position 0 always starts afresh, so this call is only bookkeeping.) */
+tlb_status tlb_decoder_reset_seq(tlb_decoder *d, int32_t seq);
 /* ---- a batch of sequences in one session (cfg.batch > 1) ----
  * The reference's matmul entry takes any number of activation rows (crates/tl_runtime/src/system.rs:180-222) and the TL
  * program's layers are batch-agnostic (examples/apps/llama3/chatbot_llama3.tl:220-236).  Here one token per sequence goes

@@ -15,6 +15,7 @@ from ._lib import DecoderCfg, TlbError, check, declared_symbols, lib  # noqa: F4
 
 F32, F16, Q4_0, Q8_0, Q4_K, Q6_K = 0, 1, 2, 8, 12, 14
 Q4_1, Q5_0, Q5_1, Q8_1 = 3, 6, 7, 9
+I32, BF16 = 26, 30
 ROPE_CPU, ROPE_HALF = 0, 1
 TIE_LAST, TIE_FIRST = 0, 1
 _NP_DT = {0: np.float32, 1: np.float64, 2: np.float16, 4: np.int32, 5: np.int64, 6: np.uint8, 7: np.uint32}
@@ -268,6 +269,17 @@ class TensorMap:
         check(lib().tlb_map_new(C.byref(out)))
         return TensorMap(out)
 
+    @staticmethod
+    def load_dir(path):
+        """A model folder: config.json + model.safetensors."""
+        out = C.c_void_p()
+        check(lib().tlb_model_load(C.byref(out), str(path).encode()))
+        return TensorMap(out)
+
+    def set_config(self, text):
+        """Describes the model whose tensors the map holds by the text of a config.json."""
+        check(lib().tlb_map_set_config(self.h, text.encode()))
+
     def meta_number(self, key):
         v = C.c_double()
         check(lib().tlb_map_meta_number(self.h, key.encode(), C.byref(v)))
@@ -436,14 +448,17 @@ class Tokenizer:
 
 
 class Decoder:
-    """Fused decode session over a TensorMap holding a Llama-shaped model."""
+    """Fused decode session over a TensorMap holding a Llama-shaped model, or a model described by a config.json (cfg None or
+    weights.decoder_cfg(); f32: all of its products in 32 bits)."""
 
-    def __init__(self, cfg, weights, kv_f16=True, max_seq=4096, tie_rule=TIE_LAST, tp_size=1, tp_rank=0, batch=1):
+    def __init__(self, cfg, weights, kv_f16=True, max_seq=4096, tie_rule=TIE_LAST, tp_size=1, tp_rank=0, batch=1, f32=False):
+        if cfg is None:
+            cfg = weights.decoder_cfg()
         self.cfg = DecoderCfg(n_layers=cfg["n_layers"], d_model=cfg["d_model"], n_heads=cfg["n_heads"],
                               n_kv_heads=cfg["n_kv_heads"], head_dim=cfg["head_dim"], ffn=cfg["ffn"],
                               vocab=cfg["vocab"], eps=cfg["eps"], rope_base=cfg["rope_base"],
                               attn_scale=cfg["attn_scale"], kv_f16=int(kv_f16), max_seq=max_seq,
-                              tie_rule=tie_rule, tp_size=tp_size, tp_rank=tp_rank, batch=batch)
+                              tie_rule=tie_rule, tp_size=tp_size, tp_rank=tp_rank, batch=batch, f32=int(f32))
         self.batch = max(1, batch)
         self.h = C.c_void_p()
         check(lib().tlb_decoder_create(C.byref(self.h), C.byref(self.cfg), weights.h))
@@ -467,6 +482,18 @@ class Decoder:
         check(lib().tlb_decoder_prefill(self.h, toks, len(tokens), pos0, pos0 if rope_pos0 is None else rope_pos0, rope_step,
                                         C.byref(nxt) if read else None))
         return nxt.value
+
+    def prefill_logits(self, tokens, pos0=0, want=None, seq=0):
+        """The same pass, with the logits of the tokens at the offsets `want` (all of them when None): [len(want), vocab]."""
+        want = list(range(len(tokens))) if want is None else list(want)
+        toks = (C.c_int32 * max(1, len(tokens)))(*[int(t) for t in tokens])
+        w = (C.c_int32 * max(1, len(want)))(*[int(t) for t in want])
+        out = np.empty((len(want), self.cfg.vocab), dtype=np.float32)
+        check(lib().tlb_decoder_prefill_logits(self.h, seq, toks, len(tokens), pos0, w, len(want), out.ctypes.data_as(C.c_void_p)))
+        return out
+
+    def reset_seq(self, seq=0):
+        check(lib().tlb_decoder_reset_seq(self.h, seq))
 
     def sample_top_p(self, temp, top_p, u):
         """Sample from the logits of the last step / prompt on the device; returns the token id."""

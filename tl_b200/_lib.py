@@ -27,7 +27,7 @@ class DecoderCfg(C.Structure):
                 ("n_kv_heads", C.c_int32), ("head_dim", C.c_int32), ("ffn", C.c_int32), ("vocab", C.c_int32),
                 ("eps", C.c_float), ("rope_base", C.c_float), ("attn_scale", C.c_float),
                 ("kv_f16", C.c_int32), ("max_seq", C.c_int32), ("tie_rule", C.c_int32),
-                ("tp_size", C.c_int32), ("tp_rank", C.c_int32), ("batch", C.c_int32)]
+                ("tp_size", C.c_int32), ("tp_rank", C.c_int32), ("batch", C.c_int32), ("f32", C.c_int32)]
 
 
 def declared_symbols():
@@ -120,6 +120,8 @@ def lib():
     d("tlb_decoder_step_batch", S, vp, pi32, pi32, pi32, pi32)
     d("tlb_decoder_generate_batch", S, vp, pi32, pi32, i32, pi32)
     d("tlb_decoder_logits_batch", S, vp, vp)
+    d("tlb_model_load", S, pvp, C.c_char_p); d("tlb_map_set_config", S, vp, C.c_char_p)
+    d("tlb_decoder_prefill_logits", S, vp, i32, pi32, i32, i32, pi32, i32, vp); d("tlb_decoder_reset_seq", S, vp, i32)
     d("tlb_tp_unique_id", S, vp, sz); d("tlb_tp_init", S, vp, sz, C.c_int, C.c_int, C.c_double); d("tlb_tp_poll", S)
     d("tlb_tp_shutdown", S); d("tlb_tp_rank", C.c_int); d("tlb_tp_size", C.c_int); d("tlb_allreduce", S, vp)
     d("tlb_tp_p2p_export", S, vp, sz); d("tlb_tp_p2p_attach", S, vp, C.c_int); d("tlb_tp_p2p_disable", S); d("tlb_tp_p2p_enable", S); d("tlb_tp_exchange_in_launch", S, C.c_int)

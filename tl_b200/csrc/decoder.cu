@@ -15,6 +15,7 @@
 // between two buffers so no kernel updates memory that another CTA of the same launch reads.  All
 // kernels are launched with programmatic dependent launch: what a kernel can fetch without its
 // predecessor's results (weights, norm weights, RoPE tables, older KV rows) is requested before it waits.
+#include "model_desc.h"
 #include "tlb_internal.h"
 
 #include <cstdlib>
@@ -97,6 +98,10 @@ struct tlb_decoder {
     float *part = nullptr;        // tp > 1: this rank's partial o_proj / ffn_down result, summed over the ranks in place
     float *pair = nullptr;        // tp > 1: (best logit, its global index) of this shard, then of every shard [1 + tp][2]
     float *logits_all = nullptr;  // tp > 1: the gathered logits of all shards (tlb_decoder_logits)
+    // A model described by a config.json (model_desc.h): its layers run in layered.cu; the state words, graphs, argmax, sampler,
+    // token rings and entry points are this session's, as for the Llama chain.
+    LayeredModel *lay = nullptr;
+    std::vector<int> seq_len;     // layered: tokens each sequence has behind it (a recurrent state only goes on from there)
 };
 
 namespace {
@@ -257,11 +262,14 @@ void set_w(MatvecJob &j, int i, const tlb_qtensor *q, float *out)
 // the kernel chain of one decode step (launched eagerly or into a capturing stream)
 // output_norm + head + greedy token (with the advance of the decode state) on the residual in xb.
 // ssq_parts: per-tile sums of squares of xb left by the launch that wrote it, or null (the head launch sums itself).
-tlb_status enqueue_head(tlb_decoder *d, const float *ssq_parts, const float *x = nullptr, const float *x2 = nullptr, float *x_out = nullptr)
+// Layered models: the head on xb unless the step left the logits already (head_done).
+tlb_status enqueue_head(tlb_decoder *d, const float *ssq_parts, const float *x = nullptr, const float *x2 = nullptr, float *x_out = nullptr, bool head_done = false)
 {
     const tlb_decoder_cfg &c = d->cfg;
     const int dm = c.d_model;
-    {   // output_norm + head (tp > 1: this rank's rows of the vocabulary)
+    if (d->lay) {
+        if (!head_done) TLB_TRY(layered_head(d->lay, d->xb, 1, d->logits));
+    } else {   // output_norm + head (tp > 1: this rank's rows of the vocabulary)
         MatvecJob j;
         j.n_w = 1;
         set_w(j, 0, d->head, d->logits);
@@ -392,6 +400,10 @@ tlb_status enqueue_step_tp(tlb_decoder *d)
 
 tlb_status enqueue_step(tlb_decoder *d)
 {
+    if (d->lay) {
+        TLB_TRY(layered_step(d->lay, d->state, d->state + 1, d->state + 2, d->xb, d->logits));
+        return enqueue_head(d, nullptr, nullptr, nullptr, nullptr, true);
+    }
     // A tensor-parallel shard with peer memory attached runs the single-GPU chain on its own heads / hidden units: o_proj
     // and ffn_down add their partial sums over the ranks inside the launch, tile by tile (MatvecJob::tp_reduce), so what
     // they leave - the residual and the per-tile sums of its squares - is what the next launch expects anyway.  Without
@@ -596,16 +608,20 @@ tlb_status row_parallel(tlb_decoder *d, const tlb_qtensor *w, const GemmAct &a, 
 }
 
 // output_norm + head + greedy tokens for `rows` residual rows x (sequences row0 ..): logits to blogits[row0 ..]
-tlb_status batch_head(tlb_decoder *d, const float *x, int rows, int row0)
+tlb_status batch_head(tlb_decoder *d, const float *x, int rows, int row0, bool head_done = false)
 {
     const tlb_decoder_cfg &c = d->cfg;
     const int tie_first = c.tie_rule == TLB_TIE_FIRST;
-    GemmAct a;
-    TLB_TRY(qgemm_prepare(&a, x, nullptr, rows, c.d_model, d->out_norm->f32(), c.eps));
     float *lg = d->blogits + (size_t)row0 * d->V;
-    tlb_status st = qgemm_run(d->head, a, lg, nullptr);
-    qgemm_release(&a);
-    TLB_TRY(st);
+    if (d->lay) {
+        if (!head_done) TLB_TRY(layered_head(d->lay, x, rows, lg));
+    } else {
+        GemmAct a;
+        TLB_TRY(qgemm_prepare(&a, x, nullptr, rows, c.d_model, d->out_norm->f32(), c.eps));
+        tlb_status st = qgemm_run(d->head, a, lg, nullptr);
+        qgemm_release(&a);
+        TLB_TRY(st);
+    }
     if (d->tp > 1) {
         argmax_rows_kernel<<<rows, 1024, 0, ctx()->stream>>>(lg, d->V, tie_first, d->tp_r * d->V, d->bpair, nullptr, nullptr, nullptr, nullptr, nullptr, d->B, 0, row0);
         TLB_CUDA(cudaGetLastError());
@@ -628,6 +644,14 @@ tlb_status enqueue_step_batch(tlb_decoder *d)
     const tlb_decoder_cfg &c = d->cfg;
     const int B = d->B, dm = c.d_model, qd = d->H * c.head_dim, kvd = d->KVH * c.head_dim, F = d->F;
     const size_t esz = c.kv_f16 ? 2 : 4;
+    if (d->lay) {
+        TLB_TRY(layered_step_batch(d->lay, d->btok, d->bpos, d->brope, B, d->bx, d->blogits));
+        TLB_TRY(batch_head(d, d->bx, B, 0, true));
+        bump_index_kernel<<<1, 1, 0, ctx()->stream>>>(d->bidx);
+        TLB_CUDA(cudaGetLastError());
+        count_launch();
+        return TLB_OK;
+    }
     TLB_TRY(launch_embed_rows(d->btok, d->emb->f32(), d->bx, B, dm));
     float *x = d->bx, *x2 = d->bx2;
     for (int l = 0; l < c.n_layers; l++) {
@@ -725,6 +749,17 @@ tlb_status ensure_graph(tlb_decoder *d)
     return TLB_OK;
 }
 
+// Layered models: n tokens of sequence `seq` from position `pos` on.  Position 0 starts the sequence afresh; any other position
+// must be where the sequence stands, since a recurrent state holds exactly the tokens behind it.
+tlb_status advance_seq(tlb_decoder *d, int seq, int pos, int n)
+{
+    if (!d->lay) return TLB_OK;
+    if (pos != 0 && pos != d->seq_len[seq])
+        return fail(TLB_ERR_ARG, "sequence %d stands at position %d: it can go on from there or start again at 0, not at %d", seq, d->seq_len[seq], pos);
+    d->seq_len[seq] = pos + n;
+    return TLB_OK;
+}
+
 tlb_status set_state(tlb_decoder *d, int token, int pos, int rope_pos, int out_idx)
 {
     // pageable source: the runtime stages the 16 bytes before returning, so the next call may reuse the stack
@@ -756,10 +791,53 @@ tlb_status tlb_decoder_destroy(tlb_decoder *d)
         tlb_tensor_release(w.attn_norm); tlb_tensor_release(w.ffn_norm);
     }
     tlb_tensor_release(d->emb); tlb_tensor_release(d->out_norm); tlb_qtensor_release(d->head);
+    layered_destroy(d->lay);
     for (void *p : d->allocs) cudaFree(p);
     if (d->h_state) cudaFreeHost(d->h_state);
     if (d->tp > 1) g_tp_sessions--;
     delete d;
+    return TLB_OK;
+}
+
+// A session over a model described by a config.json.
+static tlb_status create_layered(tlb_decoder **out, const tlb_decoder_cfg &cfg, tlb_map *m)
+{
+    if (cfg.max_seq < 1) return fail(TLB_ERR_ARG, "decoder config has a non-positive size");
+    if (cfg.batch < 0 || cfg.batch > 64) return fail(TLB_ERR_ARG, "batch %d: a session holds 1 to 64 sequences", cfg.batch);
+    if (cfg.tp_size > 1) return fail(TLB_ERR_ARG, "models described by a config.json run on one GPU (tp_size 1)");
+    ModelDesc desc;
+    TLB_TRY(model_desc_from_map(m, &desc));
+    tlb_decoder *d = new tlb_decoder();
+    d->cfg = cfg;
+    TLB_TRY(tlb_decoder_cfg_from_map(m, &d->cfg));
+    d->B = cfg.batch > 1 ? cfg.batch : 1;
+    d->V = desc.vocab;
+    d->seq_len.assign(d->B, 0);
+    const size_t dm = desc.width, V = desc.vocab, B = d->B;
+    auto build = [&]() -> tlb_status {
+        LayeredCfg lc;
+        lc.max_seq = cfg.max_seq; lc.batch = d->B; lc.f32 = cfg.f32 != 0;
+        TLB_TRY(layered_create(&d->lay, desc, m, lc));
+        TLB_TRY(dalloc(d, &d->xb, dm));
+        TLB_TRY(dalloc(d, &d->logits, V));
+        TLB_TRY(dalloc(d, &d->counters, 1));            // the argmax counter (no KV heads in front of it)
+        TLB_TRY(dalloc(d, &d->state, 4));
+        d->tokens_cap = cfg.max_seq;
+        TLB_TRY(dalloc(d, &d->tokens_out, d->tokens_cap));
+        TLB_TRY(dalloc(d, &d->amax_v, kArgmaxBlocks));
+        TLB_TRY(dalloc(d, &d->amax_i, kArgmaxBlocks));
+        if (B > 1) {
+            TLB_TRY(dalloc(d, &d->btok, B)); TLB_TRY(dalloc(d, &d->bpos, B)); TLB_TRY(dalloc(d, &d->brope, B)); TLB_TRY(dalloc(d, &d->bidx, 1));
+            TLB_TRY(dalloc(d, &d->bx, B * dm)); TLB_TRY(dalloc(d, &d->bx2, B * dm));
+            TLB_TRY(dalloc(d, &d->blogits, B * V));
+            TLB_TRY(dalloc(d, &d->btokens_out, (size_t)d->tokens_cap * B));
+        }
+        TLB_CUDA(cudaMallocHost((void **)&d->h_state, 4 * sizeof(int)));
+        return tlb_sync();
+    };
+    tlb_status st = build();
+    if (st != TLB_OK) { tlb_decoder_destroy(d); return st; }
+    *out = d;
     return TLB_OK;
 }
 
@@ -769,6 +847,7 @@ tlb_status tlb_decoder_create(tlb_decoder **out, const tlb_decoder_cfg *cfg, tlb
     *out = nullptr;
     if (!cfg || !m) return fail(TLB_ERR_NULL, "null argument");
     if (!ensure_init()) return TLB_ERR_DEVICE;
+    if (map_has_model_config(m)) return create_layered(out, *cfg, m);
     const tlb_decoder_cfg &c = *cfg;
     if (c.n_layers < 1 || c.d_model < 1 || c.n_heads < 1 || c.n_kv_heads < 1 || c.head_dim < 1 || c.ffn < 1 || c.vocab < 1 || c.max_seq < 1)
         return fail(TLB_ERR_ARG, "decoder config has a non-positive size");
@@ -898,6 +977,7 @@ tlb_status tlb_decoder_create(tlb_decoder **out, const tlb_decoder_cfg *cfg, tlb
 tlb_status tlb_decoder_kv_write(tlb_decoder *d, int layer, int pos0, int n, const float *k, const float *v)
 {
     if (!d || !k || !v) return fail(TLB_ERR_NULL, "null argument");
+    if (d->lay) return fail(TLB_ERR_ARG, "kv_write: the layers of this model do not share one cache shape; feed the tokens instead");
     const tlb_decoder_cfg &c = d->cfg;
     if (layer < 0 || layer >= c.n_layers || pos0 < 0 || n < 0 || pos0 + n > c.max_seq)
         return fail(TLB_ERR_INDEX, "kv_write: layer %d rows [%d, %d) out of range", layer, pos0, pos0 + n);
@@ -932,6 +1012,7 @@ tlb_status tlb_decoder_step(tlb_decoder *d, int32_t token, int32_t pos, int32_t 
     if (pos < 0 || pos >= d->cfg.max_seq || rope_pos < 0 || rope_pos >= d->cfg.max_seq)
         return fail(TLB_ERR_INDEX, "position %d / %d outside the cache of %d rows", pos, rope_pos, d->cfg.max_seq);
     TLB_TRY(ensure_graph(d));
+    TLB_TRY(advance_seq(d, 0, pos, 1));
     TLB_TRY(set_state(d, token, pos, rope_pos, 0));
     TLB_CUDA(cudaGraphLaunch(d->graph, ctx()->stream));
     ctx()->launches += d->graph_kernels;
@@ -949,6 +1030,7 @@ tlb_status tlb_decoder_generate(tlb_decoder *d, int32_t first_token, int32_t sta
     if (first_token < 0 || first_token >= d->cfg.vocab) return fail(TLB_ERR_INDEX, "Embedding index %d out of range", first_token);
     if (n < 0 || start_pos < 0 || start_pos + n > d->cfg.max_seq) return fail(TLB_ERR_INDEX, "positions [%d, %d) outside the cache of %d rows", start_pos, start_pos + n, d->cfg.max_seq);
     TLB_TRY(ensure_graph(d));
+    TLB_TRY(advance_seq(d, 0, start_pos, n));
     TLB_TRY(set_state(d, first_token, start_pos, start_pos, 0));
     for (int i = 0; i < n; i++) TLB_CUDA(cudaGraphLaunch(d->graph, ctx()->stream));
     ctx()->launches += d->graph_kernels * (uint64_t)n;
@@ -981,6 +1063,12 @@ tlb_status tlb_decoder_hidden(tlb_decoder *d, float *hidden_out)
 tlb_status tlb_decoder_stats(const tlb_decoder *d, int32_t ctx_len, uint64_t *weight_bytes, uint64_t *kv_bytes, int32_t *kernels_per_step)
 {
     if (!d) return fail(TLB_ERR_NULL, "null decoder");
+    if (d->lay) {
+        if (weight_bytes) *weight_bytes = layered_weight_bytes(d->lay);
+        if (kv_bytes) *kv_bytes = layered_state_bytes(d->lay, ctx_len);
+        if (kernels_per_step) *kernels_per_step = layered_kernels_per_step(d->lay) + 1;
+        return TLB_OK;
+    }
     uint64_t wb = d->head->nbytes() + (uint64_t)d->cfg.d_model * 4 * (2 * d->cfg.n_layers + 2);
     for (const LayerW &w : d->layers)
         wb += w.q->nbytes() + w.k->nbytes() + w.v->nbytes() + w.o->nbytes() + w.gate->nbytes() + w.up->nbytes() + w.down->nbytes();
@@ -997,6 +1085,7 @@ tlb_status tlb_decoder_stats(const tlb_decoder *d, int32_t ctx_len, uint64_t *we
 tlb_status tlb_decoder_time_kernel(tlb_decoder *d, const char *which, int copies, int iters, float *us_per_launch, uint64_t *bytes_per_launch)
 {
     if (!d || !which || !us_per_launch) return fail(TLB_ERR_NULL, "null argument");
+    if (d->lay) return fail(TLB_ERR_ARG, "time_kernel times the launches of the Llama chain");
     const tlb_decoder_cfg &c = d->cfg;
     const int dm = c.d_model, qd = d->H * c.head_dim, kvd = d->KVH * c.head_dim, F = d->F;
     if (copies < 1) copies = 1;
@@ -1077,6 +1166,7 @@ constexpr int kPrefillChunk = 2048;
 
 bool prefill_batched_ok(const tlb_decoder *d)
 {
+    if (d->lay) return true;
     const tlb_decoder_cfg &c = d->cfg;
     const int qd = d->H * c.head_dim, kvd = d->KVH * c.head_dim;
     for (const LayerW &w : d->layers)
@@ -1099,10 +1189,11 @@ struct Scratch {
     ~Scratch() { for (Storage *s : all) storage_release(s); }
 };
 
-// T prompt tokens of sequence `seq` (0 for a single-sequence session) into cache rows pos0 ..; the residual of the last
-// token is copied to last_row_out when given.  With tensor parallelism every rank runs this on its shard.
-tlb_status prefill_chunk(tlb_decoder *d, int seq, const int32_t *tokens, int T, int pos0, int rope0, int rope_step, float *last_row_out)
+// T prompt tokens of sequence `seq` (0 for a single-sequence session) into cache rows pos0 ..; the residuals of the tokens
+// want[i] (offsets among the T) are copied to rows_out [n_want, d_model].  With tensor parallelism every rank runs this on its shard.
+tlb_status prefill_chunk(tlb_decoder *d, int seq, const int32_t *tokens, int T, int pos0, int rope0, int rope_step, const int32_t *want, int n_want, float *rows_out)
 {
+    if (d->lay) return layered_prefill(d->lay, seq, tokens, T, pos0, rope0, rope_step, want, n_want, rows_out);
     const tlb_decoder_cfg &c = d->cfg;
     const int dm = c.d_model, qd = d->H * c.head_dim, kvd = d->KVH * c.head_dim, F = d->F;
     const size_t esz = c.kv_f16 ? 2 : 4;
@@ -1163,7 +1254,20 @@ tlb_status prefill_chunk(tlb_decoder *d, int seq, const int32_t *tokens, int T, 
         qgemm_release(&a);
         TLB_TRY(st);
     }
-    if (last_row_out) TLB_CUDA(cudaMemcpyAsync(last_row_out, x + (size_t)(T - 1) * dm, (size_t)dm * sizeof(float), cudaMemcpyDeviceToDevice, ctx()->stream));
+    for (int i = 0; i < n_want; i++)
+        TLB_CUDA(cudaMemcpyAsync(rows_out + (size_t)i * dm, x + (size_t)want[i] * dm, (size_t)dm * sizeof(float), cudaMemcpyDeviceToDevice, ctx()->stream));
+    return TLB_OK;
+}
+
+// A whole prompt, chunk by chunk; the residual of its last token goes to last_row.
+tlb_status prefill_all(tlb_decoder *d, int seq, const int32_t *tokens, int n, int pos0, int rope_pos0, int rope_step, float *last_row)
+{
+    TLB_TRY(advance_seq(d, seq, pos0, n));
+    for (int off = 0; off < n; off += kPrefillChunk) {
+        const int T = std::min(kPrefillChunk, n - off);
+        const int32_t last = T - 1;
+        TLB_TRY(prefill_chunk(d, seq, tokens + off, T, pos0 + off, rope_pos0 + off * rope_step, rope_step, &last, off + T == n ? 1 : 0, last_row));
+    }
     return TLB_OK;
 }
 }  // namespace
@@ -1178,17 +1282,14 @@ extern "C" tlb_status tlb_decoder_prefill(tlb_decoder *d, const int32_t *tokens,
     const int64_t last_rope = (int64_t)rope_pos0 + (int64_t)(n - 1) * rope_step;
     if (pos0 < 0 || (int64_t)pos0 + n > c.max_seq || rope_pos0 < 0 || rope_step < 0 || last_rope >= c.max_seq)
         return fail(TLB_ERR_INDEX, "positions [%d, %d) / rotation rows up to %lld outside the cache of %d rows", pos0, pos0 + n, (long long)last_rope, c.max_seq);
-    if (n <= 4 || !prefill_batched_ok(d)) {
+    if (n <= (d->lay ? 1 : 4) || !prefill_batched_ok(d)) {
         // few tokens, or a shape the GEMM path does not take: the fused single-token chain, token by token
         int32_t tok = 0;
         for (int i = 0; i < n; i++) TLB_TRY(tlb_decoder_step(d, tokens[i], pos0 + i, rope_pos0 + i * rope_step, i == n - 1 ? &tok : nullptr));
         if (next) *next = tok;
         return TLB_OK;
     }
-    for (int off = 0; off < n; off += kPrefillChunk) {
-        const int T = std::min(kPrefillChunk, n - off);
-        TLB_TRY(prefill_chunk(d, 0, tokens + off, T, pos0 + off, rope_pos0 + off * rope_step, rope_step, off + T == n ? d->xb : nullptr));
-    }
+    TLB_TRY(prefill_all(d, 0, tokens, n, pos0, rope_pos0, rope_step, d->xb));
     // head on the last token; the state then names the next token and the row it will occupy
     TLB_TRY(set_state(d, tokens[n - 1], pos0 + n - 1, (int)last_rope, 0));
     TLB_TRY(enqueue_head(d, nullptr));
@@ -1242,6 +1343,7 @@ extern "C" tlb_status tlb_decoder_generate_sampled(tlb_decoder *d, int32_t first
     }
     const unsigned long long zero = 0;
     TLB_CUDA(cudaMemcpyAsync(d->samp_counter, &zero, sizeof zero, cudaMemcpyHostToDevice, ctx()->stream));
+    TLB_TRY(advance_seq(d, 0, start_pos, n));
     TLB_TRY(set_state(d, first_token, start_pos, start_pos, 0));
     for (int i = 0; i < n; i++) TLB_CUDA(cudaGraphLaunch(d->sgraph, ctx()->stream));
     ctx()->launches += d->sgraph_kernels * (uint64_t)n;
@@ -1293,10 +1395,7 @@ extern "C" tlb_status tlb_decoder_prefill_seq(tlb_decoder *d, int32_t seq, const
     if (pos0 < 0 || (int64_t)pos0 + n > c.max_seq || rope_pos0 < 0 || rope_step < 0 || last_rope >= c.max_seq)
         return fail(TLB_ERR_INDEX, "positions [%d, %d) / rotation rows up to %lld outside the cache of %d rows", pos0, pos0 + n, (long long)last_rope, c.max_seq);
     float *row = d->bx2 + (size_t)seq * c.d_model;     // free between steps
-    for (int off = 0; off < n; off += kPrefillChunk) {
-        const int T = std::min(kPrefillChunk, n - off);
-        TLB_TRY(prefill_chunk(d, seq, tokens + off, T, pos0 + off, rope_pos0 + off * rope_step, rope_step, off + T == n ? row : nullptr));
-    }
+    TLB_TRY(prefill_all(d, seq, tokens, n, pos0, rope_pos0, rope_step, row));
     // the sequence's state: the last prompt token at its row; the head then names the next token and advances both
     const int32_t st3[3] = {tokens[n - 1], pos0 + n - 1, (int32_t)last_rope};
     TLB_TRY(put_ints(d->btok + seq, st3, 1)); TLB_TRY(put_ints(d->bpos + seq, st3 + 1, 1)); TLB_TRY(put_ints(d->brope + seq, st3 + 2, 1));
@@ -1326,6 +1425,7 @@ extern "C" tlb_status tlb_decoder_step_batch(tlb_decoder *d, const int32_t *toke
         if (pos[b] < 0 || pos[b] >= c.max_seq || rp < 0 || rp >= c.max_seq) return fail(TLB_ERR_INDEX, "sequence %d: position %d / %d outside the cache of %d rows", b, pos[b], rp, c.max_seq);
     }
     TLB_TRY(ensure_batch_graph(d));
+    for (int b = 0; b < d->B; b++) TLB_TRY(advance_seq(d, b, pos[b], 1));
     const int32_t zero = 0;
     TLB_TRY(put_ints(d->btok, tokens, d->B)); TLB_TRY(put_ints(d->bpos, pos, d->B)); TLB_TRY(put_ints(d->brope, rope_pos ? rope_pos : pos, d->B));
     TLB_TRY(put_ints(d->bidx, &zero, 1));
@@ -1350,6 +1450,7 @@ extern "C" tlb_status tlb_decoder_generate_batch(tlb_decoder *d, const int32_t *
         if (start_pos[b] < 0 || (int64_t)start_pos[b] + n > c.max_seq) return fail(TLB_ERR_INDEX, "sequence %d: rows [%d, %d) outside the cache of %d rows", b, start_pos[b], start_pos[b] + n, c.max_seq);
     }
     TLB_TRY(ensure_batch_graph(d));
+    for (int b = 0; b < d->B; b++) TLB_TRY(advance_seq(d, b, start_pos[b], n));
     const int32_t zero = 0;
     TLB_TRY(put_ints(d->btok, first_tokens, d->B)); TLB_TRY(put_ints(d->bpos, start_pos, d->B)); TLB_TRY(put_ints(d->brope, start_pos, d->B));
     TLB_TRY(put_ints(d->bidx, &zero, 1));
@@ -1398,5 +1499,69 @@ extern "C" tlb_status tlb_decoder_sample_top_p(tlb_decoder *d, float temp, float
     TLB_CUDA(cudaMemcpyAsync(&h, d->amax_v, sizeof(float), cudaMemcpyDeviceToHost, ctx()->stream));
     TLB_TRY(tlb_sync());
     *token = (int32_t)h;
+    return TLB_OK;
+}
+
+// n tokens of one sequence and the logits of the wanted ones.
+extern "C" tlb_status tlb_decoder_prefill_logits(tlb_decoder *d, int32_t seq, const int32_t *tokens, int32_t n, int32_t pos0, const int32_t *want, int32_t n_want, float *logits_out)
+{
+    if (!d || !tokens || (n_want > 0 && (!want || !logits_out))) return fail(TLB_ERR_NULL, "null argument");
+    const tlb_decoder_cfg &c = d->cfg;
+    if (seq < 0 || seq >= d->B) return fail(TLB_ERR_INDEX, "sequence %d outside the batch of %d", seq, d->B);
+    if (d->tp > 1) return fail(TLB_ERR_ARG, "logits of several tokens need the whole vocabulary on one GPU (tp_size 1)");
+    if (n < 1 || n_want < 0) return fail(TLB_ERR_ARG, "prefill needs at least one token");
+    if (pos0 < 0 || (int64_t)pos0 + n > c.max_seq) return fail(TLB_ERR_INDEX, "positions [%d, %d) outside the cache of %d rows", pos0, pos0 + n, c.max_seq);
+    for (int i = 0; i < n; i++)
+        if (tokens[i] < 0 || tokens[i] >= c.vocab) return fail(TLB_ERR_INDEX, "Embedding index %d out of range for vocab size %d", tokens[i], c.vocab);
+    for (int i = 0; i < n_want; i++)
+        if (want[i] < 0 || want[i] >= n) return fail(TLB_ERR_INDEX, "wanted token %d outside the %d given", want[i], n);
+    if (d->B == 1 && (n == 1 || !prefill_batched_ok(d))) {
+        // one token, or a shape the row kernels do not take: the decode chain, token by token
+        for (int i = 0; i < n; i++) {
+            TLB_TRY(tlb_decoder_step(d, tokens[i], pos0 + i, pos0 + i, nullptr));
+            for (int k = 0; k < n_want; k++)
+                if (want[k] == i) TLB_TRY(tlb_decoder_logits(d, logits_out + (size_t)k * c.vocab));
+        }
+        return tlb_sync();
+    }
+    TLB_TRY(advance_seq(d, seq, pos0, n));
+    Scratch ws;
+    float *rows = nullptr, *lg = nullptr;
+    const int kRows = 512;                                  // wanted rows the head takes at a time
+    if (n_want) {
+        TLB_TRY(ws.get(&rows, (size_t)n_want * c.d_model));
+        TLB_TRY(ws.get(&lg, (size_t)std::min(n_want, kRows) * c.vocab));
+    }
+    std::vector<int32_t> local, place;
+    for (int off = 0, done = 0; off < n; off += kPrefillChunk) {
+        const int T = std::min(kPrefillChunk, n - off);
+        local.clear();
+        for (int i = 0; i < n_want; i++)
+            if (want[i] >= off && want[i] < off + T) { local.push_back(want[i] - off); place.push_back(i); }
+        TLB_TRY(prefill_chunk(d, seq, tokens + off, T, pos0 + off, pos0 + off, 1, local.data(), (int)local.size(), rows + (size_t)done * c.d_model));
+        done += (int)local.size();
+    }
+    for (int r0 = 0; r0 < n_want; r0 += kRows) {
+        const int m = std::min(kRows, n_want - r0);
+        const float *x = rows + (size_t)r0 * c.d_model;
+        if (d->lay) TLB_TRY(layered_head(d->lay, x, m, lg));
+        else {
+            GemmAct a;
+            TLB_TRY(qgemm_prepare(&a, x, nullptr, m, c.d_model, d->out_norm->f32(), c.eps));
+            tlb_status st = qgemm_run(d->head, a, lg, nullptr);
+            qgemm_release(&a);
+            TLB_TRY(st);
+        }
+        for (int i = 0; i < m; i++)
+            TLB_CUDA(cudaMemcpyAsync(logits_out + (size_t)place[r0 + i] * c.vocab, lg + (size_t)i * c.vocab, (size_t)c.vocab * sizeof(float), cudaMemcpyDeviceToHost, ctx()->stream));
+    }
+    return tlb_sync();
+}
+
+extern "C" tlb_status tlb_decoder_reset_seq(tlb_decoder *d, int32_t seq)
+{
+    if (!d) return fail(TLB_ERR_NULL, "null decoder");
+    if (seq < 0 || seq >= d->B) return fail(TLB_ERR_INDEX, "sequence %d outside the batch of %d", seq, d->B);
+    if (d->lay) d->seq_len[seq] = 0;
     return TLB_OK;
 }

@@ -1,0 +1,519 @@
+// Linear layers on bf16 weights, and the row kernels around them (embedding, RMS norm, PolyNorm).
+//
+//   dense_matvec_kernel   one activation row (decode): streams the weight once, f32 activation and accumulation.  The prologue
+//                         makes the activation in shared memory - RMS norm, PolyNorm (its three root mean squares), an embedding
+//                         row - and the finish adds the scaled result to the residual, so a layer is five launches.
+//   dense_gemm_tc_kernel  many rows, bf16 operands: tcgen05.mma, both tiles by TMA, f32 accumulator in tensor memory.
+//   dense_gemm_f32_kernel many rows, f32 activations: plain f32 multiply-adds (no tensor core rounds the operands).
+#include <algorithm>
+
+#include "layered_kernels.h"
+#include "tc05.cuh"
+
+namespace tlb {
+
+namespace {
+
+__device__ __forceinline__ float bf_lo(uint32_t w) { return __uint_as_float(w << 16); }
+__device__ __forceinline__ float bf_hi(uint32_t w) { return __uint_as_float(w & 0xFFFF0000u); }
+__device__ __forceinline__ float warp_sum(float v)
+{
+#pragma unroll
+    for (int o = 16; o; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+}
+
+// ================================================================ one row
+constexpr int kMvThreads = 256, kMvWarps = kMvThreads / 32, kMvRows = 4, kMvChunk = 256;
+
+struct DenseMvParams {
+    const __nv_bfloat16 *w;
+    int n, k, ld, nch;                 // nch: chunks of 256 columns
+    const float *bias;
+    const float *x;
+    const __nv_bfloat16 *emb;
+    int emb_ld;
+    const int *token;
+    float *x_out;
+    const float *norm_w;
+    float norm_offset, eps;
+    const float *poly;
+    float *out;
+    const float *resid_scale;
+    int tiles;
+};
+
+// Shared position of activation element e: inside a chunk of 256 the first four of every eight come first, so that a lane's
+// eight (two 16-byte reads) are read without bank conflicts.
+__device__ __forceinline__ int xs_at(int e) { return (e & ~255) + ((e & 4) << 5) + ((e & 255) >> 3) * 4 + (e & 3); }
+
+template <int NV>
+__device__ __forceinline__ void block_sums(float (&v)[NV], float *red)
+{
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+        v[i] = warp_sum(v[i]);
+        if (lane == 0) red[warp * NV + i] = v[i];
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+        float s = 0.f;
+        for (int w = 0; w < (int)(blockDim.x >> 5); w++) s += red[w * NV + i];
+        v[i] = s;
+    }
+}
+
+// WK warps share a row group's columns (chunk c belongs to warp c % WK); 8 / WK row groups of four rows per tile.
+template <int PRO, int WK>
+__global__ void __launch_bounds__(kMvThreads, 4) dense_matvec_kernel(const DenseMvParams p)
+{
+    constexpr int GROUPS = kMvWarps / WK, TILE = GROUPS * kMvRows;
+    extern __shared__ __align__(16) float xs[];
+    __shared__ float red[kMvWarps * 3];
+    __shared__ float fold[2][GROUPS][WK][kMvRows];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, wk = warp % WK, wg = warp / WK;
+
+    // what the first tile reads does not depend on the launch before: ask L2 for it before waiting
+    {
+        const int r0 = blockIdx.x * TILE + wg * kMvRows;
+        for (int r = 0; r < kMvRows; r++) {
+            const int row = min(r0 + r, p.n - 1);
+            const __nv_bfloat16 *src = p.w + (size_t)row * p.ld;
+            for (int c = wk + (lane >> 2) * WK; c < p.nch; c += 8 * WK) {
+                const int e = c * kMvChunk + (lane & 3) * 64;
+                if (e < p.ld) asm volatile("prefetch.global.L2 [%0];" ::"l"(src + e));
+            }
+        }
+    }
+    pdl_wait();
+    pdl_launch_dependents();
+
+    const int kp = p.nch * kMvChunk;
+    if (PRO == DPRO_PLAIN) {
+        for (int e = tid; e < kp; e += kMvThreads) xs[xs_at(e)] = e < p.k ? __ldcg(p.x + e) : 0.f;
+    } else if (PRO == DPRO_NORM) {
+        const __nv_bfloat16 *er = p.emb ? p.emb + (size_t)*p.token * p.emb_ld : nullptr;
+        float ss[1] = {0.f};
+        for (int e = tid; e < p.k; e += kMvThreads) {
+            const float v = er ? __bfloat162float(er[e]) : __ldcg(p.x + e);
+            xs[xs_at(e)] = v;
+            ss[0] += v * v;
+            if (er && blockIdx.x == 0) p.x_out[e] = v;
+        }
+        block_sums(ss, red);
+        const float inv = 1.f / sqrtf(ss[0] / (float)p.k + p.eps);
+        for (int e = tid; e < kp; e += kMvThreads) {
+            float *s = xs + xs_at(e);
+            *s = e < p.k ? *s * inv * (p.norm_w[e] + p.norm_offset) : 0.f;
+        }
+    } else {
+        float ss[3] = {0.f, 0.f, 0.f};
+        for (int e = tid; e < p.k; e += kMvThreads) {
+            const float v = __ldcg(p.x + e), v2 = v * v;
+            xs[xs_at(e)] = v;
+            ss[0] += v2; ss[1] += v2 * v2; ss[2] += v2 * v2 * v2;
+        }
+        block_sums(ss, red);
+        const float inv_n = 1.f / (float)p.k;
+        const float a = p.poly[0] / sqrtf(ss[0] * inv_n + p.eps), b = p.poly[1] / sqrtf(ss[1] * inv_n + p.eps),
+                    c = p.poly[2] / sqrtf(ss[2] * inv_n + p.eps), d = p.poly[3];
+        for (int e = tid; e < kp; e += kMvThreads) {
+            float *s = xs + xs_at(e);
+            const float z = *s;
+            *s = e < p.k ? z * (a + z * (b + z * c)) + d : 0.f;
+        }
+    }
+    __syncthreads();
+
+    int flip = 0;
+    for (int tile = blockIdx.x; tile < p.tiles; tile += gridDim.x, flip ^= 1) {
+        const int r0 = tile * TILE + wg * kMvRows;
+        const uint4 *rows[kMvRows];
+#pragma unroll
+        for (int r = 0; r < kMvRows; r++) rows[r] = reinterpret_cast<const uint4 *>(p.w + (size_t)min(r0 + r, p.n - 1) * p.ld) + lane;
+        float acc[kMvRows] = {0.f, 0.f, 0.f, 0.f};
+        auto load = [&](int c, uint4 (&v)[kMvRows]) {
+            const bool in = c < p.nch && c * kMvChunk + lane * 8 < p.ld;
+#pragma unroll
+            for (int r = 0; r < kMvRows; r++) v[r] = in ? __ldcs(rows[r] + c * (kMvChunk / 8)) : make_uint4(0u, 0u, 0u, 0u);
+        };
+        auto mul = [&](int c, const uint4 (&v)[kMvRows]) {
+            if (c >= p.nch) return;
+            const float4 xa = *reinterpret_cast<const float4 *>(xs + c * kMvChunk + lane * 4);
+            const float4 xb = *reinterpret_cast<const float4 *>(xs + c * kMvChunk + 128 + lane * 4);
+#pragma unroll
+            for (int r = 0; r < kMvRows; r++) {
+                float s = acc[r];
+                s = fmaf(bf_lo(v[r].x), xa.x, s); s = fmaf(bf_hi(v[r].x), xa.y, s);
+                s = fmaf(bf_lo(v[r].y), xa.z, s); s = fmaf(bf_hi(v[r].y), xa.w, s);
+                s = fmaf(bf_lo(v[r].z), xb.x, s); s = fmaf(bf_hi(v[r].z), xb.y, s);
+                s = fmaf(bf_lo(v[r].w), xb.z, s); s = fmaf(bf_hi(v[r].w), xb.w, s);
+                acc[r] = s;
+            }
+        };
+        for (int c = wk; c < p.nch; c += 2 * WK) {
+            uint4 va[kMvRows], vb[kMvRows];
+            load(c, va);
+            load(c + WK, vb);
+            mul(c, va);
+            mul(c + WK, vb);
+        }
+#pragma unroll
+        for (int r = 0; r < kMvRows; r++) acc[r] = warp_sum(acc[r]);
+        float y = lane == 0 ? acc[0] : (lane == 1 ? acc[1] : (lane == 2 ? acc[2] : acc[3]));
+        if (WK > 1) {
+            if (lane < kMvRows) fold[flip][wg][wk][lane] = y;
+            __syncthreads();
+            if (wk == 0 && lane < kMvRows) {
+                y = 0.f;
+#pragma unroll
+                for (int i = 0; i < WK; i++) y += fold[flip][wg][i][lane];
+            }
+        }
+        const int row = r0 + lane;
+        if (wk == 0 && lane < kMvRows && row < p.n) {
+            if (p.bias) y += p.bias[row];
+            if (p.resid_scale) p.out[row] = __ldcg(p.out + row) + p.resid_scale[row] * y;
+            else p.out[row] = y;
+        }
+    }
+}
+
+// ================================================================ many rows, tensor cores
+constexpr int kTcRows = 128, kTcK = 64, kTcThreads = 192;
+constexpr uint32_t kTcWBytes = kTcRows * kTcK * 2;
+
+struct DenseTcParams {
+    float *out;
+    const float *bias, *resid_scale;
+    int n, T, ldo, nt, kt, stages;
+    uint32_t tmem_cols;
+    int *err;
+};
+
+// One CTA: 128 weight rows (lanes of the accumulator) x nt tokens (its columns).  Warps 0-3 write out (a warp's 32 lanes are 32
+// consecutive output features of one token: coalesced), warp 4 lane 0 issues TMA, warp 5 lane 0 the MMAs.  Every wait is bounded.
+__global__ void __launch_bounds__(kTcThreads, 1)
+dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ CUtensorMap xmap, const DenseTcParams p)
+{
+    extern __shared__ uint8_t tc_smem[];
+    __shared__ int abort_word;
+    __shared__ uint32_t tmem_slot;
+    volatile int *abort_flag = &abort_word;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const uint32_t base = (smem_u32(tc_smem) + 1023u) & ~1023u;
+    const uint32_t xbytes = (uint32_t)p.nt * (kTcK * 2), stage = kTcWBytes + xbytes;
+    const uint32_t bars = base + (uint32_t)p.stages * stage;
+    const uint32_t full = bars, empty = bars + 8u * p.stages, done = bars + 16u * p.stages;
+    const int t0 = blockIdx.x * p.nt, n0 = blockIdx.y * kTcRows;
+
+    if (tid == 0) {
+        abort_word = 0;
+        for (int i = 0; i < p.stages; i++) { mbar_init(full + 8 * i, 1); mbar_init(empty + 8 * i, 1); }
+        mbar_init(done, 1);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+    }
+    if (warp == 5) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_slot)), "r"(p.tmem_cols) : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = tmem_slot;
+
+    if (warp < 4) {
+        if (mbar_wait(done, 0, abort_flag, p.err, 61)) {
+            tc_fence_after();
+            const int row = n0 + warp * 32 + lane;
+            const bool in = row < p.n;
+            const float bias = in && p.bias ? p.bias[row] : 0.f, rs = in && p.resid_scale ? p.resid_scale[row] : 0.f;
+            for (int c0 = 0; c0 < p.nt && t0 + c0 < p.T; c0 += 32) {
+                uint32_t v[32];
+                tmem_ld32(tmem + ((uint32_t)(warp * 32) << 16) + (uint32_t)c0, v);
+                tmem_wait_ld();
+                if (!in) continue;
+                float *dst = p.out + (size_t)(t0 + c0) * p.ldo + row;
+                const int m = min(32, p.T - t0 - c0);
+                if (p.resid_scale) {
+                    float r[32];
+#pragma unroll
+                    for (int i = 0; i < 32; i++) r[i] = i < m ? dst[(size_t)i * p.ldo] : 0.f;
+#pragma unroll
+                    for (int i = 0; i < 32; i++)
+                        if (i < m) dst[(size_t)i * p.ldo] = fmaf(rs, __uint_as_float(v[i]), r[i]);
+                } else {
+#pragma unroll
+                    for (int i = 0; i < 32; i++)
+                        if (i < m) dst[(size_t)i * p.ldo] = __uint_as_float(v[i]) + bias;
+                }
+            }
+        }
+    } else if (warp == 4) {
+        if (lane == 0) {
+            int issued = 0;
+            for (int k = 0; k < p.kt; k++) {
+                const int s = k % p.stages;
+                if (k >= p.stages && !mbar_wait(empty + 8 * s, (uint32_t)(k / p.stages - 1) & 1u, abort_flag, p.err, 62)) break;
+                mbar_expect_tx(full + 8 * s, stage);
+                tma_load_2d(base + (uint32_t)s * stage, &wmap, k * kTcK, n0, full + 8 * s);
+                tma_load_2d(base + (uint32_t)s * stage + kTcWBytes, &xmap, k * kTcK, t0, full + 8 * s);
+                issued = k + 1;
+            }
+            if (*abort_flag)
+                for (int k = max(0, issued - p.stages); k < issued; k++) mbar_wait_drain(full + 8 * (k % p.stages), (uint32_t)(k / p.stages) & 1u);
+        }
+    } else if (lane == 0) {
+        // f32 accumulator, bf16 operands, both K-major, M 128, N nt
+        const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(p.nt >> 3) << 17) | ((uint32_t)(kTcRows >> 4) << 24);
+        for (int k = 0; k < p.kt; k++) {
+            const int s = k % p.stages;
+            if (!mbar_wait(full + 8 * s, (uint32_t)(k / p.stages) & 1u, abort_flag, p.err, 63)) break;
+            tc_fence_after();
+            const uint64_t wd = smem_desc_sw128(base + (uint32_t)s * stage), xd = smem_desc_sw128(base + (uint32_t)s * stage + kTcWBytes);
+#pragma unroll
+            for (int j = 0; j < 4; j++) umma_f16_ss(tmem, wd + 2u * j, xd + 2u * j, idesc, (k | j) != 0);
+            umma_commit(empty + 8 * s);
+        }
+        umma_commit(done);                       // also after an abort: MMAs in flight end before the tensor memory is freed
+        if (*abort_flag) mbar_wait_drain(done, 0);
+    }
+    tc_fence_before();
+    __syncthreads();
+    if (warp == 5) {
+        __syncwarp();
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(p.tmem_cols) : "memory");
+    }
+}
+
+// ================================================================ many rows, f32 operands
+struct DenseF32Params {
+    const __nv_bfloat16 *w;
+    int n, k, ld;
+    const float *bias, *x, *resid_scale;
+    int ldx, T, ldo;
+    float *out;
+};
+constexpr int kSgT = 64, kSgN = 64, kSgK = 16;
+
+__global__ void __launch_bounds__(256) dense_gemm_f32_kernel(const DenseF32Params p)
+{
+    __shared__ float sx[kSgK][kSgT + 4], sw[kSgK][kSgN + 4];
+    const int tid = threadIdx.x, n0 = blockIdx.y * kSgN, t0 = blockIdx.x * kSgT;
+    const int tn = tid & 15, tt = tid >> 4;
+    float acc[4][4] = {};
+    for (int k0 = 0; k0 < p.k; k0 += kSgK) {
+        for (int i = tid; i < kSgT * kSgK; i += 256) {
+            const int r = i / kSgK, c = i % kSgK;
+            sx[c][r] = t0 + r < p.T && k0 + c < p.k ? p.x[(size_t)(t0 + r) * p.ldx + k0 + c] : 0.f;
+            sw[c][r] = n0 + r < p.n && k0 + c < p.k ? __bfloat162float(p.w[(size_t)(n0 + r) * p.ld + k0 + c]) : 0.f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int c = 0; c < kSgK; c++) {
+            const float4 a = *reinterpret_cast<const float4 *>(&sx[c][tt * 4]), b = *reinterpret_cast<const float4 *>(&sw[c][tn * 4]);
+            const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+            for (int i = 0; i < 4; i++)
+#pragma unroll
+                for (int j = 0; j < 4; j++) acc[i][j] = fmaf(av[i], bv[j], acc[i][j]);
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < 4; i++)
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+            const int t = t0 + tt * 4 + i, n = n0 + tn * 4 + j;
+            if (t >= p.T || n >= p.n) continue;
+            float *o = p.out + (size_t)t * p.ldo + n;
+            if (p.resid_scale) *o = fmaf(p.resid_scale[n], acc[i][j], *o);
+            else *o = acc[i][j] + (p.bias ? p.bias[n] : 0.f);
+        }
+}
+
+// ================================================================ rows
+__device__ __forceinline__ void store_act(float *p, float v) { *p = v; }
+__device__ __forceinline__ void store_act(__nv_bfloat16 *p, float v) { *p = __float2bfloat16_rn(v); }
+
+template <typename TA>
+__global__ void __launch_bounds__(256) norm_rows_kernel(const float *__restrict__ x, int width, const float *__restrict__ w, float offset, float eps,
+                                                        TA *__restrict__ out, int ld)
+{
+    __shared__ float red[8];
+    const float *row = x + (size_t)blockIdx.x * width;
+    float ss[1] = {0.f};
+    for (int i = threadIdx.x; i < width; i += 256) ss[0] += row[i] * row[i];
+    block_sums(ss, red);
+    const float inv = 1.f / sqrtf(ss[0] / (float)width + eps);
+    TA *o = out + (size_t)blockIdx.x * ld;
+    for (int i = threadIdx.x; i < ld; i += 256) store_act(o + i, i < width ? row[i] * inv * (w[i] + offset) : 0.f);
+}
+
+template <typename TA>
+__global__ void __launch_bounds__(512) poly_rows_kernel(const float *__restrict__ z, int ff, int ldz, const float *__restrict__ coef, float eps,
+                                                        TA *__restrict__ out, int ld)
+{
+    __shared__ float red[16 * 3];
+    const float *row = z + (size_t)blockIdx.x * ldz;
+    float ss[3] = {0.f, 0.f, 0.f};
+    for (int i = threadIdx.x; i < ff; i += 512) {
+        const float v2 = row[i] * row[i];
+        ss[0] += v2; ss[1] += v2 * v2; ss[2] += v2 * v2 * v2;
+    }
+    block_sums(ss, red);
+    const float inv_n = 1.f / (float)ff;
+    const float a = coef[0] / sqrtf(ss[0] * inv_n + eps), b = coef[1] / sqrtf(ss[1] * inv_n + eps), c = coef[2] / sqrtf(ss[2] * inv_n + eps), d = coef[3];
+    TA *o = out + (size_t)blockIdx.x * ld;
+    for (int i = threadIdx.x; i < ld; i += 512) {
+        const float v = i < ff ? row[i] : 0.f;
+        store_act(o + i, i < ff ? v * (a + v * (b + v * c)) + d : 0.f);
+    }
+}
+
+__global__ void embed_bf16_kernel(const int *__restrict__ tokens, const __nv_bfloat16 *__restrict__ table, int width, int ld, float *__restrict__ x)
+{
+    const __nv_bfloat16 *src = table + (size_t)tokens[blockIdx.x] * ld;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) x[(size_t)blockIdx.x * width + i] = __bfloat162float(src[i]);
+}
+
+__global__ void gather_rows_kernel(const float *__restrict__ x, int width, const int *__restrict__ idx, float *__restrict__ out)
+{
+    const float *src = x + (size_t)idx[blockIdx.x] * width;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) out[(size_t)blockIdx.x * width + i] = src[i];
+}
+
+__global__ void pack_rows_kernel(const __nv_bfloat16 *__restrict__ src, int k, __nv_bfloat16 *__restrict__ dst, int ld)
+{
+    for (int i = threadIdx.x; i < k; i += blockDim.x) dst[(size_t)blockIdx.x * ld + i] = src[(size_t)blockIdx.x * k + i];
+}
+
+tlb_status launched(const char *what)
+{
+    cudaError_t e = cudaGetLastError();
+    if (e != cudaSuccess) return cuda_fail(e, what);
+    count_launch();
+    return TLB_OK;
+}
+
+template <int PRO, int WK>
+tlb_status run_matvec(const DenseMvParams &p, bool pdl)
+{
+    Context *c = ctx();
+    const size_t smem = (size_t)p.nch * kMvChunk * sizeof(float);
+    static size_t allowed = 48 << 10;
+    if (smem > allowed) {
+        TLB_CUDA(cudaFuncSetAttribute(dense_matvec_kernel<PRO, WK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        allowed = smem;
+    }
+    const int per_sm = std::max(1, std::min(4, (int)(((size_t)220 << 10) / (smem + 2048))));
+    const int grid = std::min(p.tiles, c->sm_count * per_sm);
+    TLB_CUDA(launch_chained(dense_matvec_kernel<PRO, WK>, dim3(grid), dim3(kMvThreads), smem, pdl, p));
+    count_launch();
+    return TLB_OK;
+}
+
+template <int PRO>
+tlb_status pick_matvec(DenseMvParams p, bool pdl)
+{
+    // the fewest warps per row group that still give every SM two tiles
+    int wk = 1;
+    auto tiles = [&](int w) { return (p.n + kMvWarps / w * kMvRows - 1) / (kMvWarps / w * kMvRows); };
+    while (wk < 8 && tiles(wk) < 2 * ctx()->sm_count && wk * 2 <= p.nch) wk *= 2;
+    p.tiles = tiles(wk);
+    switch (wk) {
+    case 1: return run_matvec<PRO, 1>(p, pdl);
+    case 2: return run_matvec<PRO, 2>(p, pdl);
+    case 4: return run_matvec<PRO, 4>(p, pdl);
+    default: return run_matvec<PRO, 8>(p, pdl);
+    }
+}
+
+}  // namespace
+
+bool dense_matvec_supported(int k) { return k >= 1 && k <= 48 * 1024; }
+
+tlb_status launch_dense_matvec(const DenseMatvecJob &j)
+{
+    if (!ctx()) return TLB_ERR_DEVICE;
+    if (!dense_matvec_supported(j.w.k)) return fail(TLB_ERR_SHAPE, "a linear layer over %d inputs does not fit the matvec's shared memory", j.w.k);
+    DenseMvParams p = {};
+    p.w = j.w.w; p.n = j.w.n; p.k = j.w.k; p.ld = j.w.ld; p.nch = (j.w.ld + kMvChunk - 1) / kMvChunk;
+    p.bias = j.w.bias; p.x = j.x; p.emb = j.emb; p.emb_ld = act_ld(j.w.k); p.token = j.token; p.x_out = j.x_out;
+    p.norm_w = j.norm_w; p.norm_offset = j.norm_offset; p.eps = j.eps; p.poly = j.poly; p.out = j.out; p.resid_scale = j.resid_scale;
+    if (j.pro == DPRO_NORM) return pick_matvec<DPRO_NORM>(p, j.pdl);
+    if (j.pro == DPRO_POLY) return pick_matvec<DPRO_POLY>(p, j.pdl);
+    return pick_matvec<DPRO_PLAIN>(p, j.pdl);
+}
+
+tlb_status launch_dense_gemm(const DenseGemmJob &j, bool f32)
+{
+    Context *c = ctx();
+    if (!c) return TLB_ERR_DEVICE;
+    if (j.T < 1) return TLB_OK;
+    if (f32) {
+        DenseF32Params p;
+        p.w = j.w.w; p.n = j.w.n; p.k = j.w.k; p.ld = j.w.ld; p.bias = j.w.bias; p.x = (const float *)j.x; p.resid_scale = j.resid_scale;
+        p.ldx = j.ldx; p.T = j.T; p.ldo = j.ldo; p.out = j.out;
+        dense_gemm_f32_kernel<<<dim3((j.T + kSgT - 1) / kSgT, (j.w.n + kSgN - 1) / kSgN), 256, 0, c->stream>>>(p);
+        return launched("f32 GEMM launch");
+    }
+    DenseTcParams p;
+    p.out = j.out; p.bias = j.w.bias; p.resid_scale = j.resid_scale; p.n = j.w.n; p.T = j.T; p.ldo = j.ldo;
+    p.nt = std::min(256, (j.T + 31) / 32 * 32);
+    p.tmem_cols = 32;
+    while (p.tmem_cols < (uint32_t)p.nt) p.tmem_cols *= 2;
+    p.kt = (j.w.k + kTcK - 1) / kTcK;
+    const size_t stage = kTcWBytes + (size_t)p.nt * kTcK * 2;
+    p.stages = (int)std::min<size_t>(8, ((size_t)216 << 10) / stage);
+    p.err = c->err_flag;
+    CUtensorMap wmap, xmap;
+    if (!encode_f16_map(&wmap, j.w.w, (uint64_t)j.w.k, (uint64_t)j.w.n, (uint64_t)j.w.ld * 2, kTcK, kTcRows, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16) ||
+        !encode_f16_map(&xmap, j.x, (uint64_t)j.w.k, (uint64_t)j.T, (uint64_t)j.ldx * 2, kTcK, (uint32_t)p.nt, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16))
+        return fail(TLB_ERR_DEVICE, "GEMM: cuTensorMapEncodeTiled failed or is not available");
+    const size_t smem = (size_t)p.stages * stage + 16 * p.stages + 8 + 1024;
+    static size_t allowed = 0;
+    if (smem > allowed) {
+        TLB_CUDA(cudaFuncSetAttribute(dense_gemm_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        allowed = smem;
+    }
+    dense_gemm_tc_kernel<<<dim3((j.T + p.nt - 1) / p.nt, (j.w.n + kTcRows - 1) / kTcRows), kTcThreads, smem, c->stream>>>(wmap, xmap, p);
+    return launched("GEMM launch");
+}
+
+tlb_status launch_norm_rows(const float *x, int T, int width, const float *w, float offset, float eps, void *out, int ld, bool f32)
+{
+    if (f32) norm_rows_kernel<<<T, 256, 0, ctx()->stream>>>(x, width, w, offset, eps, (float *)out, ld);
+    else norm_rows_kernel<<<T, 256, 0, ctx()->stream>>>(x, width, w, offset, eps, (__nv_bfloat16 *)out, ld);
+    return launched("norm launch");
+}
+
+tlb_status launch_poly_rows(const float *z, int T, int ff, int ldz, const float *coef, float eps, void *out, int ld, bool f32)
+{
+    if (f32) poly_rows_kernel<<<T, 512, 0, ctx()->stream>>>(z, ff, ldz, coef, eps, (float *)out, ld);
+    else poly_rows_kernel<<<T, 512, 0, ctx()->stream>>>(z, ff, ldz, coef, eps, (__nv_bfloat16 *)out, ld);
+    return launched("PolyNorm launch");
+}
+
+tlb_status launch_embed_bf16(const int *tokens, const __nv_bfloat16 *table, int width, int ld, float *x, int T)
+{
+    embed_bf16_kernel<<<T, 256, 0, ctx()->stream>>>(tokens, table, width, ld, x);
+    return launched("embedding launch");
+}
+
+tlb_status launch_gather_rows(const float *x, int width, const int *idx, int n, float *out)
+{
+    gather_rows_kernel<<<n, 256, 0, ctx()->stream>>>(x, width, idx, out);
+    return launched("gather launch");
+}
+
+tlb_status launch_pack_rows(const __nv_bfloat16 *src, int n, int k, __nv_bfloat16 *dst, int ld, int col0)
+{
+    pack_rows_kernel<<<n, 256, 0, ctx()->stream>>>(src, k, dst + col0, ld);
+    return launched("weight packing launch");
+}
+
+}  // namespace tlb

@@ -5,6 +5,10 @@
 // Differences from the reference by design: quantized tensors are repacked once into the tiled
 // device layout while loading (the reference copies the raw bytes into a Vec<u8> and uploads them
 // on first use), and host bytes are not kept afterwards.
+#include <cuda_bf16.h>
+
+#include "json.h"
+#include "model_desc.h"
 #include "tlb_internal.h"
 
 #include <fcntl.h>
@@ -13,7 +17,9 @@
 #include <unistd.h>
 
 #include <algorithm>
+#include <fstream>
 #include <map>
+#include <sstream>
 
 using namespace tlb;
 
@@ -21,7 +27,8 @@ struct MapEntry {
     int type = 0;
     std::vector<int64_t> shape;   // row-major
     tlb_qtensor *q = nullptr;     // quantized types
-    tlb_tensor *f32 = nullptr;    // F32 / F16 data, or the cached dequantisation of q
+    tlb_tensor *f32 = nullptr;    // F32 / F16 data, or the cached dequantisation of q / widening of raw
+    tlb_tensor *raw = nullptr;    // BF16 and I32 data as stored
 };
 
 struct tlb_map {
@@ -43,9 +50,15 @@ __global__ void f16_to_f32_kernel2(const __half *a, float *out, int64_t n)
         out[i] = __half2float(a[i]);
 }
 
+__global__ void bf16_to_f32_kernel(const __nv_bfloat16 *a, float *out, int64_t n)
+{
+    for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x)
+        out[i] = __bfloat162float(a[i]);
+}
+
 static bool ggml_known(int type)
 {
-    return type == TLB_GGML_F32 || type == TLB_GGML_F16 || type == TLB_GGML_Q4_0 || type == TLB_GGML_Q4_1 || type == TLB_GGML_Q5_0 ||
+    return type == TLB_GGML_BF16 || type == TLB_GGML_I32 || type == TLB_GGML_F32 || type == TLB_GGML_F16 || type == TLB_GGML_Q4_0 || type == TLB_GGML_Q4_1 || type == TLB_GGML_Q5_0 ||
            type == TLB_GGML_Q5_1 || type == TLB_GGML_Q8_0 || type == TLB_GGML_Q8_1 || type == TLB_GGML_Q4_K || type == TLB_GGML_Q6_K;
 }
 
@@ -75,6 +88,8 @@ static tlb_status map_add(tlb_map *m, const std::string &name, int type, const i
     e.shape.assign(shape, shape + rank);
     if (type == TLB_GGML_F32) {
         TLB_TRY(tlb_tensor_from_host(&e.f32, bytes, TLB_F32, shape, rank));
+    } else if (type == TLB_GGML_BF16 || type == TLB_GGML_I32) {
+        TLB_TRY(tlb_tensor_from_host(&e.raw, bytes, type == TLB_GGML_BF16 ? TLB_BF16 : TLB_I32, shape, rank));
     } else if (type == TLB_GGML_F16) {  // F16 -> f32, exact widening (quantized.rs:167-180)
         tlb_tensor *h = nullptr;
         TLB_TRY(tlb_tensor_from_host(&h, bytes, TLB_F16, shape, rank));
@@ -184,9 +199,111 @@ static bool gguf_skip_value(Reader &r, uint32_t t, uint64_t *uint_val, double *n
     return r.ok;
 }
 
+// f32 form of a BF16 tensor, kept beside the stored one
+static tlb_status widen_raw(MapEntry &e, const char *name)
+{
+    if (!e.raw || e.raw->dt != TLB_BF16) return fail(TLB_ERR_TYPE, "Tensor '%s' holds integers", name);
+    TLB_TRY(new_tensor(&e.f32, TLB_F32, e.shape.data(), (int)e.shape.size()));
+    const int64_t n = e.f32->numel();
+    if (n) {
+        bf16_to_f32_kernel<<<(int)std::min<int64_t>((n + 255) / 256, 148 * 16), 256, 0, ctx()->stream>>>((const __nv_bfloat16 *)e.raw->data(), e.f32->f32(), n);
+        TLB_CUDA(cudaGetLastError());
+        count_launch();
+    }
+    return TLB_OK;
+}
+
+bool map_has(const tlb_map *m, const std::string &name) { return m->entries.count(name) != 0; }
+
+const tlb_tensor *map_raw_bf16(const tlb_map *m, const std::string &name)
+{
+    auto it = m->entries.find(name);
+    return it == m->entries.end() || !it->second.raw || it->second.raw->dt != TLB_BF16 ? nullptr : it->second.raw;
+}
+
+// A safetensors file: 8-byte little-endian length, that many bytes of JSON (name -> dtype, shape, data_offsets), the data.
+static tlb_status safetensors_into(tlb_map *m, const std::string &path)
+{
+    int fd = open(path.c_str(), O_RDONLY);
+    if (fd < 0) return fail(TLB_ERR_ARG, "Failed to open %s", path.c_str());
+    struct stat sb;
+    if (fstat(fd, &sb) != 0) { close(fd); return fail(TLB_ERR_ARG, "cannot stat %s", path.c_str()); }
+    const size_t fsize = (size_t)sb.st_size;
+    if (fsize < 8) { close(fd); return fail(TLB_ERR_ARG, "%s is too small", path.c_str()); }
+    void *mm = mmap(nullptr, fsize, PROT_READ, MAP_PRIVATE, fd, 0);
+    close(fd);
+    if (mm == MAP_FAILED) return fail(TLB_ERR_ARG, "Failed to mmap %s", path.c_str());
+    tlb_status st = TLB_OK;
+    const uint8_t *p = (const uint8_t *)mm;
+    uint64_t hlen;
+    memcpy(&hlen, p, 8);
+    do {
+        if (hlen > fsize - 8) { st = fail(TLB_ERR_ARG, "%s: the header is longer than the file", path.c_str()); break; }
+        const std::string text((const char *)p + 8, (size_t)hlen);
+        JReader r{text.c_str(), text.c_str() + text.size()};
+        JVal root;
+        if (!r.value(root) || !root.is(JVal::OBJ)) { st = fail(TLB_ERR_ARG, "%s: the header is not a JSON object", path.c_str()); break; }
+        const uint8_t *data = p + 8 + hlen;
+        const uint64_t dsize = fsize - 8 - hlen;
+        for (auto &kv : root.obj) {
+            if (kv.first == "__metadata__") continue;
+            const JVal *dt = kv.second.get("dtype"), *sh = kv.second.get("shape"), *off = kv.second.get("data_offsets");
+            if (!dt || !dt->is(JVal::STR) || !sh || !sh->is(JVal::ARR) || !off || !off->is(JVal::ARR) || off->arr.size() != 2 || sh->arr.size() > (size_t)kMaxRank) {
+                st = fail(TLB_ERR_ARG, "%s: malformed entry '%s'", path.c_str(), kv.first.c_str());
+                break;
+            }
+            int type = -1;
+            if (dt->str == "BF16") type = TLB_GGML_BF16;
+            else if (dt->str == "F32") type = TLB_GGML_F32;
+            else if (dt->str == "F16") type = TLB_GGML_F16;
+            else if (dt->str == "I32") type = TLB_GGML_I32;
+            if (type < 0) { st = fail(TLB_ERR_TYPE, "%s: '%s' has dtype %s (BF16, F16, F32, I32 are read)", path.c_str(), kv.first.c_str(), dt->str.c_str()); break; }
+            std::vector<int64_t> shape;
+            bool ok = true;
+            auto whole = [&](const JVal &v, double max) { const bool g = v.is(JVal::NUM) && v.num >= 0 && v.num <= max && v.num == (double)(int64_t)v.num; ok &= g; return g ? (int64_t)v.num : 0; };
+            for (const JVal &v : sh->arr) shape.push_back(whole(v, 1e15));
+            const uint64_t b = (uint64_t)whole(off->arr[0], 1e15), e = (uint64_t)whole(off->arr[1], 1e15);
+            if (!ok || b > e || e > dsize) { st = fail(TLB_ERR_ARG, "%s: '%s' lies outside the file", path.c_str(), kv.first.c_str()); break; }
+            st = map_add(m, kv.first, type, shape.data(), (int)shape.size(), data + b, (size_t)(e - b));
+            if (st != TLB_OK) break;
+        }
+    } while (0);
+    munmap(mm, fsize);
+    return st;
+}
+
 }  // namespace tlb
 
 extern "C" {
+
+tlb_status tlb_model_load(tlb_map **out, const char *dir)
+{
+    if (!out) return fail(TLB_ERR_NULL, "null out");
+    *out = nullptr;
+    if (!dir) return fail(TLB_ERR_NULL, "null path");
+    const std::string base = std::string(dir) + "/";
+    std::ifstream f(base + "config.json", std::ios::binary);
+    if (!f) return fail(TLB_ERR_ARG, "Failed to open %sconfig.json", base.c_str());
+    std::stringstream ss;
+    ss << f.rdbuf();
+    tlb_map *m = new tlb_map();
+    tlb_status st = tlb_map_set_config(m, ss.str().c_str());
+    if (st == TLB_OK) st = safetensors_into(m, base + "model.safetensors");
+    if (st != TLB_OK) { tlb_map_free(m); return st; }
+    *out = m;
+    return TLB_OK;
+}
+
+tlb_status tlb_map_set_config(tlb_map *m, const char *config_json)
+{
+    if (!m || !config_json) return fail(TLB_ERR_NULL, "null argument");
+    m->meta_str["config.json"] = config_json;
+    ModelDesc d;
+    tlb_status st = model_desc_from_map(m, &d);
+    if (st != TLB_OK) { m->meta_str.erase("config.json"); return st; }
+    m->meta_str["general.architecture"] = d.arch;
+    return TLB_OK;
+}
 
 tlb_status tlb_map_new(tlb_map **out)
 {
@@ -220,6 +337,15 @@ const char *tlb_map_meta_string(const tlb_map *m, const char *key)
 tlb_status tlb_decoder_cfg_from_map(const tlb_map *m, tlb_decoder_cfg *cfg)
 {
     if (!m || !cfg) return fail(TLB_ERR_NULL, "null argument");
+    if (map_has_model_config(m)) {
+        // layers may differ from one another: heads and feed-forward sizes stay with the description, the rest is filled
+        ModelDesc d;
+        TLB_TRY(model_desc_from_map(m, &d));
+        cfg->n_layers = (int32_t)d.layers.size(); cfg->d_model = d.width; cfg->vocab = d.vocab; cfg->eps = d.eps;
+        cfg->n_heads = cfg->n_kv_heads = cfg->head_dim = cfg->ffn = 0;
+        cfg->rope_base = cfg->attn_scale = 0.f;
+        return TLB_OK;
+    }
     const char *a = tlb_map_meta_string(m, "general.architecture");
     const std::string arch = a ? a : "llama";
     auto num = [&](const std::string &key, double *v) {
@@ -334,7 +460,8 @@ static tlb_status gguf_load_impl(tlb_map **out, const char *path, int tp_rank, i
             if (nelem && !nb) continue;                // not a whole number of blocks
             // "data out of bounds": skipped (gguf.rs:183-186); subtraction form, so that a huge offset cannot wrap
             if (data_off > fsize || inf.offset > fsize - data_off || nb > fsize - data_off - inf.offset) continue;
-            if ((int)inf.type != TLB_GGML_F32 && (int)inf.type != TLB_GGML_F16 && !inf.shape.empty()) {
+            const bool scalar_type = (int)inf.type == TLB_GGML_F32 || (int)inf.type == TLB_GGML_F16 || (int)inf.type == TLB_GGML_BF16 || (int)inf.type == TLB_GGML_I32;
+            if (!scalar_type && !inf.shape.empty()) {
                 // rows must hold whole blocks: K-quants need K % 256 == 0, the 32-blocks K % 32 == 0
                 const int64_t kk = inf.shape.back();
                 const bool k_quant = (int)inf.type == TLB_GGML_Q4_K || (int)inf.type == TLB_GGML_Q6_K;
@@ -424,6 +551,7 @@ tlb_status tlb_map_free(tlb_map *m)
     for (auto &kv : m->entries) {
         tlb_qtensor_release(kv.second.q);
         tlb_tensor_release(kv.second.f32);
+        tlb_tensor_release(kv.second.raw);
     }
     delete m;
     return TLB_OK;
@@ -448,6 +576,7 @@ tlb_status tlb_map_get_quantized(tlb_qtensor **out, tlb_map *m, const char *name
         // F32 / F16 tensor: the reference wraps any type in a QTensor (tensor_map.rs:279) and multiplies it through the
         // dequantise + matmul route (system.rs:236-264).  The dense QTensor shares the f32 data the map already holds.
         if (e.shape.empty()) return fail(TLB_ERR_SHAPE, "Tensor '%s' is a scalar", name);
+        if (!e.f32) TLB_TRY(widen_raw(e, name));
         tlb_qtensor *q = new tlb_qtensor();
         q->type = e.type;
         q->k = e.shape.back();
@@ -470,6 +599,7 @@ tlb_status tlb_map_get(tlb_tensor **out, tlb_map *m, const char *name)
     auto it = m->entries.find(name);
     if (it == m->entries.end()) return fail(TLB_ERR_ARG, "Tensor '%s' not found in map", name);
     MapEntry &e = it->second;
+    if (!e.f32 && e.raw) TLB_TRY(widen_raw(e, name));
     if (!e.f32) {   // cached, as QTensor::cache does
         tlb_tensor *d = nullptr;
         TLB_TRY(tlb_qtensor_dequantize(&d, e.q));

@@ -199,7 +199,8 @@ size_t ggml_raw_nbytes(int type, int64_t nelem)
     auto blocks = [&](int per, int bytes) -> size_t { return nelem % per ? 0 : (size_t)(nelem / per) * bytes; };
     switch (type) {
     case TLB_GGML_F32: return (size_t)nelem * 4;
-    case TLB_GGML_F16: return (size_t)nelem * 2;
+    case TLB_GGML_F16: case TLB_GGML_BF16: return (size_t)nelem * 2;
+    case TLB_GGML_I32: return (size_t)nelem * 4;
     case TLB_GGML_Q4_0: return blocks(32, 18);
     case TLB_GGML_Q4_1: return blocks(32, 20);
     case TLB_GGML_Q5_0: return blocks(32, 22);

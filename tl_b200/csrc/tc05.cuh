@@ -87,9 +87,10 @@ inline PFN_cuTensorMapEncodeTiled_v12000 tensor_map_encoder()
     return fn;
 }
 
-// f16 row-major [rows][cols] (row pitch in bytes) as a 2-D tiled map with 128-byte swizzle; box = box_cols (64: one
+// 16-bit row-major [rows][cols] (row pitch in bytes) as a 2-D tiled map with 128-byte swizzle; box = box_cols (64: one
 // swizzle row of f16) x box_rows.  Rows and columns past the extent read as zero.
-inline bool encode_f16_map(CUtensorMap *map, const void *base, uint64_t cols, uint64_t rows, uint64_t pitch_bytes, uint32_t box_cols, uint32_t box_rows)
+inline bool encode_f16_map(CUtensorMap *map, const void *base, uint64_t cols, uint64_t rows, uint64_t pitch_bytes, uint32_t box_cols, uint32_t box_rows,
+                           CUtensorMapDataType type = CU_TENSOR_MAP_DATA_TYPE_FLOAT16)
 {
     auto encode = tensor_map_encoder();
     if (!encode) return false;
@@ -97,7 +98,7 @@ inline bool encode_f16_map(CUtensorMap *map, const void *base, uint64_t cols, ui
     const cuuint64_t strides[1] = {pitch_bytes};
     const cuuint32_t box[2] = {box_cols, box_rows};
     const cuuint32_t estr[2] = {1, 1};
-    return encode(map, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void *>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+    return encode(map, type, 2, const_cast<void *>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
                   CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
