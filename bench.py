@@ -674,8 +674,84 @@ PARTS = {
     "qrows": "one Q4_K 57344 x 8192 weight (gate | up of the 70B shapes, 264 MB) with 16 activation rows, four calls (small case for a profiler capture)",
     "c4-4layer": "Llama-3-70B-shaped decode on one GPU, 4 layers + head, 4096-row f16 context: batch 1 (fused matvec chain) and batch 16 (few-rows streaming kernel)",
     "per-op-4layer": "the TL chatbot's op sequence through the per-op entry points (native driver), Llama-3-8B shapes cut to 4 layers, 2048 cached rows, 3 steps",
+    "mukutar": "Mukutar models (bf16 weights): decode and prompt throughput at two sizes, beside a Llama model (Q4_K) of the same sizes",
+    "mukutar-3layer": "one layer of each mixer at width 4096 + head: a 2048-token prompt and 8 decode steps (small case for a launch list)",
     "prefill-2layer": "one 2048-token prompt through two Llama-3-8B-shaped layers + head, three times (small case for a profiler capture)",
 }
+
+
+def mukutar_cfg(width, heads, kv_heads, ff, n_layers, vocab, window, dim=128):
+    """Retention, general delta and attention in turn, every head of size `dim`."""
+    mix = {"retention": dict(heads=heads, dim=dim, vdim=dim, rot=dict(base=10000.0, dims=dim), decay=[1.0 - 2.0 ** (-5 - 6 * i / heads) for i in range(heads)]),
+           "general_delta": dict(heads=heads, dim=dim),
+           "attention": dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=dim ** -0.5, mask=dict(size=window))}
+    order = ["retention", "general_delta", "attention"]
+    return {"architecture": "Mukutar", "vocab": vocab, "width": width, "norm": {"eps": 1e-5},
+            "layers": [{"type": order[i % 3], "mixer": mix[order[i % 3]], "mlp": {"kind": "dense", "ff": ff}} for i in range(n_layers)]}
+
+
+def build_mukutar_map(tl, cfg, seed=77):
+    """Seeded random weights; large matrices repeat a block of random values, generated once (the arithmetic does not depend on them)."""
+    from tl_b200 import synth
+    block = synth.to_bf16(np.random.default_rng(seed).standard_normal(1 << 22, dtype=np.float32))
+    m = tl.TensorMap.new()
+    for name, shape in synth.mukutar_specs(cfg, rank=128).items():
+        n = int(np.prod(shape))
+        if n < block.size:
+            bits = synth.to_bf16(synth.mukutar_tensor(name, shape, seed))
+        else:
+            scale = np.float32(1.0 if name == "embed" else shape[1] ** -0.5)
+            bits = np.resize(synth.to_bf16(synth.from_bf16(block) * scale), n)
+        m.add(name, synth.BF16, shape, bits)
+    m.set_config(json.dumps(cfg))
+    return m
+
+
+def time_events(tl, ev, fn, n):
+    L = tl.lib()
+    tl.sync()
+    tl.check(L.tlb_event_record(ev[0]))
+    for _ in range(n):
+        fn()
+    tl.check(L.tlb_event_record(ev[1]))
+    tl.sync()
+    return _elapsed_ms(tl, ev[0], ev[1]) / n
+
+
+def measure_mukutar(tl, ev, peaks, width, heads, kv_heads, ff, n_layers=6, vocab=32768, window=4096, prompt=2048, steps=32):
+    """Decode (batch 1, behind a prompt of `prompt` tokens) and prompt throughput of a Mukutar model, and of a Llama model of the same
+    width, heads, feed-forward size, layers and vocabulary (Q4_K, three feed-forward matrices against two).  Weights exceed L2."""
+    from tl_b200 import synth
+    toks = [int(t) for t in np.random.default_rng(6).integers(0, vocab, prompt)]
+    out = {"width": width, "heads": heads, "kv_heads": kv_heads, "ff": ff, "layers": n_layers, "vocab": vocab, "window": window, "prompt": prompt}
+    cfg = mukutar_cfg(width, heads, kv_heads, ff, n_layers, vocab, window)
+    lcfg = dict(n_layers=n_layers, d_model=width, n_heads=heads, n_kv_heads=kv_heads, head_dim=128, ffn=ff, vocab=vocab, eps=1e-5, rope_base=10000.0, attn_scale=0.08839)
+    for name in ("mukutar", "llama_q4k"):
+        if name == "mukutar":
+            wmap = build_mukutar_map(tl, cfg)
+            dec = tl.Decoder(None, wmap, max_seq=prompt + 256)
+            per_kind = {"retention": 4, "general_delta": 5, "attention": 2}      # input matrices of heads * 128 rows (attention: q, and k | v)
+            lin = sum(2.0 * width * heads * 128 * (per_kind[l["type"]] + 1) + (4.0 * width * kv_heads * 128 - 2.0 * width * heads * 128 if l["type"] == "attention" else 0.0) + 4.0 * width * ff
+                      for l in cfg["layers"])
+        else:
+            wmap = tl.map_from_tensors(synth.llama_tensors(lcfg, 1, 12, 12))
+            dec = tl.Decoder(lcfg, wmap, kv_f16=True, max_seq=prompt + 256)
+            lin = n_layers * (2.0 * width * (2 * heads + 2 * kv_heads) * 128 + 6.0 * width * ff)
+        for _ in range(2):
+            dec.prefill(toks, 0, read=False)
+        ms = time_events(tl, ev, lambda: dec.prefill(toks, 0, read=False), 3)
+        tf = lin * prompt / ms / 1e9
+        r = {"prefill_ms": round(ms, 3), "prefill_tokens_per_s": round(prompt / ms * 1e3), "prefill_linear_tflops": round(tf, 1), "prefill_frac_bf16": round(tf / peaks.get("bf16_tflops", 1590.0), 4)}
+        dec.generate(1, prompt, 8, read=False)
+        ms = time_events(tl, ev, lambda: dec.generate(1, prompt + 8, steps, read=False), 1) / steps
+        st = dec.stats(prompt + 8)
+        gbs = (st["weight_bytes"] + st["kv_bytes"]) / ms / 1e6
+        r.update({"decode_ms": round(ms, 4), "decode_tokens_per_s": round(1e3 / ms, 1), "decode_GBs": round(gbs, 1), "decode_frac_hbm": round(gbs / peaks["hbm_gbs"], 4),
+                  "weight_MB": round(st["weight_bytes"] / 1e6, 1), "kernels_per_step": st["kernels_per_step"]})
+        out[name] = r
+        dec.destroy()
+        wmap.free()
+    return out
 
 
 def run_part(args):
@@ -751,6 +827,20 @@ def run_part(args):
                                "frac_hbm": round(nbytes / ms / 1e6 / peaks["hbm_gbs"], 4)}
             dec.destroy()
         line.update({"value": res["bs16"]["tokens_per_s"], "unit": "tokens/s at batch 16 (4 layers + head)", "higher_is_better": True, "c4": res})
+    elif name == "mukutar":
+        clk = ClockSampler(0)
+        sizes = [measure_mukutar(tl, ev, peaks, 2048, 16, 4, 5632), measure_mukutar(tl, ev, peaks, 4096, 32, 8, 14336)]
+        line.update({"sizes": sizes, "value": sizes[1]["mukutar"]["decode_tokens_per_s"], "unit": "tokens/s (width 4096, 6 layers + head, batch 1)", "higher_is_better": True, "clocks": clk.stop()})
+    elif name == "mukutar-3layer":
+        wmap = build_mukutar_map(tl, mukutar_cfg(4096, 32, 8, 14336, 3, 32768, 4096))
+        dec = tl.Decoder(None, wmap, max_seq=2304)
+        toks = [int(t) for t in np.random.default_rng(6).integers(0, 32768, 2048)]
+        for _ in range(2):
+            dec.prefill(toks, 0, read=False)
+            for i in range(4):
+                dec.step(1 + i, 2048 + i, read=False)
+        ms = time_events(tl, ev, lambda: dec.prefill(toks, 0, read=False), 1)
+        line.update({"value": round(2048 / ms * 1e3, 0), "unit": "prompt tokens/s (3 layers + head)", "ms": round(ms, 3), "higher_is_better": True})
     else:
         cfg = dict(synth.LLAMA3_8B, n_layers=2)
         wmap = tl.map_from_tensors(synth.llama_tensors(cfg, 1, 12, 14))

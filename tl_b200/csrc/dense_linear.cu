@@ -339,18 +339,46 @@ __global__ void __launch_bounds__(256) dense_gemm_f32_kernel(const DenseF32Param
 __device__ __forceinline__ void store_act(float *p, float v) { *p = v; }
 __device__ __forceinline__ void store_act(__nv_bfloat16 *p, float v) { *p = __float2bfloat16_rn(v); }
 
+__device__ __forceinline__ void store_act4(float *p, float a, float b, float c, float d) { *reinterpret_cast<float4 *>(p) = make_float4(a, b, c, d); }
+__device__ __forceinline__ void store_act4(__nv_bfloat16 *p, float a, float b, float c, float d)
+{
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(a, b), hi = __floats2bfloat162_rn(c, d);
+    *reinterpret_cast<uint2 *>(p) = make_uint2(*reinterpret_cast<const uint32_t *>(&lo), *reinterpret_cast<const uint32_t *>(&hi));
+}
+
 template <typename TA>
 __global__ void __launch_bounds__(256) norm_rows_kernel(const float *__restrict__ x, int width, const float *__restrict__ w, float offset, float eps,
                                                         TA *__restrict__ out, int ld)
 {
     __shared__ float red[8];
     const float *row = x + (size_t)blockIdx.x * width;
+    TA *o = out + (size_t)blockIdx.x * ld;
     float ss[1] = {0.f};
+    if (width % 4 == 0 && width <= 256 * 4 * 8) {       // the row stays in registers: one pass over memory
+        float4 v[8];
+        const int n4 = width / 4;
+#pragma unroll
+        for (int k = 0; k < 8; k++) {
+            const int i = threadIdx.x + k * 256;
+            v[k] = i < n4 ? reinterpret_cast<const float4 *>(row)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+            ss[0] += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+        }
+        block_sums(ss, red);
+        const float inv = 1.f / sqrtf(ss[0] / (float)width + eps);
+#pragma unroll
+        for (int k = 0; k < 8; k++) {
+            const int i = threadIdx.x + k * 256;
+            if (i < n4) {
+                const float4 g = reinterpret_cast<const float4 *>(w)[i];
+                store_act4(o + 4 * i, v[k].x * inv * (g.x + offset), v[k].y * inv * (g.y + offset), v[k].z * inv * (g.z + offset), v[k].w * inv * (g.w + offset));
+            }
+        }
+        return;
+    }
     for (int i = threadIdx.x; i < width; i += 256) ss[0] += row[i] * row[i];
     block_sums(ss, red);
     const float inv = 1.f / sqrtf(ss[0] / (float)width + eps);
-    TA *o = out + (size_t)blockIdx.x * ld;
-    for (int i = threadIdx.x; i < ld; i += 256) store_act(o + i, i < width ? row[i] * inv * (w[i] + offset) : 0.f);
+    for (int i = threadIdx.x; i < width; i += 256) store_act(o + i, row[i] * inv * (w[i] + offset));
 }
 
 template <typename TA>
@@ -359,19 +387,37 @@ __global__ void __launch_bounds__(512) poly_rows_kernel(const float *__restrict_
 {
     __shared__ float red[16 * 3];
     const float *row = z + (size_t)blockIdx.x * ldz;
-    float ss[3] = {0.f, 0.f, 0.f};
-    for (int i = threadIdx.x; i < ff; i += 512) {
-        const float v2 = row[i] * row[i];
-        ss[0] += v2; ss[1] += v2 * v2; ss[2] += v2 * v2 * v2;
-    }
-    block_sums(ss, red);
-    const float inv_n = 1.f / (float)ff;
-    const float a = coef[0] / sqrtf(ss[0] * inv_n + eps), b = coef[1] / sqrtf(ss[1] * inv_n + eps), c = coef[2] / sqrtf(ss[2] * inv_n + eps), d = coef[3];
     TA *o = out + (size_t)blockIdx.x * ld;
-    for (int i = threadIdx.x; i < ld; i += 512) {
-        const float v = i < ff ? row[i] : 0.f;
-        store_act(o + i, i < ff ? v * (a + v * (b + v * c)) + d : 0.f);
+    const float inv_n = 1.f / (float)ff;
+    float ss[3] = {0.f, 0.f, 0.f};
+    auto add = [&](float v) {
+        const float v2 = v * v;
+        ss[0] += v2; ss[1] += v2 * v2; ss[2] += v2 * v2 * v2;
+    };
+    if (ff % 4 == 0 && ff <= 512 * 4 * 8) {              // the row stays in registers
+        float4 v[8];
+        const int n4 = ff / 4;
+#pragma unroll
+        for (int k = 0; k < 8; k++) {
+            const int i = threadIdx.x + k * 512;
+            v[k] = i < n4 ? reinterpret_cast<const float4 *>(row)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int k = 0; k < 8; k++) { add(v[k].x); add(v[k].y); add(v[k].z); add(v[k].w); }
+        block_sums(ss, red);
+        const float a = coef[0] / sqrtf(ss[0] * inv_n + eps), b = coef[1] / sqrtf(ss[1] * inv_n + eps), c = coef[2] / sqrtf(ss[2] * inv_n + eps), d = coef[3];
+        auto act = [&](float x) { return x * (a + x * (b + x * c)) + d; };
+#pragma unroll
+        for (int k = 0; k < 8; k++) {
+            const int i = threadIdx.x + k * 512;
+            if (i < n4) store_act4(o + 4 * i, act(v[k].x), act(v[k].y), act(v[k].z), act(v[k].w));
+        }
+        return;
     }
+    for (int i = threadIdx.x; i < ff; i += 512) add(row[i]);
+    block_sums(ss, red);
+    const float a = coef[0] / sqrtf(ss[0] * inv_n + eps), b = coef[1] / sqrtf(ss[1] * inv_n + eps), c = coef[2] / sqrtf(ss[2] * inv_n + eps), d = coef[3];
+    for (int i = threadIdx.x; i < ff; i += 512) store_act(o + i, row[i] * (a + row[i] * (b + row[i] * c)) + d);
 }
 
 __global__ void embed_bf16_kernel(const int *__restrict__ tokens, const __nv_bfloat16 *__restrict__ table, int width, int ld, float *__restrict__ x)

@@ -378,15 +378,16 @@ tlb_status layered_step_batch(LayeredModel *lm, const int *tokens, const int *po
     const bool f32 = lm->cfg.f32;
     TLB_TRY(launch_embed_bf16(tokens, lm->embed, W, lm->embed_ld, x, batch));
     for (const Layer &L : lm->layers) {
-        TLB_TRY(launch_norm_rows(x, batch, W, L.norm1->f32(), off, eps, lm->act, lm->lda, f32));
-        TLB_TRY(rows_gemm(lm, L.in, lm->act, lm->lda, batch, lm->proj, lm->ldp, nullptr));
-        TLB_TRY(decode_mixer(lm, L, batch, pos, rope_pos, lm->act, lm->lda, f32, false));
-        TLB_TRY(rows_gemm(lm, L.o, lm->act, lm->lda, batch, x, W, L.ls1));
+        const int ldw = act_ld(W), ldo = act_ld(L.out_width), ldf = act_ld(L.up.n);
+        TLB_TRY(launch_norm_rows(x, batch, W, L.norm1->f32(), off, eps, lm->act, ldw, f32));
+        TLB_TRY(rows_gemm(lm, L.in, lm->act, ldw, batch, lm->proj, lm->ldp, nullptr));
+        TLB_TRY(decode_mixer(lm, L, batch, pos, rope_pos, lm->act, ldo, f32, false));
+        TLB_TRY(rows_gemm(lm, L.o, lm->act, ldo, batch, x, W, L.ls1));
         if (!L.up.w) continue;
-        TLB_TRY(launch_norm_rows(x, batch, W, L.norm2->f32(), off, eps, lm->act, lm->lda, f32));
-        TLB_TRY(rows_gemm(lm, L.up, lm->act, lm->lda, batch, lm->up, lm->ldu, nullptr));
-        TLB_TRY(launch_poly_rows(lm->up, batch, L.up.n, lm->ldu, L.act->f32(), eps, lm->act, lm->lda, f32));
-        TLB_TRY(rows_gemm(lm, L.down, lm->act, lm->lda, batch, x, W, L.ls2));
+        TLB_TRY(launch_norm_rows(x, batch, W, L.norm2->f32(), off, eps, lm->act, ldw, f32));
+        TLB_TRY(rows_gemm(lm, L.up, lm->act, ldw, batch, lm->up, lm->ldu, nullptr));
+        TLB_TRY(launch_poly_rows(lm->up, batch, L.up.n, lm->ldu, L.act->f32(), eps, lm->act, ldf, f32));
+        TLB_TRY(rows_gemm(lm, L.down, lm->act, ldf, batch, x, W, L.ls2));
     }
     return layered_head(lm, x, batch, logits);
 }
@@ -417,9 +418,9 @@ tlb_status layered_prefill(LayeredModel *lm, int seq, const int32_t *tokens, int
     if (n_want) TLB_CUDA(cudaMemcpyAsync(ids + T, want, (size_t)n_want * sizeof(int), cudaMemcpyHostToDevice, ctx()->stream));
     TLB_TRY(launch_embed_bf16(ids, lm->embed, W, lm->embed_ld, x, T));
     for (const Layer &L : lm->layers) {
-        const int lda = lm->lda, ldp = lm->ldp;
-        TLB_TRY(launch_norm_rows(x, T, W, L.norm1->f32(), off, eps, act, lda, f32));
-        TLB_TRY(rows_gemm(lm, L.in, act, lda, T, proj, ldp, nullptr));
+        const int ldp = lm->ldp, ldw = act_ld(W), lda = act_ld(L.out_width), ldf = act_ld(L.up.n);
+        TLB_TRY(launch_norm_rows(x, T, W, L.norm1->f32(), off, eps, act, ldw, f32));
+        TLB_TRY(rows_gemm(lm, L.in, act, ldw, T, proj, ldp, nullptr));
         if (L.d->mix.kind == MixerKind::Attention) {
             TLB_TRY(launch_mix_attn_prefill(attn_args(lm, L, proj, ldp), seq, T, pos0, act, lda, f32));
         } else if (L.d->mix.kind == MixerKind::Retention) {
@@ -431,10 +432,10 @@ tlb_status layered_prefill(LayeredModel *lm, int seq, const int32_t *tokens, int
         }
         TLB_TRY(rows_gemm(lm, L.o, act, lda, T, x, W, L.ls1));
         if (!L.up.w) continue;
-        TLB_TRY(launch_norm_rows(x, T, W, L.norm2->f32(), off, eps, act, lda, f32));
-        TLB_TRY(rows_gemm(lm, L.up, act, lda, T, u, lm->ldu, nullptr));
-        TLB_TRY(launch_poly_rows(u, T, L.up.n, lm->ldu, L.act->f32(), eps, act, lda, f32));
-        TLB_TRY(rows_gemm(lm, L.down, act, lda, T, x, W, L.ls2));
+        TLB_TRY(launch_norm_rows(x, T, W, L.norm2->f32(), off, eps, act, ldw, f32));
+        TLB_TRY(rows_gemm(lm, L.up, act, ldw, T, u, lm->ldu, nullptr));
+        TLB_TRY(launch_poly_rows(u, T, L.up.n, lm->ldu, L.act->f32(), eps, act, ldf, f32));
+        TLB_TRY(rows_gemm(lm, L.down, act, ldf, T, x, W, L.ls2));
     }
     if (n_want) TLB_TRY(launch_gather_rows(x, W, ids + T, n_want, rows_out));
     return TLB_OK;

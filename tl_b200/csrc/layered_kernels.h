@@ -48,7 +48,7 @@ struct DenseGemmJob {
 };
 tlb_status launch_dense_gemm(const DenseGemmJob &j, bool f32);
 
-// rows in the activation type, columns past the row's size zero up to ld
+// rows in the activation type, pitch ld
 tlb_status launch_norm_rows(const float *x, int T, int width, const float *w, float offset, float eps, void *out, int ld, bool f32);
 tlb_status launch_poly_rows(const float *z, int T, int ff, int ldz, const float *coef, float eps, void *out, int ld, bool f32);
 tlb_status launch_embed_bf16(const int *tokens, const __nv_bfloat16 *table, int width, int ld, float *x, int T);

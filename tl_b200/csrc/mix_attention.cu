@@ -1,6 +1,6 @@
 // Softmax attention with a sliding window, a per-head bias by distance and a sink, over a KV cache per sequence: the kernels
 // that take any head size and either cache type.
-//   mix_attn_decode_kernel   one new token per sequence: append, then 128 keys per CTA (16-byte loads, f32 arithmetic), merged by
+//   mix_attn_decode_kernel   one new token per sequence: append, then 64 keys per CTA (16-byte loads, f32 arithmetic), merged by
 //                            the last CTA of a (sequence, KV head)
 //   mix_attn_rows_kernel     many tokens, one warp per (token, head): f32 caches, and head sizes the tensor-core kernel does
 //                            not take (mix_attention_tc.cu)
@@ -14,7 +14,7 @@ namespace tlb {
 
 namespace {
 
-constexpr int kDecThreads = 256, kDecKeys = 128;
+constexpr int kDecThreads = 256, kDecKeys = 64;
 constexpr int kMaxHeadDim = 256;
 
 __device__ __forceinline__ void store_act(float *p, float v) { *p = v; }
@@ -59,7 +59,7 @@ __global__ void __launch_bounds__(kDecThreads) mix_attn_decode_kernel(const MixA
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int sp = blockIdx.x, g = blockIdx.y, b = blockIdx.z;
     const int rep = a.H / a.KVH, h0 = g * rep;
-    float *sq = dec_smem, *sp_w = sq + rep * a.ldk, *s_m = sp_w + rep * kDecKeys, *s_l = s_m + rep, *s_red = s_l + rep + (rep & 1) * 2;
+    float *sq = dec_smem, *sp_w = sq + rep * a.ldk, *s_b = sp_w + rep * kDecKeys, *s_m = s_b + rep * kDecKeys, *s_l = s_m + rep, *s_red = s_l + rep + (rep & 1) * 2;
     pdl_wait();
     pdl_launch_dependents();
     const int pos = j.pos[b];
@@ -73,6 +73,10 @@ __global__ void __launch_bounds__(kDecThreads) mix_attn_decode_kernel(const MixA
         const int r = i / a.ldk, d = i - r * a.ldk;
         sq[i] = d < a.D ? __ldcg(row + (size_t)(h0 + r) * a.D + d) : 0.f;
     }
+    for (int i = tid; i < rep * kDecKeys; i += kDecThreads) {
+        const int r = i / kDecKeys, key = i - r * kDecKeys;
+        s_b[i] = a.bias && key < nk ? a.bias[(size_t)(h0 + r) * a.bias_n + (pos - key0 - key)] : 0.f;
+    }
     if (sp == nsplit - 1) {          // the new token's rows: this CTA writes them and reads them back like any other
         const float *kn = row + (size_t)a.H * a.D + (size_t)g * a.D, *vn = row + (size_t)(a.H + a.KVH) * a.D + (size_t)g * a.DV;
         for (int d = tid; d < a.D; d += kDecThreads) store_cache(kc + (size_t)pos * a.ldk + d, __ldcg(kn + d));
@@ -85,35 +89,42 @@ __global__ void __launch_bounds__(kDecThreads) mix_attn_decode_kernel(const MixA
     int lpk = 1;
     while (lpk < nvk && lpk < 32) lpk *= 2;
     const int kpw = 32 / lpk, sub = lane / lpk, ln = lane % lpk;
-    for (int r0 = 0; r0 < rep; r0 += 8) {
-        const int nr = min(8, rep - r0);
-        for (int kk = warp * kpw; kk < nk; kk += (kDecThreads / 32) * kpw) {
-            const int key = kk + sub;
-            float acc[8] = {};
-            if (key < nk) {
-                const CT *kr = kc + (size_t)(key0 + key) * a.ldk;
-                for (int v = ln; v < nvk; v += lpk) {
-                    float kv[VE];
-                    Vec<CT>::load(kr + v * VE, kv);
+    constexpr int UK = 4;                       // keys in flight per lane
+    const int stride = (kDecThreads / 32) * kpw;
+    for (int r0 = 0; r0 < rep; r0 += 4) {
+        const int nr = min(4, rep - r0);
+        for (int kk = warp * kpw + sub; kk - sub < nk; kk += UK * stride) {
+            float acc[UK][4] = {};
+            for (int v = ln; v < nvk; v += lpk) {
+                float kv[UK][VE];
 #pragma unroll
-                    for (int r = 0; r < 8; r++) {
-                        if (r < nr) {
-                            const float *qr = sq + (r0 + r) * a.ldk + v * VE;
+                for (int u = 0; u < UK; u++) Vec<CT>::load(kc + (size_t)(key0 + min(kk + u * stride, nk - 1)) * a.ldk + v * VE, kv[u]);
 #pragma unroll
-                            for (int e = 0; e < VE; e++) acc[r] = fmaf(qr[e], kv[e], acc[r]);
+                for (int r = 0; r < 4; r++) {
+                    if (r < nr) {
+                        const float *qr = sq + (r0 + r) * a.ldk + v * VE;
+#pragma unroll
+                        for (int e = 0; e < VE; e++) {
+                            const float q = qr[e];
+#pragma unroll
+                            for (int u = 0; u < UK; u++) acc[u][r] = fmaf(q, kv[u][e], acc[u][r]);
                         }
                     }
                 }
             }
+            for (int o = lpk >> 1; o; o >>= 1) {
 #pragma unroll
-            for (int r = 0; r < 8; r++) {
-                if (r < nr) {
-                    for (int o = lpk >> 1; o; o >>= 1) acc[r] += __shfl_xor_sync(0xffffffffu, acc[r], o);
-                    if (ln == 0 && key < nk) {
-                        float s = acc[r] * a.scale;
-                        if (a.bias) s -= a.bias[(size_t)(h0 + r0 + r) * a.bias_n + (pos - key0 - key)];
-                        sp_w[(r0 + r) * kDecKeys + key] = s;
-                    }
+                for (int u = 0; u < UK; u++)
+#pragma unroll
+                    for (int r = 0; r < 4; r++) acc[u][r] += __shfl_xor_sync(0xffffffffu, acc[u][r], o);
+            }
+#pragma unroll
+            for (int u = 0; u < UK; u++) {
+                const int key = kk + u * stride;
+                if (ln == 0 && key < nk) {
+#pragma unroll
+                    for (int r = 0; r < 4; r++)
+                        if (r < nr) sp_w[(r0 + r) * kDecKeys + key] = acc[u][r] * a.scale - s_b[(r0 + r) * kDecKeys + key];
                 }
             }
         }
@@ -140,6 +151,7 @@ __global__ void __launch_bounds__(kDecThreads) mix_attn_decode_kernel(const MixA
         float acc[4][VE] = {};
         if (slice < ks) {
             const CT *vr = vc + (size_t)key0 * a.ldv + vec * VE;
+#pragma unroll 4
             for (int k = slice; k < nk; k += ks) {
                 float vv[VE];
                 Vec<CT>::load(vr + (size_t)k * a.ldv, vv);
@@ -162,6 +174,7 @@ __global__ void __launch_bounds__(kDecThreads) mix_attn_decode_kernel(const MixA
         for (int i = tid; i < nr * a.DV; i += kDecThreads) {
             const int r = i / a.DV, d = i - r * a.DV;
             float s = 0.f;
+#pragma unroll 8
             for (int k = 0; k < min(ks, nk); k++) s += s_red[((size_t)k * 4 + r) * a.ldv + d];
             const int rr = r0 + r;
             if (nsplit == 1) {
@@ -188,18 +201,30 @@ __global__ void __launch_bounds__(kDecThreads) mix_attn_decode_kernel(const MixA
     if (!last_cta) return;
     __threadfence();
     const float *pall = j.partial + (((size_t)b * a.KVH + g) * gridDim.x * rep) * prow;
+    // every split's factor exp(m - M) / denominator, a warp per head; then the weighted sums
+    float *s_f = s_red;
+    for (int r = warp; r < rep; r += kDecThreads / 32) {
+        float m = a.sink ? a.sink[h0 + r] : -INFINITY, den = 0.f;
+        for (int s = lane; s < nsplit; s += 32) m = fmaxf(m, __ldcg(pall + ((size_t)s * rep + r) * prow + a.ldv));
+        for (int o = 16; o; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+        for (int s = lane; s < nsplit; s += 32) {
+            const float *ps = pall + ((size_t)s * rep + r) * prow + a.ldv, f = expf(__ldcg(ps) - m);
+            s_f[r * nsplit + s] = f;
+            den += f * __ldcg(ps + 1);
+        }
+        for (int o = 16; o; o >>= 1) den += __shfl_xor_sync(0xffffffffu, den, o);
+        if (a.sink) den += expf(a.sink[h0 + r] - m);
+        __syncwarp();
+        for (int s = lane; s < nsplit; s += 32) s_f[r * nsplit + s] /= den;
+    }
+    __syncthreads();
     for (int i = tid; i < rep * a.DV; i += kDecThreads) {
         const int r = i / a.DV, d = i - r * a.DV;
-        float m = a.sink ? a.sink[h0 + r] : -INFINITY;
-        for (int s = 0; s < nsplit; s++) m = fmaxf(m, __ldcg(pall + ((size_t)s * rep + r) * prow + a.ldv));
-        float den = a.sink ? expf(a.sink[h0 + r] - m) : 0.f, o = 0.f;
-        for (int s = 0; s < nsplit; s++) {
-            const float *ps = pall + ((size_t)s * rep + r) * prow;
-            const float f = expf(__ldcg(ps + a.ldv) - m);
-            den += f * __ldcg(ps + a.ldv + 1);
-            o += f * __ldcg(ps + d);
-        }
-        store_act(out + (size_t)(h0 + r) * a.DV + d, o / den);
+        const float *ps = pall + (size_t)r * prow + d;
+        float o = 0.f;
+#pragma unroll 16
+        for (int s = 0; s < nsplit; s++) o = fmaf(s_f[r * nsplit + s], __ldcg(ps + (size_t)s * rep * prow), o);
+        store_act(out + (size_t)(h0 + r) * a.DV + d, o);
     }
     if (tid == 0) j.counters[b * a.KVH + g] = 0;
 }
@@ -284,7 +309,7 @@ tlb_status run_decode(const MixAttnDecode &j)
 {
     const MixAttn &a = j.a;
     const int rep = a.H / a.KVH;
-    const size_t smem = (size_t)(rep * a.ldk + rep * kDecKeys + 2 * rep + 2 + dec_red_floats<CT>()) * sizeof(float);
+    const size_t smem = (size_t)(rep * a.ldk + 2 * rep * kDecKeys + 2 * rep + 2 + std::max(dec_red_floats<CT>(), rep * decode_splits(a))) * sizeof(float);
     if (smem > ctx()->smem_optin) return fail(TLB_ERR_SHAPE, "attention: %d query heads per KV head of size %d do not fit shared memory", rep, a.D);
     static size_t allowed = 48 << 10;
     if (smem > allowed) {

@@ -37,6 +37,17 @@ __device__ __forceinline__ float lanes8_sum(float v)
     v += __shfl_xor_sync(0xffffffffu, v, 4);
     return v;
 }
+// Eight values per lane -> lane l (of eight) gets the sum over the lanes of value l: 4 + 2 + 1 shuffles instead of 24.
+__device__ __forceinline__ float lanes8_scatter(const float (&y)[8], int l)
+{
+    float a[4], b[2];
+    const bool u4 = l & 4, u2 = l & 2, u1 = l & 1;
+#pragma unroll
+    for (int i = 0; i < 4; i++) a[i] = (u4 ? y[i + 4] : y[i]) + __shfl_xor_sync(0xffffffffu, u4 ? y[i] : y[i + 4], 4);
+#pragma unroll
+    for (int i = 0; i < 2; i++) b[i] = (u2 ? a[i + 2] : a[i]) + __shfl_xor_sync(0xffffffffu, u2 ? a[i] : a[i + 2], 2);
+    return (u1 ? b[1] : b[0]) + __shfl_xor_sync(0xffffffffu, u1 ? b[0] : b[1], 1);
+}
 __device__ __forceinline__ float warp_sum(float v)
 {
 #pragma unroll
@@ -195,12 +206,21 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const ScanParams p)
         __syncthreads();
         const float *buf = scan_smem + b * kScanTok * ROW;
         const int nt = min(kScanTok, p.T - t0);
-#pragma unroll 2
-        for (int t = 0; t < nt; t++) {
+        auto token = [&](int t) {
             const float *r = buf + t * ROW;
             const float v = r[NV * DP + col];
-            const float y = DELTA ? S.delta(r, r + DP, r + 2 * DP, r + 3 * DP, v, l) : S.retain(r, r + DP, decay, v, l);
-            const float sum = lanes8_sum(y);
+            return DELTA ? S.delta(r, r + DP, r + 2 * DP, r + 3 * DP, v, l) : S.retain(r, r + DP, decay, v, l);
+        };
+        int t = 0;
+        for (; t + 8 <= nt; t += 8) {
+            float y[8];
+#pragma unroll
+            for (int i = 0; i < 8; i++) y[i] = token(t + i);
+            const float sum = lanes8_scatter(y, l);
+            if (live) o[(size_t)(t0 + t + l) * ldo] = sum;
+        }
+        for (; t < nt; t++) {
+            const float sum = lanes8_sum(token(t));
             if (l == 0 && live) o[(size_t)(t0 + t) * ldo] = sum;
         }
         __syncthreads();

@@ -164,3 +164,94 @@ def write_gguf(path, tensors, metadata=None, alignment=32):
         for name, (t, data, shape) in tensors.items():
             f.write(data.tobytes())
             f.write(b"\0" * ((alignment - data.size % alignment) % alignment))
+
+
+# ---- models described by a config.json (bf16 tensors) -----------------------------------------------------------
+BF16 = 30
+
+
+def to_bf16(a):
+    """f32 array -> bf16 bit patterns (uint16), round to nearest even."""
+    u = np.ascontiguousarray(a, dtype=np.float32).view(np.uint32)
+    return ((u + np.uint32(0x7FFF) + ((u >> np.uint32(16)) & np.uint32(1))) >> np.uint32(16)).astype(np.uint16)
+
+
+def from_bf16(u):
+    return (np.asarray(u, dtype=np.uint16).astype(np.uint32) << np.uint32(16)).view(np.float32)
+
+
+def mukutar_specs(cfg, rank=64):
+    """Name -> shape of every tensor of a Mukutar model with this config.json; rank: inner size of the decay's projection."""
+    W = cfg["width"]
+    s = {"embed": (cfg["vocab"], W), "head": (cfg["vocab"], W), "final.norm": (W,)}
+    for i, lay in enumerate(cfg["layers"]):
+        p, m = "l%d." % i, lay["mixer"]
+        q, H, D = p + "mix.", m["heads"], m["dim"]
+        s[p + "norm1"] = s[p + "ls1"] = (W,)
+        if lay["type"] == "attention":
+            G, DV = m["kv_heads"], m["vdim"]
+            for n, r in (("q", H * D), ("k", G * D), ("v", G * DV)):
+                s[q + n] = (r, W)
+                s[q + n + ".b"] = (r,)
+            s[q + "r1"] = s[q + "r2"] = s[q + "sink"] = (H,)
+        elif lay["type"] == "retention":
+            DV = m["vdim"]
+            for n, r in (("q", H * D), ("k", H * D), ("v", H * DV), ("g", H * DV)):
+                s[q + n] = (r, W)
+        else:
+            DV = D
+            for n in "rkvga":
+                s[q + n] = (H * D, W)
+            s[q + "a.b"] = s[q + "w0"] = s[q + "norm"] = (H * D,)
+            s[q + "w1"], s[q + "w2"] = (rank, W), (H * D, rank)
+        s[q + "o"] = (W, H * DV)
+        if lay.get("mlp"):
+            F = lay["mlp"]["ff"]
+            s[p + "norm2"] = s[p + "ls2"] = (W,)
+            s[p + "mlp.up"], s[p + "mlp.down"], s[p + "mlp.act"] = (F, W), (W, F), (4,)
+    return s
+
+
+def mukutar_tensor(name, shape, seed):
+    """Seeded f32 values of one tensor, of a size a trained model's could have; rounded to bf16 they are the stored ones."""
+    r = _rng(seed, name)
+    leaf = name.split(".", 1)[-1]
+    x = r.standard_normal(int(np.prod(shape)), dtype=np.float32).reshape(shape)
+    if len(shape) == 2:
+        return x if name == "embed" else x * np.float32(shape[1] ** -0.5)
+    if leaf.startswith("ls"):
+        return 0.5 + 0.1 * x
+    if leaf in ("mix.r1", "mix.r2"):
+        return 0.2 + 0.3 * np.abs(x)
+    if leaf == "mix.norm":
+        return 1.0 + 0.1 * x
+    if leaf == "mlp.act":
+        return np.float32(0.5) + 0.3 * x
+    if leaf in ("mix.sink", "mix.w0", "mix.a.b"):
+        return x
+    return 0.1 * x
+
+
+def mukutar_tensors(cfg, seed, rank=64):
+    """Name -> bf16 bits (uint16) of a whole model."""
+    return {n: to_bf16(mukutar_tensor(n, s, seed)) for n, s in mukutar_specs(cfg, rank).items()}
+
+
+def write_model_dir(path, cfg, tensors):
+    """A model folder: config.json and model.safetensors (bf16 bits as uint16, int32 and float32 arrays)."""
+    import json
+    import os
+    os.makedirs(path, exist_ok=True)
+    with open(os.path.join(path, "config.json"), "w") as f:
+        json.dump(cfg, f)
+    names = {"uint16": "BF16", "int32": "I32", "float32": "F32", "float16": "F16"}
+    head, at = {}, 0
+    for n, a in tensors.items():
+        head[n] = {"dtype": names[str(a.dtype)], "shape": list(a.shape), "data_offsets": [at, at + a.nbytes]}
+        at += a.nbytes
+    text = json.dumps(head).encode()
+    text += b" " * (-len(text) % 8)
+    with open(os.path.join(path, "model.safetensors"), "wb") as f:
+        f.write(struct.pack("<Q", len(text)) + text)
+        for a in tensors.values():
+            f.write(np.ascontiguousarray(a).tobytes())
