@@ -402,17 +402,18 @@ tlb_status layered_prefill(LayeredModel *lm, int seq, const int32_t *tokens, int
     Rows ws;
     int *ids;
     float *x, *proj, *u, *o, *dly = nullptr;
+    float2 *look = nullptr;
     void *act, *th = nullptr;
-    size_t n_dly = 0, n_th = 0;
+    size_t n_dly = 0, n_th = 0, n_look = 0;
     for (const Layer &L : lm->layers)
-        if (L.d->mix.kind == MixerKind::GeneralDelta) { n_dly = std::max(n_dly, (size_t)L.w2.n); n_th = std::max(n_th, (size_t)L.w2.k); }
+        if (L.d->mix.kind == MixerKind::GeneralDelta) { n_dly = std::max(n_dly, (size_t)L.w2.n); n_th = std::max(n_th, (size_t)L.w2.k); n_look = std::max(n_look, (size_t)L.d->mix.heads); }
     TLB_TRY(ws.get(&ids, ((size_t)T + std::max(n_want, 1)) * sizeof(int)));
     TLB_TRY(ws.get(&x, (size_t)T * W * 4));
     TLB_TRY(ws.get(&proj, (size_t)T * lm->ldp * 4));
     TLB_TRY(ws.get(&u, (size_t)T * lm->ldu * 4));
     TLB_TRY(ws.get(&o, (size_t)T * lm->ldm * 4));
     TLB_TRY(ws.get(&act, (size_t)T * lm->lda * es));
-    if (n_dly) { TLB_TRY(ws.get(&dly, (size_t)T * n_dly * 4)); TLB_TRY(ws.get(&th, (size_t)T * n_th * es)); }
+    if (n_dly) { TLB_TRY(ws.get(&dly, (size_t)T * n_dly * 4)); TLB_TRY(ws.get(&th, (size_t)T * n_th * es)); TLB_TRY(ws.get(&look, (size_t)T * n_look * sizeof(float2))); }
     // pageable sources: staged before the calls return
     TLB_CUDA(cudaMemcpyAsync(ids, tokens, (size_t)T * sizeof(int), cudaMemcpyHostToDevice, ctx()->stream));
     if (n_want) TLB_CUDA(cudaMemcpyAsync(ids + T, want, (size_t)n_want * sizeof(int), cudaMemcpyHostToDevice, ctx()->stream));
@@ -428,7 +429,7 @@ tlb_status layered_prefill(LayeredModel *lm, int seq, const int32_t *tokens, int
         } else {
             TLB_TRY(launch_tanh_split(proj + 5 * (size_t)L.w2.n, T, L.d->mix.rank, ldp, th, L.w2.k / 2, f32));
             TLB_TRY(rows_gemm(lm, L.w2, th, L.w2.k, T, dly, L.w2.n, nullptr));
-            TLB_TRY(launch_delta_prefill(recur_args(lm, L, proj, ldp), seq, T, pos0, dly, o, act, lda, f32));
+            TLB_TRY(launch_delta_prefill(recur_args(lm, L, proj, ldp), seq, T, pos0, dly, look, o, act, lda, f32));
         }
         TLB_TRY(rows_gemm(lm, L.o, act, lda, T, x, W, L.ls1));
         if (!L.up.w) continue;

@@ -121,8 +121,8 @@ tlb_status launch_retention_decode(const MixRecurDecode &j);
 tlb_status launch_delta_decode(const MixRecurDecode &j);
 // T tokens of one sequence; `o` is scratch [T, H * DV] f32; out in the activation type
 tlb_status launch_retention_prefill(const MixRecur &m, int seq, int T, int pos0, int rope0, int rope_step, float *o, void *out, int ldo, bool f32);
-// decay: scratch [T, H * D] f32 that holds W_w2 tanh(W_w1 h) on entry
-tlb_status launch_delta_prefill(const MixRecur &m, int seq, int T, int pos0, float *decay, float *o, void *out, int ldo, bool f32);
+// decay: scratch [T, H * D] f32 that holds W_w2 tanh(W_w1 h) on entry; look: scratch [T, H]
+tlb_status launch_delta_prefill(const MixRecur &m, int seq, int T, int pos0, float *decay, float2 *look, float *o, void *out, int ldo, bool f32);
 // tanh of the first step of the decay's projection as two activation-type terms (value and remainder): out [T, 2 * ldh]
 tlb_status launch_tanh_split(const float *x, int T, int rank, int ldx, void *out, int ldh, bool f32);
 

@@ -59,7 +59,7 @@ __global__ void __launch_bounds__(kDecThreads) mix_attn_decode_kernel(const MixA
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int sp = blockIdx.x, g = blockIdx.y, b = blockIdx.z;
     const int rep = a.H / a.KVH, h0 = g * rep;
-    float *sq = dec_smem, *sp_w = sq + rep * a.ldk, *s_b = sp_w + rep * kDecKeys, *s_m = s_b + rep * kDecKeys, *s_l = s_m + rep, *s_red = s_l + rep + (rep & 1) * 2;
+    float *sq = dec_smem, *sp_w = sq + rep * a.ldk, *s_b = sp_w + rep * kDecKeys, *s_m = s_b + rep * kDecKeys, *s_l = s_m + rep, *s_red = s_l + rep + (-2 * rep & 3);        // 16-byte aligned
     pdl_wait();
     pdl_launch_dependents();
     const int pos = j.pos[b];
@@ -104,10 +104,13 @@ __global__ void __launch_bounds__(kDecThreads) mix_attn_decode_kernel(const MixA
                     if (r < nr) {
                         const float *qr = sq + (r0 + r) * a.ldk + v * VE;
 #pragma unroll
-                        for (int e = 0; e < VE; e++) {
-                            const float q = qr[e];
+                        for (int e4 = 0; e4 < VE; e4 += 4) {
+                            const float4 q4 = *reinterpret_cast<const float4 *>(qr + e4);
+                            const float q[4] = {q4.x, q4.y, q4.z, q4.w};
 #pragma unroll
-                            for (int u = 0; u < UK; u++) acc[u][r] = fmaf(q, kv[u][e], acc[u][r]);
+                            for (int e = 0; e < 4; e++)
+#pragma unroll
+                                for (int u = 0; u < UK; u++) acc[u][r] = fmaf(q[e], kv[u][e4 + e], acc[u][r]);
                         }
                     }
                 }
@@ -168,7 +171,8 @@ __global__ void __launch_bounds__(kDecThreads) mix_attn_decode_kernel(const MixA
             for (int r = 0; r < 4; r++)
                 if (r < nr)
 #pragma unroll
-                    for (int e = 0; e < VE; e++) s_red[((size_t)slice * 4 + r) * a.ldv + vec * VE + e] = acc[r][e];
+                    for (int e = 0; e < VE; e += 4)
+                        *reinterpret_cast<float4 *>(s_red + ((size_t)slice * 4 + r) * a.ldv + vec * VE + e) = make_float4(acc[r][e], acc[r][e + 1], acc[r][e + 2], acc[r][e + 3]);
         }
         __syncthreads();
         for (int i = tid; i < nr * a.DV; i += kDecThreads) {
@@ -309,7 +313,7 @@ tlb_status run_decode(const MixAttnDecode &j)
 {
     const MixAttn &a = j.a;
     const int rep = a.H / a.KVH;
-    const size_t smem = (size_t)(rep * a.ldk + 2 * rep * kDecKeys + 2 * rep + 2 + std::max(dec_red_floats<CT>(), rep * decode_splits(a))) * sizeof(float);
+    const size_t smem = (size_t)(rep * a.ldk + 2 * rep * kDecKeys + 2 * rep + 4 + std::max(dec_red_floats<CT>(), rep * decode_splits(a))) * sizeof(float);
     if (smem > ctx()->smem_optin) return fail(TLB_ERR_SHAPE, "attention: %d query heads per KV head of size %d do not fit shared memory", rep, a.D);
     static size_t allowed = 48 << 10;
     if (smem > allowed) {

@@ -1,9 +1,9 @@
 // Linear recurrences with a matrix state per head, in 32-bit floats throughout.
 //   retention       S <- decay S + k v^T;                                        o = S^T q
 //   general delta   S <- diag(w) S - (a u)(u^T S) + k v^T,  u = k / |k|;         o = S^T r
-// The state's value channels (columns) never mix, so a column lives in the registers of eight lanes - lane l holds key channels
-// 32 c + 4 l .. + 3 - from the first token of a launch to the last: a prompt is scanned token by token exactly as decoding would
-// do it, whatever its length or the place where it was cut, with one shuffle reduction per product with the state.
+// The state's value channels (columns) never mix, so a column lives in the registers of a few lanes - each some
+// of its key channels - from the first token of a launch to the last: a prompt is scanned token by token as decoding would do it,
+// whatever its length or the place where it was cut.
 // State in memory: [sequence][head][value channel][key channel padded to a multiple of 32].
 // Around the scan: what enters it is prepared per token and head (rotation and scale; decay, removal vector), what leaves it is
 // divided by its root mean square per head and gated.  Decoding does all of it in one launch.
@@ -16,7 +16,7 @@ namespace tlb {
 
 namespace {
 
-constexpr int kScanThreads = 256, kScanCols = kScanThreads / 8, kScanTok = 16;
+constexpr int kScanThreads = 128, kScanTok = 16;
 constexpr int kStepThreads = 512, kStepCols = kStepThreads / 8;
 constexpr float kUnitEps = 1e-6f;             // inside the root of the unit key
 
@@ -36,17 +36,6 @@ __device__ __forceinline__ float lanes8_sum(float v)
     v += __shfl_xor_sync(0xffffffffu, v, 2);
     v += __shfl_xor_sync(0xffffffffu, v, 4);
     return v;
-}
-// Eight values per lane -> lane l (of eight) gets the sum over the lanes of value l: 4 + 2 + 1 shuffles instead of 24.
-__device__ __forceinline__ float lanes8_scatter(const float (&y)[8], int l)
-{
-    float a[4], b[2];
-    const bool u4 = l & 4, u2 = l & 2, u1 = l & 1;
-#pragma unroll
-    for (int i = 0; i < 4; i++) a[i] = (u4 ? y[i + 4] : y[i]) + __shfl_xor_sync(0xffffffffu, u4 ? y[i] : y[i + 4], 4);
-#pragma unroll
-    for (int i = 0; i < 2; i++) b[i] = (u2 ? a[i + 2] : a[i]) + __shfl_xor_sync(0xffffffffu, u2 ? a[i] : a[i + 2], 2);
-    return (u1 ? b[1] : b[0]) + __shfl_xor_sync(0xffffffffu, u1 ? b[0] : b[1], 1);
 }
 __device__ __forceinline__ float warp_sum(float v)
 {
@@ -134,10 +123,22 @@ struct Column {
 };
 
 // ================================================================ scan of a prompt
+// A group of L lanes owns CB columns; lane l of it holds key channels 4 (i L + l) .. + 3 for i < N4 of each, so a vector read from
+// shared memory (16 bytes per lane, without bank conflicts) serves CB columns.  The outputs of L / CB tokens are summed over the
+// lanes together: every lane ends up with one of them.
+// General delta: u^T S of the next token is taken from the state BEFORE this token's update,
+//   k'^T S_t = (k' w)^T S_(t-1) - (k' . rem) (k^T S_(t-1)) + (k' . k) v,
+// so its reduction over the lanes overlaps this token's update instead of standing in front of the next one.
+template <int NC> struct ScanShape {
+    static constexpr int DP = 32 * NC, L = NC % 2 ? 8 : 16, N4 = DP / (4 * L), CB = N4 <= 4 ? 4 : 2, TB = L / CB;
+    static constexpr int COLS = kScanThreads / L * CB;       // columns per CTA
+};
+
 struct ScanParams {
     int H, D, DV, T;
     const float *q, *k, *v, *w, *rem;         // row 0, head 0 of each; rows `ld*` apart, heads D (v: DV) apart
     int ldq, ldk, ldv, ldw, ldr;
+    const float2 *look;                       // general delta: [T][H] (k' . rem, k' . k) of the next token's key
     const float *decay;
     float *state;                             // [H][DV][32 NC]
     int from_zero;
@@ -148,84 +149,192 @@ __device__ __forceinline__ void cp_async4(void *dst, const void *src)
 {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
+__device__ __forceinline__ void cp_async8(void *dst, const void *src)
+{
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 8;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
 __device__ __forceinline__ void cp_async16(void *dst, const void *src)
 {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
 
+// N values per lane (N a power of two): afterwards lane l of every N consecutive lanes holds the sum over those N lanes of value
+// l, with N - 1 shuffles.
+template <int N>
+__device__ __forceinline__ float scatter_sum(const float (&y)[N], int l)
+{
+    if constexpr (N == 1) {
+        return y[0];
+    } else {
+        float a[N / 2];
+        const bool up = l & (N / 2);
+#pragma unroll
+        for (int i = 0; i < N / 2; i++) a[i] = (up ? y[i + N / 2] : y[i]) + __shfl_xor_sync(0xffffffffu, up ? y[i] : y[i + N / 2], N / 2);
+        return scatter_sum<N / 2>(a, l);
+    }
+}
+// sums of N values over L lanes, in every lane
+template <int N, int L>
+__device__ __forceinline__ void all_sum(float (&y)[N], int lane)
+{
+    float s = scatter_sum<N>(y, lane);
+#pragma unroll
+    for (int o = N; o < L; o <<= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+#pragma unroll
+    for (int c = 0; c < N; c++) y[c] = __shfl_sync(0xffffffffu, s, (lane & ~(N - 1)) | c);
+}
+
 template <int NC, bool DELTA>
 __global__ void __launch_bounds__(kScanThreads) scan_kernel(const ScanParams p)
 {
-    constexpr int DP = 32 * NC, NV = DELTA ? 4 : 2, ROW = NV * DP + kScanCols;
-    extern __shared__ __align__(16) float scan_smem[];       // [2][kScanTok][ROW]: vectors, then the CTA's value channels
-    const int tid = threadIdx.x, l = tid & 7, col = tid >> 3, h = blockIdx.y, c0 = blockIdx.x * kScanCols, gcol = c0 + col;
-    const bool live = gcol < p.DV;
-    for (int i = tid; i < 2 * kScanTok * ROW; i += kScanThreads) scan_smem[i] = 0.f;
+    using S = ScanShape<NC>;
+    constexpr int DP = S::DP, L = S::L, N4 = S::N4, CB = S::CB, TB = S::TB, COLS = S::COLS, NP = 2 * N4;
+    constexpr int NV = DELTA ? 4 : 2, ROW = NV * DP + COLS + 4, BUF = kScanTok * ROW + DP;     // k has one row more than the chunk
+    extern __shared__ __align__(16) float scan_smem[];       // [2][BUF]; a row: q, k, (w, rem), value channels, look-ahead products
+    const int tid = threadIdx.x, lane = tid & 31, l = lane % L, h = blockIdx.y, c0 = blockIdx.x * COLS, col = tid / L * CB;
+    for (int i = tid; i < 2 * BUF; i += kScanThreads) scan_smem[i] = 0.f;
     __syncthreads();
     const float *src[4] = {p.q + (size_t)h * p.D, p.k + (size_t)h * p.D, DELTA ? p.w + (size_t)h * p.D : nullptr, DELTA ? p.rem + (size_t)h * p.D : nullptr};
     const int lds[4] = {p.ldq, p.ldk, p.ldw, p.ldr};
     bool wide = p.D % 4 == 0;
 #pragma unroll
     for (int i = 0; i < NV; i++) wide = wide && lds[i] % 4 == 0 && (reinterpret_cast<uintptr_t>(src[i]) & 15) == 0;
-    const int nv = min(kScanCols, p.DV - c0);
+    const int nv = min(COLS, p.DV - c0);
     auto fetch = [&](int t0, float *buf) {
         const int nt = min(kScanTok, p.T - t0);
 #pragma unroll
         for (int i = 0; i < NV; i++) {
-            if (wide) {
-                const int per = p.D / 4;
-                for (int e = tid; e < nt * per; e += kScanThreads) {
-                    const int t = e / per, d = (e - t * per) * 4;
-                    cp_async16(buf + t * ROW + i * DP + d, src[i] + (size_t)(t0 + t) * lds[i] + d);
-                }
-            } else {
-                for (int e = tid; e < nt * p.D; e += kScanThreads) {
-                    const int t = e / p.D, d = e - t * p.D;
-                    cp_async4(buf + t * ROW + i * DP + d, src[i] + (size_t)(t0 + t) * lds[i] + d);
-                }
+            const int rows = DELTA && i == 1 ? min(kScanTok + 1, p.T - t0) : nt;      // the key behind the chunk comes too
+            const int step = wide ? 4 : 1, per = p.D / step;
+            for (int e = tid; e < rows * per; e += kScanThreads) {
+                const int t = e / per, d = (e - t * per) * step;
+                float *dst = buf + t * ROW + i * DP + d;
+                if (i == 1 && t == kScanTok) dst = buf + kScanTok * ROW + d;
+                const float *s = src[i] + (size_t)(t0 + t) * lds[i] + d;
+                if (wide) cp_async16(dst, s);
+                else cp_async4(dst, s);
             }
         }
         for (int e = tid; e < nt * nv; e += kScanThreads) {
             const int t = e / nv, d = e - t * nv;
             cp_async4(buf + t * ROW + NV * DP + d, p.v + (size_t)(t0 + t) * p.ldv + (size_t)h * p.DV + c0 + d);
         }
+        if (DELTA)
+            for (int t = tid; t < nt; t += kScanThreads) cp_async8(buf + t * ROW + NV * DP + COLS, p.look + (size_t)(t0 + t) * p.H + h);
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    float *st = p.state + ((size_t)h * p.DV + gcol) * DP;
-    Column<NC> S;
-    if (live && !p.from_zero) S.load(st, l);
-    else S.zero();
+    auto vec = [&](const float *row, f2 (&x)[NP]) {
+#pragma unroll
+        for (int i = 0; i < N4; i++) lds_f2x2(row + 4 * (i * L + l), x[2 * i], x[2 * i + 1]);
+    };
+    f2 st[CB][NP];
+#pragma unroll
+    for (int c = 0; c < CB; c++) {
+        const int gc = c0 + col + c;
+        const float *sp = p.state + ((size_t)h * p.DV + gc) * DP;
+#pragma unroll
+        for (int i = 0; i < N4; i++) {
+            ulonglong2 x = make_ulonglong2(0ull, 0ull);
+            if (gc < p.DV && !p.from_zero) x = __ldcg(reinterpret_cast<const ulonglong2 *>(sp + 4 * (i * L + l)));
+            st[c][2 * i] = x.x; st[c][2 * i + 1] = x.y;
+        }
+    }
     const f2 decay = DELTA ? 0ull : pack2(p.decay[h], p.decay[h]);
-    float *o = p.o + (size_t)h * p.DV + gcol;
     const size_t ldo = (size_t)p.H * p.DV;
+    float *o = p.o + (size_t)h * p.DV + c0 + col;
+    auto dot = [&](const f2 (&x)[NP], const f2 (&s)[NP]) {
+        f2 a = mul2(x[0], s[0]), b = mul2(x[1], s[1]);
+#pragma unroll
+        for (int i = 2; i < NP; i += 2) { a = fma2(x[i], s[i], a); b = fma2(x[i + 1], s[i + 1], b); }
+        return sum2(add2(a, b));
+    };
+    f2 kc[NP];                    // general delta: this token's key, and k^T S of it per column
+    float ks[CB];
+    // one token: the state moves on, y = this lane's share of the outputs
+    auto token = [&](const float *r, const float *knext, float *y) {
+        float v[CB];
+#pragma unroll
+        for (int c = 0; c < CB; c++) v[c] = r[NV * DP + col + c];
+        f2 q[NP];
+        if (DELTA) {
+            const float2 lk = *reinterpret_cast<const float2 *>(r + NV * DP + COLS);
+            f2 kn[NP], w[NP], x[NP];
+            vec(knext, kn);
+            vec(r + 2 * DP, w);
+            float d[CB];
+#pragma unroll
+            for (int i = 0; i < NP; i++) x[i] = mul2(kn[i], w[i]);
+#pragma unroll
+            for (int c = 0; c < CB; c++) d[c] = dot(x, st[c]);
+            all_sum<CB, L>(d, lane);
+            vec(r + 3 * DP, x);
+            vec(r, q);
+#pragma unroll
+            for (int c = 0; c < CB; c++) {
+                const f2 vv = pack2(v[c], v[c]), kk = pack2(-ks[c], -ks[c]);
+#pragma unroll
+                for (int i = 0; i < NP; i++) st[c][i] = fma2(w[i], st[c][i], fma2(x[i], kk, mul2(kc[i], vv)));
+                y[c] = dot(q, st[c]);
+                ks[c] = d[c] - lk.x * ks[c] + lk.y * v[c];
+            }
+#pragma unroll
+            for (int i = 0; i < NP; i++) kc[i] = kn[i];
+        } else {
+            f2 k[NP];
+            vec(r + DP, k);
+            vec(r, q);
+#pragma unroll
+            for (int c = 0; c < CB; c++) {
+                const f2 vv = pack2(v[c], v[c]);
+#pragma unroll
+                for (int i = 0; i < NP; i++) st[c][i] = fma2(decay, st[c][i], mul2(k[i], vv));
+                y[c] = dot(q, st[c]);
+            }
+        }
+    };
     fetch(0, scan_smem);
     for (int t0 = 0, b = 0; t0 < p.T; t0 += kScanTok, b ^= 1) {
-        if (t0 + kScanTok < p.T) fetch(t0 + kScanTok, scan_smem + (b ^ 1) * kScanTok * ROW);
+        if (t0 + kScanTok < p.T) fetch(t0 + kScanTok, scan_smem + (b ^ 1) * BUF);
         else asm volatile("cp.async.commit_group;" ::: "memory");
         asm volatile("cp.async.wait_group 1;" ::: "memory");
         __syncthreads();
-        const float *buf = scan_smem + b * kScanTok * ROW;
+        const float *buf = scan_smem + b * BUF;
         const int nt = min(kScanTok, p.T - t0);
-        auto token = [&](int t) {
-            const float *r = buf + t * ROW;
-            const float v = r[NV * DP + col];
-            return DELTA ? S.delta(r, r + DP, r + 2 * DP, r + 3 * DP, v, l) : S.retain(r, r + DP, decay, v, l);
-        };
-        int t = 0;
-        for (; t + 8 <= nt; t += 8) {
-            float y[8];
+        if (DELTA && t0 == 0) {
+            vec(buf + DP, kc);
 #pragma unroll
-            for (int i = 0; i < 8; i++) y[i] = token(t + i);
-            const float sum = lanes8_scatter(y, l);
-            if (live) o[(size_t)(t0 + t + l) * ldo] = sum;
+            for (int c = 0; c < CB; c++) ks[c] = dot(kc, st[c]);
+            all_sum<CB, L>(ks, lane);
+        }
+        auto next_key = [&](int t) { return t + 1 < kScanTok ? buf + (t + 1) * ROW + DP : buf + kScanTok * ROW; };   // past the last token: anything, unused
+        int t = 0;
+        for (; t + TB <= nt; t += TB) {
+            float y[TB * CB];
+#pragma unroll
+            for (int i = 0; i < TB; i++) token(buf + (t + i) * ROW, next_key(t + i), y + i * CB);
+            const float sum = scatter_sum<TB * CB>(y, l);
+            const int yt = l / CB, yc = l % CB;
+            if (c0 + col + yc < p.DV) o[(size_t)(t0 + t + yt) * ldo + yc] = sum;
         }
         for (; t < nt; t++) {
-            const float sum = lanes8_sum(token(t));
-            if (l == 0 && live) o[(size_t)(t0 + t) * ldo] = sum;
+            float y[CB];
+            token(buf + t * ROW, next_key(t), y);
+            all_sum<CB, L>(y, lane);
+#pragma unroll
+            for (int c = 0; c < CB; c++)
+                if (l == c && c0 + col + c < p.DV) o[(size_t)(t0 + t) * ldo + c] = y[c];
         }
         __syncthreads();
     }
-    if (live) S.store(st, l);
+#pragma unroll
+    for (int c = 0; c < CB; c++) {
+        const int gc = c0 + col + c;
+        float *sp = p.state + ((size_t)h * p.DV + gc) * DP;
+        if (gc < p.DV) {
+#pragma unroll
+            for (int i = 0; i < N4; i++) *reinterpret_cast<ulonglong2 *>(sp + 4 * (i * L + l)) = make_ulonglong2(st[c][2 * i], st[c][2 * i + 1]);
+        }
+    }
 }
 
 // ---- what enters the scan
@@ -251,8 +360,9 @@ __global__ void retention_prep_kernel(const MixRecur m, int rope0, int rope_step
     }
 }
 
-// one warp per (token, head): decay <- exp(-exp(-1/2) sigmoid(decay + w0)), a <- sigmoid(a) k / (k . k + eps).  The bias of a is in already.
-__global__ void __launch_bounds__(256) delta_prep_kernel(const MixRecur m, int T, float *__restrict__ decay)
+// one warp per (token, head): decay <- exp(-exp(-1/2) sigmoid(decay + w0)), a <- sigmoid(a) k / (k . k + eps), and the two products
+// with the next token's key that the scan looks ahead with.  The bias of a is in already.
+__global__ void __launch_bounds__(256) delta_prep_kernel(const MixRecur m, int T, float *__restrict__ decay, float2 *__restrict__ look)
 {
     const int lane = threadIdx.x & 31;
     const int64_t u = (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5);
@@ -266,10 +376,18 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const MixRecur m, int T
     for (int d = lane; d < m.D; d += 32) ss += k[d] * k[d];
     ss = 1.f / (warp_sum(ss) + kUnitEps);
     const float rate = expf(-0.5f);
+    const float *kn = t + 1 < T ? k + m.ldp : k;
+    float kr = 0.f, kk = 0.f;
     for (int d = lane; d < m.D; d += 32) {
         dc[d] = expf(-rate * sigmoid_f(dc[d] + w0[d]));
-        a[d] = sigmoid_f(a[d]) * k[d] * ss;
+        const float rem = sigmoid_f(a[d]) * k[d] * ss;
+        a[d] = rem;
+        kr += kn[d] * rem;
+        kk += kn[d] * k[d];
     }
+    kr = warp_sum(kr);
+    kk = warp_sum(kk);
+    if (lane == 0) look[u] = make_float2(kr, kk);
 }
 
 __device__ __forceinline__ float gate_value(bool delta, float y, float g, float nw) { return delta ? y * nw * sigmoid_f(g) : y * (g * sigmoid_f(g)); }
@@ -413,14 +531,14 @@ __global__ void __launch_bounds__(kStepThreads) recur_step_kernel(const MixRecur
 template <int NC, bool DELTA>
 tlb_status scan_nc(const ScanParams &p)
 {
-    constexpr int ROW = (DELTA ? 4 : 2) * 32 * NC + kScanCols;
-    const size_t smem = (size_t)2 * kScanTok * ROW * sizeof(float);
+    constexpr int COLS = ScanShape<NC>::COLS, ROW = (DELTA ? 4 : 2) * 32 * NC + COLS + 4;
+    const size_t smem = (size_t)2 * (kScanTok * ROW + 32 * NC) * sizeof(float);
     static bool set = false;
     if (!set) {
         TLB_CUDA(cudaFuncSetAttribute(scan_kernel<NC, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         set = true;
     }
-    scan_kernel<NC, DELTA><<<dim3((p.DV + kScanCols - 1) / kScanCols, p.H), kScanThreads, smem, ctx()->stream>>>(p);
+    scan_kernel<NC, DELTA><<<dim3((p.DV + COLS - 1) / COLS, p.H), kScanThreads, smem, ctx()->stream>>>(p);
     TLB_CUDA(cudaGetLastError());
     count_launch();
     return TLB_OK;
@@ -506,10 +624,10 @@ tlb_status launch_retention_prefill(const MixRecur &m, int seq, int T, int pos0,
     return post(m, T, o, 2 * HD + m.H * m.DV, out, ldo, f32);
 }
 
-tlb_status launch_delta_prefill(const MixRecur &m, int seq, int T, int pos0, float *decay, float *o, void *out, int ldo, bool f32)
+tlb_status launch_delta_prefill(const MixRecur &m, int seq, int T, int pos0, float *decay, float2 *look, float *o, void *out, int ldo, bool f32)
 {
     const int HD = m.H * m.D;
-    delta_prep_kernel<<<(unsigned)(((int64_t)T * m.H + 7) / 8), 256, 0, ctx()->stream>>>(m, T, decay);
+    delta_prep_kernel<<<(unsigned)(((int64_t)T * m.H + 7) / 8), 256, 0, ctx()->stream>>>(m, T, decay, look);
     TLB_CUDA(cudaGetLastError());
     count_launch();
     ScanParams p = {};
@@ -517,6 +635,7 @@ tlb_status launch_delta_prefill(const MixRecur &m, int seq, int T, int pos0, flo
     p.q = m.proj; p.k = m.proj + HD; p.v = m.proj + 2 * HD; p.w = decay; p.rem = m.proj + 4 * (size_t)HD;
     p.ldq = p.ldk = p.ldv = p.ldr = m.ldp;
     p.ldw = HD;
+    p.look = look;
     p.state = m.state + (size_t)seq * m.seq_stride;
     p.from_zero = pos0 == 0;
     p.o = o;
