@@ -423,6 +423,15 @@ __global__ void __launch_bounds__(512) poly_rows_kernel(const float *__restrict_
 __global__ void embed_bf16_kernel(const int *__restrict__ tokens, const __nv_bfloat16 *__restrict__ table, int width, int ld, float *__restrict__ x)
 {
     const __nv_bfloat16 *src = table + (size_t)tokens[blockIdx.x] * ld;
+    if (width % 8 == 0) {
+        float4 *dst = reinterpret_cast<float4 *>(x + (size_t)blockIdx.x * width);
+        for (int i = threadIdx.x; i < width / 8; i += blockDim.x) {
+            const uint4 v = reinterpret_cast<const uint4 *>(src)[i];
+            dst[2 * i] = make_float4(bf_lo(v.x), bf_hi(v.x), bf_lo(v.y), bf_hi(v.y));
+            dst[2 * i + 1] = make_float4(bf_lo(v.z), bf_hi(v.z), bf_lo(v.w), bf_hi(v.w));
+        }
+        return;
+    }
     for (int i = threadIdx.x; i < width; i += blockDim.x) x[(size_t)blockIdx.x * width + i] = __bfloat162float(src[i]);
 }
 

@@ -413,7 +413,7 @@ tlb_status layered_prefill(LayeredModel *lm, int seq, const int32_t *tokens, int
     TLB_TRY(ws.get(&u, (size_t)T * lm->ldu * 4));
     TLB_TRY(ws.get(&o, (size_t)T * lm->ldm * 4));
     TLB_TRY(ws.get(&act, (size_t)T * lm->lda * es));
-    if (n_dly) { TLB_TRY(ws.get(&dly, (size_t)T * n_dly * 4)); TLB_TRY(ws.get(&th, (size_t)T * n_th * es)); TLB_TRY(ws.get(&look, (size_t)T * n_look * sizeof(float2))); }
+    if (n_dly) { TLB_TRY(ws.get(&dly, (size_t)T * n_dly * 4)); TLB_TRY(ws.get(&th, (size_t)T * n_th * es)); TLB_TRY(ws.get(&look, (size_t)scan_look_ld(T) * n_look * sizeof(float2))); }
     // pageable sources: staged before the calls return
     TLB_CUDA(cudaMemcpyAsync(ids, tokens, (size_t)T * sizeof(int), cudaMemcpyHostToDevice, ctx()->stream));
     if (n_want) TLB_CUDA(cudaMemcpyAsync(ids + T, want, (size_t)n_want * sizeof(int), cudaMemcpyHostToDevice, ctx()->stream));

@@ -88,6 +88,8 @@ tlb_status launch_mix_attn_prefill(const MixAttn &a, int seq, int T, int pos0, v
 bool mix_attn_supported(int D, int DV);
 tlb_status launch_mix_attn_prefill_tc(const MixAttn &a, int seq, int T, int pos0, void *out, int ldo);   // mix_attention_tc.cu: f16 cache
 bool mix_attn_prefill_tc_supported(int D, int DV);
+tlb_status launch_mix_attn_prefill_tc5(const MixAttn &a, int seq, int T, int pos0, void *out, int ldo);  // prefill_attn_tc.cu: f16 cache, tcgen05
+bool mix_attn_prefill_tc5_supported(int D, int DV, int T);
 
 // ---------------------------------------------------------------- mix_recurrent.cu
 // Linear recurrences with a matrix state per head, S[value channel][key channel] (key channels padded to ld), f32.
@@ -121,7 +123,8 @@ tlb_status launch_retention_decode(const MixRecurDecode &j);
 tlb_status launch_delta_decode(const MixRecurDecode &j);
 // T tokens of one sequence; `o` is scratch [T, H * DV] f32; out in the activation type
 tlb_status launch_retention_prefill(const MixRecur &m, int seq, int T, int pos0, int rope0, int rope_step, float *o, void *out, int ldo, bool f32);
-// decay: scratch [T, H * D] f32 that holds W_w2 tanh(W_w1 h) on entry; look: scratch [T, H]
+// decay: scratch [T, H * D] f32 that holds W_w2 tanh(W_w1 h) on entry; look: scratch [H, scan_look_ld(T)]
+int scan_look_ld(int T);
 tlb_status launch_delta_prefill(const MixRecur &m, int seq, int T, int pos0, float *decay, float2 *look, float *o, void *out, int ldo, bool f32);
 // tanh of the first step of the decay's projection as two activation-type terms (value and remainder): out [T, 2 * ldh]
 tlb_status launch_tanh_split(const float *x, int T, int rank, int ldx, void *out, int ldh, bool f32);

@@ -146,7 +146,7 @@ __global__ void __launch_bounds__(kDecThreads) mix_attn_decode_kernel(const MixA
 
     // weighted sum of V: a thread owns 16 bytes of the row for every ks-th key
     const int nvv = a.ldv / VE, ks = kDecThreads / nvv, vec = tid % nvv, slice = tid / nvv;
-    const int prow = a.ldv + 2;
+    const int prow = a.ldv + 4;                 // weighted sums, maximum, sum of exponentials; whole 16-byte lines
     float *part = j.partial + ((((size_t)b * a.KVH + g) * gridDim.x + sp) * rep) * prow;
     TO *out = reinterpret_cast<TO *>(j.out) + (size_t)b * j.ldo;
     for (int r0 = 0; r0 < rep; r0 += 4) {
@@ -222,13 +222,36 @@ __global__ void __launch_bounds__(kDecThreads) mix_attn_decode_kernel(const MixA
         for (int s = lane; s < nsplit; s += 32) s_f[r * nsplit + s] /= den;
     }
     __syncthreads();
-    for (int i = tid; i < rep * a.DV; i += kDecThreads) {
-        const int r = i / a.DV, d = i - r * a.DV;
-        const float *ps = pall + (size_t)r * prow + d;
-        float o = 0.f;
+    // 16 bytes of a head's row per thread; the splits are dealt over as many threads as there are
+    const int q4 = a.ldv / 4, items = rep * q4, ng = max(1, kDecThreads / items), sub_s = (nsplit + ng - 1) / ng;
+    float4 *s_o = reinterpret_cast<float4 *>(s_red + (rep * nsplit + 3) / 4 * 4);      // ng > 1: [ng][items]
+    for (int i0 = 0; i0 < items; i0 += kDecThreads) {
+        const int item = i0 + (ng > 1 ? tid % items : tid), gr = ng > 1 ? tid / items : 0;
+        const bool in = item < items && gr < ng;
+        const int r = in ? item / q4 : 0, d = in ? (item - r * q4) * 4 : 0;
+        float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (in) {
+            const float *ps = pall + (size_t)r * prow + d;
+            const int s1 = min(nsplit, (gr + 1) * sub_s);
 #pragma unroll 16
-        for (int s = 0; s < nsplit; s++) o = fmaf(s_f[r * nsplit + s], __ldcg(ps + (size_t)s * rep * prow), o);
-        store_act(out + (size_t)(h0 + r) * a.DV + d, o);
+            for (int s = gr * sub_s; s < s1; s++) {
+                const float4 x = __ldcg(reinterpret_cast<const float4 *>(ps + (size_t)s * rep * prow));
+                const float f = s_f[r * nsplit + s];
+                o.x = fmaf(f, x.x, o.x); o.y = fmaf(f, x.y, o.y); o.z = fmaf(f, x.z, o.z); o.w = fmaf(f, x.w, o.w);
+            }
+            if (gr > 0) s_o[gr * items + item] = o;
+        }
+        if (ng > 1) __syncthreads();
+        if (in && gr == 0) {
+            for (int k = 1; k < ng; k++) {
+                const float4 x = s_o[k * items + item];
+                o.x += x.x; o.y += x.y; o.z += x.z; o.w += x.w;
+            }
+            const float v[4] = {o.x, o.y, o.z, o.w};
+#pragma unroll
+            for (int e = 0; e < 4; e++)
+                if (d + e < a.DV) store_act(out + (size_t)(h0 + r) * a.DV + d + e, v[e]);
+        }
     }
     if (tid == 0) j.counters[b * a.KVH + g] = 0;
 }
@@ -313,7 +336,7 @@ tlb_status run_decode(const MixAttnDecode &j)
 {
     const MixAttn &a = j.a;
     const int rep = a.H / a.KVH;
-    const size_t smem = (size_t)(rep * a.ldk + 2 * rep * kDecKeys + 2 * rep + 4 + std::max(dec_red_floats<CT>(), rep * decode_splits(a))) * sizeof(float);
+    const size_t smem = (size_t)(rep * a.ldk + 2 * rep * kDecKeys + 2 * rep + 4 + std::max(dec_red_floats<CT>(), rep * decode_splits(a) + 4 + 4 * kDecThreads)) * sizeof(float);
     if (smem > ctx()->smem_optin) return fail(TLB_ERR_SHAPE, "attention: %d query heads per KV head of size %d do not fit shared memory", rep, a.D);
     static size_t allowed = 48 << 10;
     if (smem > allowed) {
@@ -329,7 +352,7 @@ tlb_status run_decode(const MixAttnDecode &j)
 
 bool mix_attn_supported(int D, int DV) { return D >= 1 && D <= kMaxHeadDim && DV >= 1 && DV <= kMaxHeadDim; }
 
-size_t mix_attn_decode_partial_floats(const MixAttn &a, int batch) { return (size_t)batch * a.KVH * decode_splits(a) * (a.H / a.KVH) * (a.ldv + 2); }
+size_t mix_attn_decode_partial_floats(const MixAttn &a, int batch) { return (size_t)batch * a.KVH * decode_splits(a) * (a.H / a.KVH) * (a.ldv + 4); }
 
 tlb_status launch_mix_attn_decode(const MixAttnDecode &j)
 {
@@ -345,6 +368,7 @@ tlb_status launch_mix_attn_prefill(const MixAttn &a, int seq, int T, int pos0, v
     else mix_attn_append_kernel<__half><<<T, 256, 0, c->stream>>>(a, seq, pos0);
     count_launch();
     TLB_CUDA(cudaGetLastError());
+    if (!f32 && mix_attn_prefill_tc5_supported(a.D, a.DV, T)) return launch_mix_attn_prefill_tc5(a, seq, T, pos0, out, ldo);
     if (!f32 && mix_attn_prefill_tc_supported(a.D, a.DV)) return launch_mix_attn_prefill_tc(a, seq, T, pos0, out, ldo);
     const dim3 grid((T + kRowWarps - 1) / kRowWarps, a.H);
     if (f32) mix_attn_rows_kernel<float, float><<<grid, kRowWarps * 32, 0, c->stream>>>(a, seq, T, pos0, (float *)out, ldo);

@@ -71,20 +71,17 @@ mix_attn_tc_kernel(const MixAttn a, int seq, int T, int pos0, __nv_bfloat16 *__r
     const int t_end = (pos0 + last_q) / kK + 1, t_begin = max(0, pos0 + qb - a.window + 1) / kK;
     auto tile_async = [&](int t) {
         __half *ks = at_smem + (size_t)(t & 1) * 2 * kK * RS, *vs = ks + kK * RS;
-        const int nk = a.ldk / 8, nv = a.ldv / 8;
-        for (int i = tid; i < kK * nk; i += kThreads) {
-            const int key = i / nk, ch = i - key * nk;
-            cp_async16(smem_u32(ks + key * RS + ch * 8), kc + (size_t)min(t * kK + key, a.max_seq - 1) * a.ldk + ch * 8);
-        }
-        for (int i = tid; i < kK * nv; i += kThreads) {
-            const int key = i / nv, ch = i - key * nv;
-            cp_async16(smem_u32(vs + key * RS + ch * 8), vc + (size_t)min(t * kK + key, a.max_seq - 1) * a.ldv + ch * 8);
+        constexpr int CW = P <= 128 ? 16 : 32;               // threads per row
+        const int ch = tid % CW;
+        for (int key = tid / CW; key < kK; key += kThreads / CW) {
+            const size_t row = min(t * kK + key, a.max_seq - 1);
+            if (ch * 8 < a.ldk) cp_async16(smem_u32(ks + key * RS + ch * 8), kc + row * a.ldk + ch * 8);
+            if (ch * 8 < a.ldv) cp_async16(smem_u32(vs + key * RS + ch * 8), vc + row * a.ldv + ch * 8);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
-        if (a.bias) {      // entry i: distance (first query of the CTA) - (last key of the tile) + i
-            const int d = pos0 + qb - (t * kK + kK - 1) + tid;
-            s_bias[(t & 1) * 128 + tid] = kLog2e * a.bias[(size_t)h * a.bias_n + min(max(d, 0), a.bias_n - 1)];
-        }
+        // entry i: distance (first query of the CTA) - (last key of the tile) + i
+        const int dist = pos0 + qb - (t * kK + kK - 1) + tid;
+        s_bias[(t & 1) * 128 + tid] = a.bias ? kLog2e * a.bias[(size_t)h * a.bias_n + min(max(dist, 0), a.bias_n - 1)] : 0.f;
     };
     tile_async(t_begin);
     __syncthreads();
@@ -129,28 +126,38 @@ mix_attn_tc_kernel(const MixAttn a, int seq, int T, int pos0, __nv_bfloat16 *__r
                 ldmatrix_x4(q_addr + ks * 32 + 32, q2[1][0], q2[1][1], q2[1][2], q2[1][3]);
             }
 #pragma unroll
-            for (int nb = 0; nb < kK / 8; nb++) {
-                uint32_t b0, b1, b2, b3;
-                ldmatrix_x4(smem_u32(Ks + (nb * 8 + (lane & 7)) * RS + (lane >> 3) * 8 + ks * 16), b0, b1, b2, b3);
-                hmma16816(s[nb], q2[0][0], q2[0][1], q2[0][2], q2[0][3], b0, b1);
-                hmma16816(s[nb], q2[1][0], q2[1][1], q2[1][2], q2[1][3], b2, b3);
+            for (int n4 = 0; n4 < kK / 8; n4 += 4) {           // four independent accumulators between two uses of one
+                uint32_t kb[4][4];
+#pragma unroll
+                for (int i = 0; i < 4; i++)
+                    ldmatrix_x4(smem_u32(Ks + ((n4 + i) * 8 + (lane & 7)) * RS + (lane >> 3) * 8 + ks * 16), kb[i][0], kb[i][1], kb[i][2], kb[i][3]);
+#pragma unroll
+                for (int i = 0; i < 4; i++) hmma16816(s[n4 + i], q2[0][0], q2[0][1], q2[0][2], q2[0][3], kb[i][0], kb[i][1]);
+#pragma unroll
+                for (int i = 0; i < 4; i++) hmma16816(s[n4 + i], q2[1][0], q2[1][1], q2[1][2], q2[1][3], kb[i][2], kb[i][3]);
             }
         }
         // inside = every key of the tile is seen by every query of the warp
         const bool inside = key0 + kK - 1 <= pos0 + q0 && key0 > pos0 + q0 + 15 - a.window;
+        const float *bt = s_bias + (t & 1) * 128 + warp * 16 + g + (kK - 1) - 2 * c;       // minus 8 nb + e of the key, plus 8 for row 1
+#pragma unroll
+        for (int nb = 0; nb < kK / 8; nb++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) s[nb][e] = fmaf(s[nb][e], scale2, -bt[8 * (e >> 1) - 8 * nb - (e & 1)]);
+        if (!inside) {
+#pragma unroll
+            for (int nb = 0; nb < kK / 8; nb++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) {
+                    const int key = key0 + nb * 8 + 2 * c + (e & 1);
+                    if (key > pq[e >> 1] || key <= pq[e >> 1] - a.window) s[nb][e] = -INFINITY;
+                }
+        }
         float tmax[2] = {-INFINITY, -INFINITY};
-        const float *bt = s_bias + (t & 1) * 128 + warp * 16 + g + (kK - 1);       // minus the key's place in the tile, plus 8 for row 1
 #pragma unroll
         for (int nb = 0; nb < kK / 8; nb++) {
-#pragma unroll
-            for (int e = 0; e < 4; e++) {
-                const int kl = nb * 8 + 2 * c + (e & 1), key = key0 + kl, r = e >> 1;
-                float v = s[nb][e] * scale2;
-                if (a.bias) v -= bt[8 * r - kl];
-                if (!inside && (key > pq[r] || key <= pq[r] - a.window)) v = -INFINITY;
-                s[nb][e] = v;
-                tmax[r] = fmaxf(tmax[r], v);
-            }
+            tmax[0] = fmaxf(tmax[0], fmaxf(s[nb][0], s[nb][1]));
+            tmax[1] = fmaxf(tmax[1], fmaxf(s[nb][2], s[nb][3]));
         }
         float corr[2], mref[2];
 #pragma unroll
@@ -162,22 +169,8 @@ mix_attn_tc_kernel(const MixAttn a, int seq, int T, int pos0, __nv_bfloat16 *__r
             corr[r] = exp2_approx(mrow[r] - mref[r]);
             mrow[r] = mn;
         }
-        float tsum[2] = {0.f, 0.f};
-        uint32_t ph[kK / 16][4], pl[kK / 16][4];
-#pragma unroll
-        for (int nb = 0; nb < kK / 8; nb++) {
-#pragma unroll
-            for (int r = 0; r < 2; r++) {
-                const float e0 = exp2_approx(s[nb][2 * r] - mref[r]), e1 = exp2_approx(s[nb][2 * r + 1] - mref[r]);
-                tsum[r] += e0 + e1;
-                const uint32_t hi = pack_h2(e0, e1);
-                ph[nb >> 1][(nb & 1) * 2 + r] = hi;
-                pl[nb >> 1][(nb & 1) * 2 + r] = rest_h2(e0, e1, hi);
-            }
-        }
-#pragma unroll
-        for (int r = 0; r < 2; r++) lrow[r] = lrow[r] * corr[r] + tsum[r];
         if (__any_sync(0xffffffffu, corr[0] != 1.f || corr[1] != 1.f)) {
+            lrow[0] *= corr[0]; lrow[1] *= corr[1];
 #pragma unroll
             for (int nb = 0; nb < P / 8; nb++) {
                 o[nb][0] *= corr[0]; o[nb][1] *= corr[0];
@@ -186,14 +179,27 @@ mix_attn_tc_kernel(const MixAttn a, int seq, int T, int pos0, __nv_bfloat16 *__r
         }
 #pragma unroll
         for (int ks = 0; ks < kK / 16; ks++) {
+            // weights of 16 keys, as values and remainders
+            uint32_t ph[4], pl[4];
 #pragma unroll
-            for (int nb = 0; nb < P / 8; nb += 2) {
-                uint32_t b0, b1, b2, b3;
-                ldmatrix_x4_trans(smem_u32(Vs + (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * RS + nb * 8 + (lane >> 4) * 8), b0, b1, b2, b3);
-                hmma16816(o[nb], ph[ks][0], ph[ks][1], ph[ks][2], ph[ks][3], b0, b1);
-                hmma16816(o[nb + 1], ph[ks][0], ph[ks][1], ph[ks][2], ph[ks][3], b2, b3);
-                hmma16816(o[nb], pl[ks][0], pl[ks][1], pl[ks][2], pl[ks][3], b0, b1);
-                hmma16816(o[nb + 1], pl[ks][0], pl[ks][1], pl[ks][2], pl[ks][3], b2, b3);
+            for (int i = 0; i < 2; i++)
+#pragma unroll
+                for (int r = 0; r < 2; r++) {
+                    const float e0 = exp2_approx(s[2 * ks + i][2 * r] - mref[r]), e1 = exp2_approx(s[2 * ks + i][2 * r + 1] - mref[r]);
+                    lrow[r] += e0 + e1;
+                    ph[2 * i + r] = pack_h2(e0, e1);
+                    pl[2 * i + r] = rest_h2(e0, e1, ph[2 * i + r]);
+                }
+#pragma unroll
+            for (int nb = 0; nb < P / 8; nb += 4) {
+                uint32_t vb[2][4];
+#pragma unroll
+                for (int i = 0; i < 2; i++)
+                    ldmatrix_x4_trans(smem_u32(Vs + (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * RS + (nb + 2 * i) * 8 + (lane >> 4) * 8), vb[i][0], vb[i][1], vb[i][2], vb[i][3]);
+#pragma unroll
+                for (int i = 0; i < 4; i++) hmma16816(o[nb + i], ph[0], ph[1], ph[2], ph[3], vb[i >> 1][2 * (i & 1)], vb[i >> 1][2 * (i & 1) + 1]);
+#pragma unroll
+                for (int i = 0; i < 4; i++) hmma16816(o[nb + i], pl[0], pl[1], pl[2], pl[3], vb[i >> 1][2 * (i & 1)], vb[i >> 1][2 * (i & 1) + 1]);
             }
         }
         __syncthreads();

@@ -16,7 +16,7 @@ namespace tlb {
 
 namespace {
 
-constexpr int kScanThreads = 128, kScanTok = 16;
+constexpr int kScanThreads = 256, kScanTok = 16;      // consuming threads (a warp more fetches), tokens per chunk
 constexpr int kStepThreads = 512, kStepCols = kStepThreads / 8;
 constexpr float kUnitEps = 1e-6f;             // inside the root of the unit key
 
@@ -29,6 +29,12 @@ __device__ __forceinline__ f2 add2(f2 a, f2 b) { f2 d; asm("add.rn.f32x2 %0, %1,
 
 __device__ __forceinline__ void store_act(float *p, float v) { *p = v; }
 __device__ __forceinline__ void store_act(__nv_bfloat16 *p, float v) { *p = __float2bfloat16_rn(v); }
+__device__ __forceinline__ void store_act4(float *p, float a, float b, float c, float d) { *reinterpret_cast<float4 *>(p) = make_float4(a, b, c, d); }
+__device__ __forceinline__ void store_act4(__nv_bfloat16 *p, float a, float b, float c, float d)
+{
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(a, b), hi = __floats2bfloat162_rn(c, d);
+    *reinterpret_cast<uint2 *>(p) = make_uint2(*reinterpret_cast<const uint32_t *>(&lo), *reinterpret_cast<const uint32_t *>(&hi));
+}
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float lanes8_sum(float v)
 {
@@ -130,7 +136,7 @@ struct Column {
 //   k'^T S_t = (k' w)^T S_(t-1) - (k' . rem) (k^T S_(t-1)) + (k' . k) v,
 // so its reduction over the lanes overlaps this token's update instead of standing in front of the next one.
 template <int NC> struct ScanShape {
-    static constexpr int DP = 32 * NC, L = NC % 2 ? 8 : 16, N4 = DP / (4 * L), CB = N4 <= 4 ? 4 : 2, TB = L / CB;
+    static constexpr int DP = 32 * NC, L = NC % 4 == 0 ? 32 : NC % 2 ? 8 : 16, N4 = DP / (4 * L), CB = N4 <= 4 ? 4 : 2, TB = L / CB;
     static constexpr int COLS = kScanThreads / L * CB;       // columns per CTA
 };
 
@@ -138,7 +144,9 @@ struct ScanParams {
     int H, D, DV, T;
     const float *q, *k, *v, *w, *rem;         // row 0, head 0 of each; rows `ld*` apart, heads D (v: DV) apart
     int ldq, ldk, ldv, ldw, ldr;
-    const float2 *look;                       // general delta: [T][H] (k' . rem, k' . k) of the next token's key
+    const float2 *look;                       // general delta: [H][look_ld] (k' . rem, k' . k) of the next token's key
+    int look_ld;                              // >= T rounded up to a chunk
+    int *err;
     const float *decay;
     float *state;                             // [H][DV][32 NC]
     int from_zero;
@@ -149,15 +157,6 @@ __device__ __forceinline__ void cp_async4(void *dst, const void *src)
 {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
-__device__ __forceinline__ void cp_async8(void *dst, const void *src)
-{
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 8;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void cp_async16(void *dst, const void *src)
-{
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-}
-
 // N values per lane (N a power of two): afterwards lane l of every N consecutive lanes holds the sum over those N lanes of value
 // l, with N - 1 shuffles.
 template <int N>
@@ -185,44 +184,77 @@ __device__ __forceinline__ void all_sum(float (&y)[N], int lane)
 }
 
 template <int NC, bool DELTA>
-__global__ void __launch_bounds__(kScanThreads) scan_kernel(const ScanParams p)
+__global__ void __launch_bounds__(kScanThreads + 32) scan_kernel(const ScanParams p)
 {
     using S = ScanShape<NC>;
     constexpr int DP = S::DP, L = S::L, N4 = S::N4, CB = S::CB, TB = S::TB, COLS = S::COLS, NP = 2 * N4;
-    constexpr int NV = DELTA ? 4 : 2, ROW = NV * DP + COLS + 4, BUF = kScanTok * ROW + DP;     // k has one row more than the chunk
-    extern __shared__ __align__(16) float scan_smem[];       // [2][BUF]; a row: q, k, (w, rem), value channels, look-ahead products
-    const int tid = threadIdx.x, lane = tid & 31, l = lane % L, h = blockIdx.y, c0 = blockIdx.x * COLS, col = tid / L * CB;
-    for (int i = tid; i < 2 * BUF; i += kScanThreads) scan_smem[i] = 0.f;
+    constexpr int NV = DELTA ? 4 : 2, ROW = NV * DP + COLS, BUF = kScanTok * ROW + DP + 2 * kScanTok;     // k has one row more than the chunk
+    extern __shared__ __align__(16) float scan_smem[];       // [2][BUF]: rows of q, k, (w, rem), value channels; one more key; look-ahead products
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, l = lane % L, h = blockIdx.y, c0 = blockIdx.x * COLS, col = tid / L * CB;
+    __shared__ __align__(8) unsigned long long full_bar[2];
+    __shared__ int abort_word;
+    volatile int *abort_flag = &abort_word;
+    for (int i = tid; i < 2 * BUF; i += kScanThreads + 32) scan_smem[i] = 0.f;
+    if (tid == 0) {
+        abort_word = 0;
+        mbar_init(smem_u32(full_bar), 1);
+        mbar_init(smem_u32(full_bar + 1), 1);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    asm volatile("fence.proxy.async.shared::cta;" ::: "memory");     // the zeros above before bulk copies into the same rows
     __syncthreads();
     const float *src[4] = {p.q + (size_t)h * p.D, p.k + (size_t)h * p.D, DELTA ? p.w + (size_t)h * p.D : nullptr, DELTA ? p.rem + (size_t)h * p.D : nullptr};
     const int lds[4] = {p.ldq, p.ldk, p.ldw, p.ldr};
-    bool wide = p.D % 4 == 0;
+    const int nv = min(COLS, p.DV - c0);
+    const float *vsrc = p.v + (size_t)h * p.DV + c0;
+    // rows that start and end on 16 bytes come as bulk copies, others element by element
+    bool wide = p.D % 4 == 0 && nv % 4 == 0 && p.ldv % 4 == 0 && (reinterpret_cast<uintptr_t>(vsrc) & 15) == 0;
 #pragma unroll
     for (int i = 0; i < NV; i++) wide = wide && lds[i] % 4 == 0 && (reinterpret_cast<uintptr_t>(src[i]) & 15) == 0;
-    const int nv = min(COLS, p.DV - c0);
-    auto fetch = [&](int t0, float *buf) {
-        const int nt = min(kScanTok, p.T - t0);
-#pragma unroll
-        for (int i = 0; i < NV; i++) {
-            const int rows = DELTA && i == 1 ? min(kScanTok + 1, p.T - t0) : nt;      // the key behind the chunk comes too
-            const int step = wide ? 4 : 1, per = p.D / step;
-            for (int e = tid; e < rows * per; e += kScanThreads) {
-                const int t = e / per, d = (e - t * per) * step;
-                float *dst = buf + t * ROW + i * DP + d;
-                if (i == 1 && t == kScanTok) dst = buf + kScanTok * ROW + d;
-                const float *s = src[i] + (size_t)(t0 + t) * lds[i] + d;
-                if (wide) cp_async16(dst, s);
-                else cp_async4(dst, s);
+    if (warp == kScanThreads / 32) {
+        // ------------------------------------------------ the fetching warp: a chunk ahead of the others
+        auto fetch = [&](int t0, int b) {
+            float *buf = scan_smem + b * BUF;
+            const int nt = min(kScanTok, p.T - t0), nk = DELTA ? min(kScanTok + 1, p.T - t0) : nt;     // the key behind the chunk comes too
+            const uint32_t bar = smem_u32(full_bar + b);
+            const float2 *look = DELTA ? p.look + (size_t)h * p.look_ld + t0 : nullptr;
+            if (wide) {
+                if (lane == 0) mbar_expect_tx(bar, (uint32_t)(((NV - 1) * nt + nk) * p.D * 4 + nt * nv * 4 + (DELTA ? kScanTok * 8 : 0)));
+                __syncwarp();
+                for (int i = lane; i < NV * kScanTok + 1; i += 32) {
+                    const bool extra = i == NV * kScanTok;
+                    const int j = extra ? 1 : i / kScanTok, t = extra ? kScanTok : i % kScanTok;
+                    if (t >= (j == 1 ? nk : nt)) continue;
+                    const float *s = j == 0 ? src[0] : (j == 1 ? src[1] : (j == 2 ? src[2] : src[3]));
+                    const int ld = j == 0 ? lds[0] : (j == 1 ? lds[1] : (j == 2 ? lds[2] : lds[3]));
+                    bulk_g2s(smem_u32(extra ? buf + kScanTok * ROW : buf + t * ROW + j * DP), s + (size_t)(t0 + t) * ld, (uint32_t)p.D * 4, bar);
+                }
+                if (lane < nt) bulk_g2s(smem_u32(buf + lane * ROW + NV * DP), vsrc + (size_t)(t0 + lane) * p.ldv, (uint32_t)nv * 4, bar);
+                if (DELTA && lane == 0) bulk_g2s(smem_u32(buf + kScanTok * ROW + DP), look, kScanTok * 8, bar);
+            } else {
+                for (int i = 0; i < NV; i++)
+                    for (int t = 0; t < (i == 1 ? nk : nt); t++) {
+                        float *dst = t == kScanTok ? buf + kScanTok * ROW : buf + t * ROW + i * DP;
+                        for (int d = lane; d < p.D; d += 32) cp_async4(dst + d, src[i] + (size_t)(t0 + t) * lds[i] + d);
+                    }
+                for (int t = 0; t < nt; t++)
+                    for (int d = lane; d < nv; d += 32) cp_async4(buf + t * ROW + NV * DP + d, vsrc + (size_t)(t0 + t) * p.ldv + d);
+                if (DELTA && lane < 2 * kScanTok) cp_async4(buf + kScanTok * ROW + DP + lane, reinterpret_cast<const float *>(look) + lane);
+                asm volatile("cp.async.wait_all;" ::: "memory");
+                __syncwarp();
+                if (lane == 0) mbar_arrive(bar);
             }
+        };
+        fetch(0, 0);
+        for (int t0 = 0, c = 0; t0 < p.T; t0 += kScanTok, c++) {
+            // buffer (c + 1) & 1 was left by the barrier that ended chunk c - 1
+            if (t0 + kScanTok < p.T) fetch(t0 + kScanTok, (c + 1) & 1);
+            __syncthreads();
         }
-        for (int e = tid; e < nt * nv; e += kScanThreads) {
-            const int t = e / nv, d = e - t * nv;
-            cp_async4(buf + t * ROW + NV * DP + d, p.v + (size_t)(t0 + t) * p.ldv + (size_t)h * p.DV + c0 + d);
-        }
-        if (DELTA)
-            for (int t = tid; t < nt; t += kScanThreads) cp_async8(buf + t * ROW + NV * DP + COLS, p.look + (size_t)(t0 + t) * p.H + h);
-        asm volatile("cp.async.commit_group;" ::: "memory");
-    };
+        // nothing is in flight any more unless a consumer gave up: its copies land before the block ends
+        if (*abort_flag) { mbar_wait_drain(smem_u32(full_bar), 0); mbar_wait_drain(smem_u32(full_bar + 1), 0); }
+        return;
+    }
     auto vec = [&](const float *row, f2 (&x)[NP]) {
 #pragma unroll
         for (int i = 0; i < N4; i++) lds_f2x2(row + 4 * (i * L + l), x[2 * i], x[2 * i + 1]);
@@ -251,13 +283,18 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const ScanParams p)
     f2 kc[NP];                    // general delta: this token's key, and k^T S of it per column
     float ks[CB];
     // one token: the state moves on, y = this lane's share of the outputs
-    auto token = [&](const float *r, const float *knext, float *y) {
+    auto token = [&](const float *r, const float *knext, const float2 *look, float *y) {
         float v[CB];
+        if constexpr (CB == 4) {
+            const float4 x = *reinterpret_cast<const float4 *>(r + NV * DP + col);
+            v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
+        } else {
 #pragma unroll
-        for (int c = 0; c < CB; c++) v[c] = r[NV * DP + col + c];
+            for (int c = 0; c < CB; c++) v[c] = r[NV * DP + col + c];
+        }
         f2 q[NP];
         if (DELTA) {
-            const float2 lk = *reinterpret_cast<const float2 *>(r + NV * DP + COLS);
+            const float2 lk = *look;
             f2 kn[NP], w[NP], x[NP];
             vec(knext, kn);
             vec(r + 2 * DP, w);
@@ -292,13 +329,9 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const ScanParams p)
             }
         }
     };
-    fetch(0, scan_smem);
-    for (int t0 = 0, b = 0; t0 < p.T; t0 += kScanTok, b ^= 1) {
-        if (t0 + kScanTok < p.T) fetch(t0 + kScanTok, scan_smem + (b ^ 1) * BUF);
-        else asm volatile("cp.async.commit_group;" ::: "memory");
-        asm volatile("cp.async.wait_group 1;" ::: "memory");
-        __syncthreads();
-        const float *buf = scan_smem + b * BUF;
+    for (int t0 = 0, ch = 0; t0 < p.T; t0 += kScanTok, ch++) {
+        const float *buf = scan_smem + (ch & 1) * BUF;
+        mbar_wait(smem_u32(full_bar + (ch & 1)), (uint32_t)(ch >> 1) & 1u, abort_flag, p.err, 71);
         const int nt = min(kScanTok, p.T - t0);
         if (DELTA && t0 == 0) {
             vec(buf + DP, kc);
@@ -307,18 +340,19 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const ScanParams p)
             all_sum<CB, L>(ks, lane);
         }
         auto next_key = [&](int t) { return t + 1 < kScanTok ? buf + (t + 1) * ROW + DP : buf + kScanTok * ROW; };   // past the last token: anything, unused
+        const float2 *look = reinterpret_cast<const float2 *>(buf + kScanTok * ROW + DP);
         int t = 0;
         for (; t + TB <= nt; t += TB) {
             float y[TB * CB];
 #pragma unroll
-            for (int i = 0; i < TB; i++) token(buf + (t + i) * ROW, next_key(t + i), y + i * CB);
+            for (int i = 0; i < TB; i++) token(buf + (t + i) * ROW, next_key(t + i), look + t + i, y + i * CB);
             const float sum = scatter_sum<TB * CB>(y, l);
             const int yt = l / CB, yc = l % CB;
             if (c0 + col + yc < p.DV) o[(size_t)(t0 + t + yt) * ldo + yc] = sum;
         }
         for (; t < nt; t++) {
             float y[CB];
-            token(buf + t * ROW, next_key(t), y);
+            token(buf + t * ROW, next_key(t), look + t, y);
             all_sum<CB, L>(y, lane);
 #pragma unroll
             for (int c = 0; c < CB; c++)
@@ -362,7 +396,7 @@ __global__ void retention_prep_kernel(const MixRecur m, int rope0, int rope_step
 
 // one warp per (token, head): decay <- exp(-exp(-1/2) sigmoid(decay + w0)), a <- sigmoid(a) k / (k . k + eps), and the two products
 // with the next token's key that the scan looks ahead with.  The bias of a is in already.
-__global__ void __launch_bounds__(256) delta_prep_kernel(const MixRecur m, int T, float *__restrict__ decay, float2 *__restrict__ look)
+__global__ void __launch_bounds__(256) delta_prep_kernel(const MixRecur m, int T, float *__restrict__ decay, float2 *__restrict__ look, int look_ld)
 {
     const int lane = threadIdx.x & 31;
     const int64_t u = (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5);
@@ -378,16 +412,30 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const MixRecur m, int T
     const float rate = expf(-0.5f);
     const float *kn = t + 1 < T ? k + m.ldp : k;
     float kr = 0.f, kk = 0.f;
-    for (int d = lane; d < m.D; d += 32) {
-        dc[d] = expf(-rate * sigmoid_f(dc[d] + w0[d]));
-        const float rem = sigmoid_f(a[d]) * k[d] * ss;
-        a[d] = rem;
-        kr += kn[d] * rem;
-        kk += kn[d] * k[d];
+    auto one = [&](float &dv, float &av, float kv, float nv, float wv) {
+        dv = expf(-rate * sigmoid_f(dv + wv));
+        av = sigmoid_f(av) * kv * ss;
+        kr += nv * av;
+        kk += nv * kv;
+    };
+    if (m.D % 4 == 0) {           // rows and heads then start on 16 bytes
+        for (int d = lane * 4; d < m.D; d += 128) {
+            float4 dv = *reinterpret_cast<float4 *>(dc + d), av = *reinterpret_cast<float4 *>(a + d);
+            const float4 kv = *reinterpret_cast<const float4 *>(k + d), nv = *reinterpret_cast<const float4 *>(kn + d), wv = *reinterpret_cast<const float4 *>(w0 + d);
+            one(dv.x, av.x, kv.x, nv.x, wv.x); one(dv.y, av.y, kv.y, nv.y, wv.y); one(dv.z, av.z, kv.z, nv.z, wv.z); one(dv.w, av.w, kv.w, nv.w, wv.w);
+            *reinterpret_cast<float4 *>(dc + d) = dv;
+            *reinterpret_cast<float4 *>(a + d) = av;
+        }
+    } else {
+        for (int d = lane; d < m.D; d += 32) {
+            float dv = dc[d], av = a[d];
+            one(dv, av, k[d], kn[d], w0[d]);
+            dc[d] = dv; a[d] = av;
+        }
     }
     kr = warp_sum(kr);
     kk = warp_sum(kk);
-    if (lane == 0) look[u] = make_float2(kr, kk);
+    if (lane == 0) look[(size_t)h * look_ld + t] = make_float2(kr, kk);
 }
 
 __device__ __forceinline__ float gate_value(bool delta, float y, float g, float nw) { return delta ? y * nw * sigmoid_f(g) : y * (g * sigmoid_f(g)); }
@@ -402,6 +450,28 @@ __global__ void __launch_bounds__(256) recur_post_kernel(const MixRecur m, int T
     const int t = (int)(u / m.H), h = (int)(u % m.H);
     const float *y = o + ((size_t)t * m.H + h) * m.DV, *g = m.proj + (size_t)t * m.ldp + g_col + (size_t)h * m.DV;
     float ss = 0.f;
+    if (m.DV % 4 == 0 && m.DV <= 256 && g_col % 4 == 0 && ldo % 4 == 0) {
+        float4 v[2], gv[2];
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+            const int d = lane * 4 + i * 128;
+            v[i] = gv[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (d < m.DV) { v[i] = *reinterpret_cast<const float4 *>(y + d); gv[i] = *reinterpret_cast<const float4 *>(g + d); }
+            ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+        }
+        const float inv = 1.f / sqrtf(warp_sum(ss) / (float)m.DV + m.eps);
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+            const int d = lane * 4 + i * 128;
+            if (d >= m.DV) continue;
+            float4 nw = make_float4(1.f, 1.f, 1.f, 1.f);
+            const bool delta = m.norm_w != nullptr;
+            if (delta) nw = *reinterpret_cast<const float4 *>(m.norm_w + h * m.DV + d);
+            store_act4(out + (size_t)t * ldo + (size_t)h * m.DV + d, gate_value(delta, v[i].x * inv, gv[i].x, nw.x), gate_value(delta, v[i].y * inv, gv[i].y, nw.y),
+                       gate_value(delta, v[i].z * inv, gv[i].z, nw.z), gate_value(delta, v[i].w * inv, gv[i].w, nw.w));
+        }
+        return;
+    }
     for (int d = lane; d < m.DV; d += 32) ss += y[d] * y[d];
     const float inv = 1.f / sqrtf(warp_sum(ss) / (float)m.DV + m.eps);
     for (int d = lane; d < m.DV; d += 32)
@@ -445,6 +515,10 @@ __global__ void __launch_bounds__(kStepThreads) recur_step_kernel(const MixRecur
     int col = tid >> 3;
     if (pos > 0 && col < m.DV) S.load(state + (size_t)col * DP, l);
     else S.zero();
+    if (DELTA) {                                             // weights: on their way while the launch in front finishes
+        const char *w2 = reinterpret_cast<const char *>(m.w2.w + (size_t)h * m.D * m.w2.ld);
+        for (size_t i = (size_t)tid * 128; i < (size_t)m.D * m.w2.ld * 2; i += kStepThreads * 128) asm volatile("prefetch.global.L2 [%0];" ::"l"(w2 + i));
+    }
     pdl_wait();
     pdl_launch_dependents();
     const int HD = m.H * m.D;
@@ -471,12 +545,21 @@ __global__ void __launch_bounds__(kStepThreads) recur_step_kernel(const MixRecur
         for (int i = 0; i < kStepThreads / 32; i++) ss += red[i];
         const float inv = 1.f / (ss + kUnitEps), rate = expf(-0.5f);
         for (int d = tid; d < m.D; d += kStepThreads) s_rem[d] *= inv;
-        for (int d = warp; d < m.D; d += kStepThreads / 32) {
-            const __nv_bfloat16 *wr = m.w2.w + (size_t)(h * m.D + d) * m.w2.ld;
-            float s = 0.f;
-            for (int i = lane; i < m.rank; i += 32) s = fmaf(__bfloat162float(wr[i]), s_t[i], s);
-            s = warp_sum(s);
-            if (lane == 0) s_w[d] = expf(-rate * sigmoid_f(s + m.w0[h * m.D + d]));
+        constexpr int NR = 8;                                // rows in flight per warp
+        for (int d0 = warp * NR; d0 < m.D; d0 += kStepThreads / 32 * NR) {
+            float s[NR] = {};
+            for (int i = lane; i < m.rank; i += 32) {
+                const __nv_bfloat16 *wr = m.w2.w + (size_t)(h * m.D + d0) * m.w2.ld + i;
+                float w[NR];
+#pragma unroll
+                for (int r = 0; r < NR; r++) w[r] = __bfloat162float(wr[(size_t)min(r, m.D - 1 - d0) * m.w2.ld]);
+#pragma unroll
+                for (int r = 0; r < NR; r++) s[r] = fmaf(w[r], s_t[i], s[r]);
+            }
+            float mine = scatter_sum<NR>(s, lane);           // lane r of every eight: row d0 + r over those eight lanes
+            mine += __shfl_xor_sync(0xffffffffu, mine, 8);
+            mine += __shfl_xor_sync(0xffffffffu, mine, 16);
+            if (lane < NR && d0 + lane < m.D) s_w[d0 + lane] = expf(-rate * sigmoid_f(mine + m.w0[h * m.D + d0 + lane]));
         }
     } else {
         const int half = m.rot / 2;
@@ -531,14 +614,14 @@ __global__ void __launch_bounds__(kStepThreads) recur_step_kernel(const MixRecur
 template <int NC, bool DELTA>
 tlb_status scan_nc(const ScanParams &p)
 {
-    constexpr int COLS = ScanShape<NC>::COLS, ROW = (DELTA ? 4 : 2) * 32 * NC + COLS + 4;
-    const size_t smem = (size_t)2 * (kScanTok * ROW + 32 * NC) * sizeof(float);
+    constexpr int COLS = ScanShape<NC>::COLS, ROW = (DELTA ? 4 : 2) * 32 * NC + COLS;
+    const size_t smem = (size_t)2 * (kScanTok * ROW + 32 * NC + 2 * kScanTok) * sizeof(float);
     static bool set = false;
     if (!set) {
         TLB_CUDA(cudaFuncSetAttribute(scan_kernel<NC, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         set = true;
     }
-    scan_kernel<NC, DELTA><<<dim3((p.DV + COLS - 1) / COLS, p.H), kScanThreads, smem, ctx()->stream>>>(p);
+    scan_kernel<NC, DELTA><<<dim3((p.DV + COLS - 1) / COLS, p.H), kScanThreads + 32, smem, ctx()->stream>>>(p);
     TLB_CUDA(cudaGetLastError());
     count_launch();
     return TLB_OK;
@@ -600,6 +683,7 @@ tlb_status post(const MixRecur &m, int T, const float *o, int g_col, void *out, 
 
 }  // namespace
 
+int scan_look_ld(int T) { return (T + kScanTok - 1) / kScanTok * kScanTok; }
 bool mix_recur_supported(int D, int DV) { return D >= 1 && D <= 256 && DV >= 1 && DV <= 4096; }
 int mix_recur_ld(int D) { return (D + 31) / 32 * 32; }
 
@@ -620,6 +704,7 @@ tlb_status launch_retention_prefill(const MixRecur &m, int seq, int T, int pos0,
     p.state = m.state + (size_t)seq * m.seq_stride;
     p.from_zero = pos0 == 0;
     p.o = o;
+    p.err = ctx()->err_flag;
     TLB_TRY(run_scan<false>(p, m.ld / 32));
     return post(m, T, o, 2 * HD + m.H * m.DV, out, ldo, f32);
 }
@@ -627,7 +712,7 @@ tlb_status launch_retention_prefill(const MixRecur &m, int seq, int T, int pos0,
 tlb_status launch_delta_prefill(const MixRecur &m, int seq, int T, int pos0, float *decay, float2 *look, float *o, void *out, int ldo, bool f32)
 {
     const int HD = m.H * m.D;
-    delta_prep_kernel<<<(unsigned)(((int64_t)T * m.H + 7) / 8), 256, 0, ctx()->stream>>>(m, T, decay, look);
+    delta_prep_kernel<<<(unsigned)(((int64_t)T * m.H + 7) / 8), 256, 0, ctx()->stream>>>(m, T, decay, look, scan_look_ld(T));
     TLB_CUDA(cudaGetLastError());
     count_launch();
     ScanParams p = {};
@@ -635,10 +720,11 @@ tlb_status launch_delta_prefill(const MixRecur &m, int seq, int T, int pos0, flo
     p.q = m.proj; p.k = m.proj + HD; p.v = m.proj + 2 * HD; p.w = decay; p.rem = m.proj + 4 * (size_t)HD;
     p.ldq = p.ldk = p.ldv = p.ldr = m.ldp;
     p.ldw = HD;
-    p.look = look;
+    p.look = look; p.look_ld = scan_look_ld(T);
     p.state = m.state + (size_t)seq * m.seq_stride;
     p.from_zero = pos0 == 0;
     p.o = o;
+    p.err = ctx()->err_flag;
     TLB_TRY(run_scan<true>(p, m.ld / 32));
     return post(m, T, o, 3 * HD, out, ldo, f32);
 }

@@ -14,10 +14,15 @@
 //               transposed f16 copy of the rows in use is made per launch so that the operand is K-major), O [128 x 128] f32
 //               in tensor memory.
 // Warp roles: 0-3 softmax / write-out, 4 TMA (lane 0), 5 MMA issue (lane 0) and tensor-memory allocation.
+// The MIX form serves the attention of layered models (launch_mix_attn_prefill_tc5): a sliding window (only tiles with a visible
+// key are visited), a bias by distance taken off the scores (consecutive table entries per tile, staged in shared memory), a sink in
+// the denominator, head sizes up to 128 (zero-filled to 128 by TMA), and weights kept in 32 bits: P goes into tensor memory as
+// two f16 terms, value and remainder, and P V is the sum of both products.
 // Every mbarrier wait is bounded (qmv_common.cuh: mbar_wait): when one runs out the CTA sets the context's error word,
 // lets its copies land, frees its tensor memory and returns.
 #include <algorithm>
 
+#include "layered_kernels.h"
 #include "tc05.cuh"
 
 namespace tlb {
@@ -29,14 +34,19 @@ constexpr int kAtThreads = 192;
 constexpr int kBoxBytes = 128 * 128;            // one TMA box: 128 rows x 64 f16
 constexpr int kTileBytes = 2 * kBoxBytes;       // a 128 x 128 f16 operand = two boxes
 // tensor memory columns
-constexpr uint32_t kColS = 0, kColO = 256, kColP = 384;
+constexpr uint32_t kColS = 0, kColO = 256, kColP = 384, kColPRest = 448;
 
 struct AtParams {
     float *out;            // [T, H * 128]
     int T, H, KVH, max_seq, pos0, vt_rows;
     float scale2;          // attn_scale * log2(e)
     int *err;
+    // MIX
+    int DV, ldo, window, bias_n, vt_first;    // vt_first: the key V^T's column 0 holds
+    const float *bias, *sink;
+    __nv_bfloat16 *out16;  // [T, ldo], head h at column h * DV
 };
+constexpr float kLog2eAt = 1.4426950408889634f;
 
 __device__ __forceinline__ float ex2f(float x)
 {
@@ -50,6 +60,7 @@ __device__ __forceinline__ uint32_t pack_h2(float a, float b)
     return *reinterpret_cast<uint32_t *>(&h);
 }
 
+template <bool MIX>
 __global__ void __launch_bounds__(kAtThreads, 1)
 prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_constant__ CUtensorMap kmap,
                             const __grid_constant__ CUtensorMap vtmap, const AtParams p)
@@ -68,7 +79,9 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __gr
     const int qtile = (int)(gridDim.x - 1 - blockIdx.x);          // late query tiles see the most cache rows: they start first
     const int q0 = qtile * kAtQ;
     const int last_q = min(q0 + kAtQ, p.T) - 1;
-    const int n_tiles = (p.pos0 + last_q) / kAtK + 1;             // tiles that hold a key <= the CTA's last query
+    const int tile0 = MIX ? max(0, p.pos0 + q0 - p.window + 1) / kAtK : 0;    // the first tile some query of the CTA sees
+    const int n_tiles = (p.pos0 + last_q) / kAtK + 1 - tile0;     // up to the tile that holds the CTA's last query
+    __shared__ float s_bias[MIX ? 4 : 1][MIX ? 160 : 1];           // per softmax warp: what its 32 queries x 128 keys need
 
     if (tid == 0) {
         abort_word = 0;
@@ -93,9 +106,19 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __gr
         const int row = warp * 32 + lane, q = q0 + row, qpos = p.pos0 + q;
         const uint32_t tl = tmem + ((uint32_t)(warp * 32) << 16);      // this warp's lanes
         float m_run = -INFINITY, l_run = 0.f;
+        if (MIX && p.sink) { m_run = p.sink[h] * kLog2eAt; l_run = 1.f; }
         bool ok = true;
         for (int t = 0; t < n_tiles && ok; t++) {
-            const int b = t & 1, key0 = t * kAtK;
+            const int b = t & 1, key0 = (tile0 + t) * kAtK;
+            if (MIX) {       // entry i: distance (the warp's first query) - (last key of the tile) + i
+                __syncwarp();
+#pragma unroll
+                for (int i = lane; i < 160; i += 32) {
+                    const int dist = p.pos0 + q0 + warp * 32 - (key0 + kAtK - 1) + i;
+                    s_bias[warp][i] = p.bias ? kLog2eAt * p.bias[(size_t)h * p.bias_n + min(max(dist, 0), p.bias_n - 1)] : 0.f;
+                }
+                __syncwarp();
+            }
             if (!mbar_wait(s_full + 8 * b, (uint32_t)(t >> 1) & 1u, abort_flag, p.err, 41)) { ok = false; break; }
             tc_fence_after();
             float s[128];
@@ -104,15 +127,29 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __gr
             tmem_wait_ld();
             const bool diagonal = key0 + kAtK - 1 > p.pos0 + q0;     // some key of the tile is ahead of some query of the CTA
             float m_tile = -INFINITY;
+            if constexpr (MIX) {
+                const float *bt = s_bias[warp] + lane + kAtK - 1;
 #pragma unroll
-            for (int c = 0; c < 128; c++) {
-                const float v = (!diagonal || key0 + c <= qpos) ? s[c] * p.scale2 : -INFINITY;
-                s[c] = v;
-                m_tile = fmaxf(m_tile, v);
+                for (int c = 0; c < 128; c++) s[c] = fmaf(s[c], p.scale2, -bt[-c]);
+                if (diagonal || key0 <= p.pos0 + last_q - p.window) {
+#pragma unroll
+                    for (int c = 0; c < 128; c++)
+                        if (key0 + c > qpos || key0 + c <= qpos - p.window) s[c] = -INFINITY;
+                }
+#pragma unroll
+                for (int c = 0; c < 128; c++) m_tile = fmaxf(m_tile, s[c]);
+            } else {
+#pragma unroll
+                for (int c = 0; c < 128; c++) {
+                    const float v = (!diagonal || key0 + c <= qpos) ? s[c] * p.scale2 : -INFINITY;
+                    s[c] = v;
+                    m_tile = fmaxf(m_tile, v);
+                }
             }
-            const float m_new = fmaxf(m_run, m_tile);                // finite from the first tile on: key 0 is visible to every query
+            float m_new = fmaxf(m_run, m_tile);                      // Llama: finite from the first tile on, key 0 is visible to every query
+            if (MIX && m_new == -INFINITY) m_new = 0.f;              // nothing seen so far: every weight is zero
             const float corr = ex2f(m_run - m_new);
-            m_run = m_new;
+            m_run = MIX ? fmaxf(m_run, m_tile) : m_new;
             if (t > 0) {
                 // the product of tile t - 1 has read P and added to O: O may be rescaled, P overwritten
                 if (!mbar_wait(o_full, (uint32_t)(t - 1) & 1u, abort_flag, p.err, 42)) { ok = false; break; }
@@ -132,14 +169,19 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __gr
             float sum = 0.f;
 #pragma unroll
             for (int c = 0; c < 2; c++) {
-                uint32_t pk[32];
+                uint32_t pk[32], rest[MIX ? 32 : 1];
 #pragma unroll
                 for (int i = 0; i < 32; i++) {
                     const float e0 = ex2f(s[c * 64 + 2 * i] - m_new), e1 = ex2f(s[c * 64 + 2 * i + 1] - m_new);
                     sum += e0 + e1;
                     pk[i] = pack_h2(e0, e1);
+                    if constexpr (MIX) {
+                        const float2 f = h2_to_f2(pk[i]);
+                        rest[i] = pack_h2(e0 - f.x, e1 - f.y);
+                    }
                 }
                 tmem_st32(tl + kColP + (uint32_t)(c * 32), pk);
+                if constexpr (MIX) tmem_st32(tl + kColPRest + (uint32_t)(c * 32), rest);
             }
             l_run = l_run * corr + sum;
             tmem_wait_st();
@@ -157,7 +199,28 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __gr
                 uint32_t o[32];
                 tmem_ld32(tl + kColO + (uint32_t)(c * 32), o);
                 tmem_wait_ld();
-                if (q < p.T) {
+                if constexpr (MIX) {
+                    if (q < p.T) {
+                        __nv_bfloat16 *d16 = p.out16 + (size_t)q * p.ldo + (size_t)h * p.DV + c * 32;
+                        if (p.DV % 8 == 0 && p.ldo % 8 == 0) {
+#pragma unroll
+                            for (int i = 0; i < 32; i += 8) {
+                                if (c * 32 + i >= p.DV) break;
+                                uint32_t w[4];
+#pragma unroll
+                                for (int k = 0; k < 4; k++) {
+                                    const __nv_bfloat162 v2 = __floats2bfloat162_rn(__uint_as_float(o[i + 2 * k]) * inv, __uint_as_float(o[i + 2 * k + 1]) * inv);
+                                    w[k] = *reinterpret_cast<const uint32_t *>(&v2);
+                                }
+                                *reinterpret_cast<uint4 *>(d16 + i) = make_uint4(w[0], w[1], w[2], w[3]);
+                            }
+                        } else {
+#pragma unroll
+                            for (int i = 0; i < 32; i++)
+                                if (c * 32 + i < p.DV) d16[i] = __float2bfloat16_rn(__uint_as_float(o[i]) * inv);
+                        }
+                    }
+                } else if (q < p.T) {
 #pragma unroll
                     for (int i = 0; i < 32; i += 4)
                         *reinterpret_cast<float4 *>(dst + c * 32 + i) = make_float4(__uint_as_float(o[i]) * inv, __uint_as_float(o[i + 1]) * inv,
@@ -176,11 +239,11 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __gr
                 const int st = t & 1;
                 if (t >= 2 && !mbar_wait(kv_empty + 8 * st, (uint32_t)((t - 2) >> 1) & 1u, abort_flag, p.err, 44)) break;
                 mbar_expect_tx(kv_full + 8 * st, 2 * kTileBytes);
-                const int key0 = t * kAtK;
+                const int key0 = (tile0 + t) * kAtK, vt0 = MIX ? p.vt_first : 0;
                 tma_load_2d(sK + st * kTileBytes, &kmap, 0, kvh * p.max_seq + key0, kv_full + 8 * st);
                 tma_load_2d(sK + st * kTileBytes + kBoxBytes, &kmap, 64, kvh * p.max_seq + key0, kv_full + 8 * st);
-                tma_load_2d(sV + st * kTileBytes, &vtmap, key0, kvh * kAtD, kv_full + 8 * st);
-                tma_load_2d(sV + st * kTileBytes + kBoxBytes, &vtmap, key0 + 64, kvh * kAtD, kv_full + 8 * st);
+                tma_load_2d(sV + st * kTileBytes, &vtmap, key0 - vt0, kvh * kAtD, kv_full + 8 * st);
+                tma_load_2d(sV + st * kTileBytes + kBoxBytes, &vtmap, key0 - vt0 + 64, kvh * kAtD, kv_full + 8 * st);
                 issued = t + 1;
             }
             if (*abort_flag) {
@@ -219,6 +282,11 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __gr
 #pragma unroll
                     for (int k16 = 0; k16 < 4; k16++)
                         umma_f16_ts(tmem + kColO, tmem + kColP + (uint32_t)(j * 32 + k16 * 8), bd + 2u * k16, idesc, (t | j | k16) != 0);
+                    if constexpr (MIX) {
+#pragma unroll
+                        for (int k16 = 0; k16 < 4; k16++)
+                            umma_f16_ts(tmem + kColO, tmem + kColPRest + (uint32_t)(j * 32 + k16 * 8), bd + 2u * k16, idesc, 1);
+                    }
                 }
                 umma_commit(o_full);
                 umma_commit(kv_empty + 8 * st);
@@ -264,7 +332,76 @@ __global__ void __launch_bounds__(256) v_transpose_kernel(const __half *__restri
         if (k0 + tx < keys_ld) dst[(size_t)(d0 + j) * keys_ld + k0 + tx] = tile[tx][j];
 }
 
+// queries of the projection rows as f16, every head padded to 128 columns
+__global__ void __launch_bounds__(256) mix_q_to_f16_kernel(const float *__restrict__ proj, int ldp, int H, int D, __half *__restrict__ qh)
+{
+    const float *row = proj + (size_t)blockIdx.x * ldp;
+    for (int i = threadIdx.x; i < H * kAtD / 2; i += blockDim.x) {
+        const int h = i / (kAtD / 2), d = (i % (kAtD / 2)) * 2;
+        const float *q = row + (size_t)h * D + d;
+        const float a = d < D ? q[0] : 0.f, b = d + 1 < D ? q[1] : 0.f;
+        reinterpret_cast<uint32_t *>(qh)[(size_t)blockIdx.x * (H * kAtD / 2) + i] = pack_h2(fminf(fmaxf(a, -65504.f), 65504.f), fminf(fmaxf(b, -65504.f), 65504.f));
+    }
+}
+// cache rows key_first .. of V as V^T [KV head][128][keys_ld] (columns counted from key_first, rows past DV zero)
+__global__ void __launch_bounds__(256) mix_v_transpose_kernel(const __half *__restrict__ vcache, __half *__restrict__ vt, int max_seq, int ldv, int key_first, int n_keys, int keys_ld)
+{
+    __shared__ __half tile[32][34];
+    const __half *src = vcache + (size_t)blockIdx.z * max_seq * ldv;
+    __half *dst = vt + (size_t)blockIdx.z * kAtD * keys_ld;
+    const int tx = threadIdx.x & 31, ty = threadIdx.x >> 5;
+    const int d0 = blockIdx.x * 32, k0 = blockIdx.y * 32;
+    for (int j = ty; j < 32; j += 8)
+        tile[j][tx] = (k0 + j < n_keys && d0 + tx < ldv) ? src[(size_t)(key_first + k0 + j) * ldv + d0 + tx] : __float2half(0.f);
+    __syncthreads();
+    for (int j = ty; j < 32; j += 8)
+        if (k0 + tx < keys_ld) dst[(size_t)(d0 + j) * keys_ld + k0 + tx] = tile[tx][j];
+}
+
 }  // namespace
+
+// Head sizes that fill most of the 128 columns, and enough queries for a tile.
+bool mix_attn_prefill_tc5_supported(int D, int DV, int T) { return std::max(D, DV) > 64 && D <= kAtD && DV <= kAtD && T >= 64; }
+
+// MixAttn over an f16 cache: T tokens of sequence seq whose rows are in the cache already.
+tlb_status launch_mix_attn_prefill_tc5(const MixAttn &a, int seq, int T, int pos0, void *out, int ldo)
+{
+    Context *c = ctx();
+    if (!c) return TLB_ERR_DEVICE;
+    // cache rows some query sees, from a tile border on
+    const int key_first = std::max(0, pos0 - a.window + 1) / kAtK * kAtK, n_keys = pos0 + T - key_first, keys_ld = (n_keys + 127) / 128 * 128;
+    Storage *qh = storage_alloc((size_t)T * a.H * kAtD * sizeof(__half));
+    Storage *vt = storage_alloc((size_t)a.KVH * kAtD * keys_ld * sizeof(__half));
+    if (!qh || !vt) { if (qh) storage_release(qh); if (vt) storage_release(vt); return TLB_ERR_ALLOC; }
+    auto done = [&](tlb_status st) { storage_release(qh); storage_release(vt); return st; };
+    const __half *kc = (const __half *)a.kcache + (size_t)seq * a.seq_stride_k, *vc = (const __half *)a.vcache + (size_t)seq * a.seq_stride_v;
+    mix_q_to_f16_kernel<<<T, 256, 0, c->stream>>>(a.proj, a.ldp, a.H, a.D, (__half *)qh->ptr);
+    mix_v_transpose_kernel<<<dim3(kAtD / 32, (unsigned)(keys_ld / 32), (unsigned)a.KVH), 256, 0, c->stream>>>(vc, (__half *)vt->ptr, a.max_seq, a.ldv, key_first, n_keys, keys_ld);
+    count_launch(2);
+    CUtensorMap qmap, kmap, vtmap;
+    if (!encode_f16_map(&qmap, qh->ptr, (uint64_t)a.H * kAtD, (uint64_t)T, (uint64_t)a.H * kAtD * 2, 64, 128) ||
+        !encode_f16_map(&kmap, kc, (uint64_t)a.ldk, (uint64_t)a.KVH * a.max_seq, (uint64_t)a.ldk * 2, 64, 128) ||
+        !encode_f16_map(&vtmap, vt->ptr, (uint64_t)keys_ld, (uint64_t)a.KVH * kAtD, (uint64_t)keys_ld * 2, 64, 128))
+        return done(fail(TLB_ERR_DEVICE, "prompt attention: cuTensorMapEncodeTiled failed or is not available"));
+    AtParams p = {};
+    p.T = T; p.H = a.H; p.KVH = a.KVH; p.max_seq = a.max_seq; p.pos0 = pos0; p.vt_rows = keys_ld;
+    p.scale2 = a.scale * kLog2eAt;
+    p.err = c->err_flag;
+    p.DV = a.DV; p.ldo = ldo; p.window = a.window; p.bias_n = a.bias_n; p.bias = a.bias; p.sink = a.sink; p.out16 = (__nv_bfloat16 *)out;
+    p.vt_first = key_first;
+    const size_t smem = (size_t)5 * kTileBytes + 1024 + 128;
+    static bool attr_set = false;
+    if (!attr_set) {
+        cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return done(cuda_fail(e, "prompt attention attribute"));
+        attr_set = true;
+    }
+    prefill_attention_tc_kernel<true><<<dim3((unsigned)((T + kAtQ - 1) / kAtQ), (unsigned)a.H), kAtThreads, smem, c->stream>>>(qmap, kmap, vtmap, p);
+    count_launch();
+    cudaError_t e = cudaGetLastError();
+    if (e != cudaSuccess) return done(cuda_fail(e, "prompt attention launch"));
+    return done(TLB_OK);
+}
 
 bool prefill_attention_tc_supported(int D, int kv_f16, int n_tokens) { return D == 128 && kv_f16 && n_tokens >= 64; }
 
@@ -288,19 +425,19 @@ tlb_status launch_prefill_attention_tc(const float *q, const void *kcache, const
         !encode_f16_map(&kmap, kcache, kAtD, (uint64_t)KVH * max_seq, kAtD * 2, 64, 128) ||
         !encode_f16_map(&vtmap, vt->ptr, (uint64_t)keys_ld, (uint64_t)KVH * kAtD, (uint64_t)keys_ld * 2, 64, 128))
         return done(fail(TLB_ERR_DEVICE, "prompt attention: cuTensorMapEncodeTiled failed or is not available"));
-    AtParams p;
+    AtParams p = {};
     p.out = out; p.T = T; p.H = H; p.KVH = KVH; p.max_seq = max_seq; p.pos0 = pos0; p.vt_rows = keys_ld;
     p.scale2 = scale * 1.4426950408889634f;
     p.err = c->err_flag;
     const size_t smem = (size_t)5 * kTileBytes + 1024 + 128;
     static bool attr_set = false;
     if (!attr_set) {
-        cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return done(cuda_fail(e, "prompt attention attribute"));
         attr_set = true;
     }
     dim3 grid((unsigned)((T + kAtQ - 1) / kAtQ), (unsigned)H);
-    prefill_attention_tc_kernel<<<grid, kAtThreads, smem, c->stream>>>(qmap, kmap, vtmap, p);
+    prefill_attention_tc_kernel<false><<<grid, kAtThreads, smem, c->stream>>>(qmap, kmap, vtmap, p);
     count_launch();
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return done(cuda_fail(e, "prompt attention launch"));
