@@ -431,3 +431,52 @@ def test_prefill_logits_of_a_llama_session(orc):
         d2 = tl.Decoder(cfg, w, kv_f16=True, max_seq=64)
         d2.prefill(t[:n])
         assert np.max(np.abs(row - d2.logits())) < 2e-2 * np.max(np.abs(row))
+
+
+def test_command_line_generates_from_a_folder_and_from_gguf(tmp_path, capsys):
+    from tl_b200 import generate
+    m = Model(config(MIXED), seed=15)
+    synth.write_model_dir(tmp_path / "m", m.cfg, m.bits)
+    prompt = toks(45, seed=5)
+    args = ["--model", str(tmp_path / "m"), "--tokens", ",".join(map(str, prompt)), "--f32"]
+    generate.main(args + ["-n", "12"])
+    assert [int(x) for x in capsys.readouterr().out.split(",")] == greedy(m, prompt, 12)[0]
+    generate.main(args + ["-n", "9", "--temp", "0.9", "--top-k", "30", "--seed", "3"])
+    a = capsys.readouterr().out
+    generate.main(args + ["-n", "9", "--temp", "0.9", "--top-k", "30", "--seed", "3"])
+    assert a == capsys.readouterr().out and len(a.split(",")) == 9
+    cfg = dict(n_layers=1, d_model=256, n_heads=4, n_kv_heads=2, head_dim=64, ffn=512, vocab=320)
+    tens = synth.llama_tensors(dict(cfg, eps=1e-5, rope_base=1e4, attn_scale=0.125), 3, synth.Q4_K, synth.Q6_K)
+    meta = {"general.architecture": "llama", "llama.block_count": 1, "llama.embedding_length": 256, "llama.attention.head_count": 4,
+            "llama.attention.head_count_kv": 2, "llama.feed_forward_length": 512}
+    synth.write_gguf(tmp_path / "l.gguf", tens, metadata=meta)
+    generate.main(["--model", str(tmp_path / "l.gguf"), "--tokens", "1,2,3,4,5,6", "-n", "5"])
+    assert len(capsys.readouterr().out.split(",")) == 5
+
+
+def test_trace_replay(tmp_path):
+    """bin/trace_run: the logits of the wanted tokens, whatever the portions, for requests one after the other."""
+    import os
+    import subprocess
+    import sys
+    m = Model(config(MIXED), seed=18)
+    synth.write_model_dir(tmp_path / "m", m.cfg, m.bits)
+    a, b = toks(30, seed=1), toks(9, seed=2)
+    wa, wb = m.ref(a), m.ref(b)
+    steps = [([("a", a[:20], [0, 19])], []), ([("a", a[20:22], [])], []), ([("a", a[22:23], [0])], []), ([("a", a[23:], [6, 2])], ["a"]),
+             ([("b", b[:1], [0])], []), ([("b", b[1:], [7])], ["b"])]
+    want = [wa[[0, 19]], None, wa[[22]], wa[[29, 25]], wb[[0]], wb[[8]]]
+    text = "".join(json.dumps({"step": i, "entries": [{"id": r, "tokens": t, "want": w} for r, t, w in e], "end": end}) + "\n" for i, (e, end) in enumerate(steps))
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    for dtype in ("float32", "bfloat16"):
+        out = tmp_path / dtype
+        out.mkdir()
+        r = subprocess.run([sys.executable, os.path.join(root, "bin", "trace_run"), "--model", str(tmp_path / "m"), "--dtype", dtype, "--out", str(out), "--max-tokens", "30"],
+                           input=text, capture_output=True, text=True, timeout=300)
+        assert r.returncode == 0, r.stderr[-2000:]
+        assert [l for l in r.stdout.splitlines() if l.startswith("done")] == ["done %d" % i for i in range(len(steps))]
+        for i, w in enumerate(want):
+            f = out / ("%d.f32" % i)
+            assert f.exists() == (w is not None)
+            if w is not None:
+                assert err(np.frombuffer(f.read_bytes(), dtype="<f4").reshape(-1, m.cfg["vocab"]), w) < TOL[dtype == "float32"]

@@ -69,10 +69,8 @@ __global__ void __launch_bounds__(kDecThreads) mix_attn_decode_kernel(const MixA
     const float *row = a.proj + (size_t)b * a.ldp;
     CT *kc = reinterpret_cast<CT *>(a.kcache) + (size_t)b * a.seq_stride_k + (size_t)g * a.max_seq * a.ldk;
     CT *vc = reinterpret_cast<CT *>(a.vcache) + (size_t)b * a.seq_stride_v + (size_t)g * a.max_seq * a.ldv;
-    for (int i = tid; i < rep * a.ldk; i += kDecThreads) {
-        const int r = i / a.ldk, d = i - r * a.ldk;
-        sq[i] = d < a.D ? __ldcg(row + (size_t)(h0 + r) * a.D + d) : 0.f;
-    }
+    for (int r = warp; r < rep; r += kDecThreads / 32)
+        for (int d = lane; d < a.ldk; d += 32) sq[r * a.ldk + d] = d < a.D ? __ldcg(row + (size_t)(h0 + r) * a.D + d) : 0.f;
     for (int i = tid; i < rep * kDecKeys; i += kDecThreads) {
         const int r = i / kDecKeys, key = i - r * kDecKeys;
         s_b[i] = a.bias && key < nk ? a.bias[(size_t)(h0 + r) * a.bias_n + (pos - key0 - key)] : 0.f;
@@ -175,23 +173,24 @@ __global__ void __launch_bounds__(kDecThreads) mix_attn_decode_kernel(const MixA
                         *reinterpret_cast<float4 *>(s_red + ((size_t)slice * 4 + r) * a.ldv + vec * VE + e) = make_float4(acc[r][e], acc[r][e + 1], acc[r][e + 2], acc[r][e + 3]);
         }
         __syncthreads();
-        for (int i = tid; i < nr * a.DV; i += kDecThreads) {
-            const int r = i / a.DV, d = i - r * a.DV;
-            float s = 0.f;
+        for (int r = tid >> 6; r < nr; r += kDecThreads / 64) {
+            for (int d = tid & 63; d < a.DV; d += 64) {
+                float s = 0.f;
 #pragma unroll 8
-            for (int k = 0; k < min(ks, nk); k++) s += s_red[((size_t)k * 4 + r) * a.ldv + d];
-            const int rr = r0 + r;
-            if (nsplit == 1) {
-                const float m0 = s_m[rr];
-                float den = s_l[rr], f = 1.f;
-                if (a.sink) {
-                    const float sk = a.sink[h0 + rr], m = fmaxf(m0, sk);
-                    f = expf(m0 - m);
-                    den = den * f + expf(sk - m);
+                for (int k = 0; k < min(ks, nk); k++) s += s_red[((size_t)k * 4 + r) * a.ldv + d];
+                const int rr = r0 + r;
+                if (nsplit == 1) {
+                    const float m0 = s_m[rr];
+                    float den = s_l[rr], f = 1.f;
+                    if (a.sink) {
+                        const float sk = a.sink[h0 + rr], m = fmaxf(m0, sk);
+                        f = expf(m0 - m);
+                        den = den * f + expf(sk - m);
+                    }
+                    store_act(out + (size_t)(h0 + rr) * a.DV + d, s * f / den);
+                } else {
+                    part[(size_t)rr * prow + d] = s;
                 }
-                store_act(out + (size_t)(h0 + rr) * a.DV + d, s * f / den);
-            } else {
-                part[(size_t)rr * prow + d] = s;
             }
         }
         __syncthreads();

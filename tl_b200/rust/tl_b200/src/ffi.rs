@@ -45,6 +45,7 @@ pub struct TlbDecoderCfg {
     pub tp_size: i32,
     pub tp_rank: i32,
     pub batch: i32,
+    pub f32: i32,
 }
 
 #[link(name = "tlb200")]
@@ -120,6 +121,8 @@ extern "C" {
     pub fn tlb_gguf_load_str(out: *mut *mut TlbMap, path: *const TlbString) -> TlbStatus;
     pub fn tlb_map_new(out: *mut *mut TlbMap) -> TlbStatus;
     pub fn tlb_map_add(m: *mut TlbMap, name: *const c_char, type_: c_int, shape: *const i64, rank: c_int, bytes: *const c_void, nbytes: usize) -> TlbStatus;
+    pub fn tlb_model_load(out: *mut *mut TlbMap, dir: *const c_char) -> TlbStatus;
+    pub fn tlb_map_set_config(m: *mut TlbMap, config_json: *const c_char) -> TlbStatus;
     pub fn tlb_map_free(m: *mut TlbMap) -> TlbStatus;
     pub fn tlb_map_count(m: *const TlbMap) -> i64;
     pub fn tlb_map_name(m: *const TlbMap, i: i64) -> *const c_char;
@@ -176,6 +179,8 @@ extern "C" {
     pub fn tlb_decoder_step(d: *mut TlbDecoder, token: i32, pos: i32, rope_pos: i32, next: *mut i32) -> TlbStatus;
     pub fn tlb_decoder_generate(d: *mut TlbDecoder, first_token: i32, start_pos: i32, n: i32, tokens_out: *mut i32) -> TlbStatus;
     pub fn tlb_decoder_prefill(d: *mut TlbDecoder, tokens: *const i32, n: i32, pos0: i32, rope_pos0: i32, rope_step: i32, next: *mut i32) -> TlbStatus;
+    pub fn tlb_decoder_prefill_logits(d: *mut TlbDecoder, seq: i32, tokens: *const i32, n: i32, pos0: i32, want: *const i32, n_want: i32, logits_out: *mut f32) -> TlbStatus;
+    pub fn tlb_decoder_reset_seq(d: *mut TlbDecoder, seq: i32) -> TlbStatus;
     pub fn tlb_decoder_kv_write_seq(d: *mut TlbDecoder, seq: c_int, layer: c_int, pos0: c_int, n: c_int, k: *const f32, v: *const f32) -> TlbStatus;
     pub fn tlb_decoder_prefill_seq(d: *mut TlbDecoder, seq: i32, tokens: *const i32, n: i32, pos0: i32, rope_pos0: i32, rope_step: i32, next: *mut i32) -> TlbStatus;
     pub fn tlb_decoder_step_batch(d: *mut TlbDecoder, tokens: *const i32, pos: *const i32, rope_pos: *const i32, next: *mut i32) -> TlbStatus;
