@@ -26,17 +26,17 @@ __device__ __forceinline__ void store_cache(__half *p, float v) { *p = __float2h
 template <typename CT> struct Vec;
 template <> struct Vec<float> {
     static constexpr int N = 4;
-    static __device__ __forceinline__ void load(const float *p, float (&v)[4])
+    static __device__ __forceinline__ void unpack(const uint4 &a, float (&v)[4])
     {
-        const float4 a = *reinterpret_cast<const float4 *>(p);
-        v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+        v[0] = __uint_as_float(a.x); v[1] = __uint_as_float(a.y); v[2] = __uint_as_float(a.z); v[3] = __uint_as_float(a.w);
     }
+    static __device__ __forceinline__ void load(const float *p, float (&v)[4]) { unpack(*reinterpret_cast<const uint4 *>(p), v); }
 };
 template <> struct Vec<__half> {
     static constexpr int N = 8;
-    static __device__ __forceinline__ void load(const __half *p, float (&v)[8])
+    static __device__ __forceinline__ void load(const __half *p, float (&v)[8]) { unpack(*reinterpret_cast<const uint4 *>(p), v); }
+    static __device__ __forceinline__ void unpack(const uint4 &a, float (&v)[8])
     {
-        const uint4 a = *reinterpret_cast<const uint4 *>(p);
         const uint32_t w[4] = {a.x, a.y, a.z, a.w};
 #pragma unroll
         for (int i = 0; i < 4; i++) {
@@ -60,15 +60,19 @@ __global__ void __launch_bounds__(kDecThreads) mix_attn_decode_kernel(const MixA
     const int sp = blockIdx.x, g = blockIdx.y, b = blockIdx.z;
     const int rep = a.H / a.KVH, h0 = g * rep;
     float *sq = dec_smem, *sp_w = sq + rep * a.ldk, *s_b = sp_w + rep * kDecKeys, *s_m = s_b + rep * kDecKeys, *s_l = s_m + rep, *s_red = s_l + rep + (-2 * rep & 3);        // 16-byte aligned
-    pdl_wait();
-    pdl_launch_dependents();
-    const int pos = j.pos[b];
+    // The position, and every cache row but the new one, were complete before the launch in front of this one started (they are
+    // an earlier step's): they may be touched before the wait.
+    const int pos = __ldcg(j.pos + b);
     const int first = max(0, pos - a.window + 1), n = pos - first + 1, nsplit = (n + kDecKeys - 1) / kDecKeys;
-    if (sp >= nsplit) return;
+    if (sp >= nsplit) { pdl_wait(); pdl_launch_dependents(); return; }
     const int key0 = first + sp * kDecKeys, nk = min(kDecKeys, pos + 1 - key0);
     const float *row = a.proj + (size_t)b * a.ldp;
     CT *kc = reinterpret_cast<CT *>(a.kcache) + (size_t)b * a.seq_stride_k + (size_t)g * a.max_seq * a.ldk;
     CT *vc = reinterpret_cast<CT *>(a.vcache) + (size_t)b * a.seq_stride_v + (size_t)g * a.max_seq * a.ldv;
+    for (int i = tid * 128; i < nk * a.ldk * (int)sizeof(CT); i += kDecThreads * 128) asm volatile("prefetch.global.L2 [%0];" ::"l"((const char *)(kc + (size_t)key0 * a.ldk) + i));
+    for (int i = tid * 128; i < nk * a.ldv * (int)sizeof(CT); i += kDecThreads * 128) asm volatile("prefetch.global.L2 [%0];" ::"l"((const char *)(vc + (size_t)key0 * a.ldv) + i));
+    pdl_wait();
+    pdl_launch_dependents();
     for (int r = warp; r < rep; r += kDecThreads / 32)
         for (int d = lane; d < a.ldk; d += 32) sq[r * a.ldk + d] = d < a.D ? __ldcg(row + (size_t)(h0 + r) * a.D + d) : 0.f;
     for (int i = tid; i < rep * kDecKeys; i += kDecThreads) {
@@ -81,6 +85,14 @@ __global__ void __launch_bounds__(kDecThreads) mix_attn_decode_kernel(const MixA
         for (int d = tid; d < a.DV; d += kDecThreads) store_cache(vc + (size_t)pos * a.ldv + d, __ldcg(vn + d));
     }
     __syncthreads();
+
+    // a thread owns 16 bytes of the V row for every ks-th key: the first few are asked for now, under the scores
+    constexpr int PV = 4;
+    const int nvv = a.ldv / VE, ks = kDecThreads / nvv, vec = tid % nvv, slice = tid / nvv;
+    const CT *vr = vc + (size_t)key0 * a.ldv + vec * VE;
+    uint4 pv[PV];
+#pragma unroll
+    for (int u = 0; u < PV; u++) pv[u] = slice < ks && slice + u * ks < nk ? *reinterpret_cast<const uint4 *>(vr + (size_t)(slice + u * ks) * a.ldv) : make_uint4(0u, 0u, 0u, 0u);
 
     // scores: `lpk` lanes per key
     const int nvk = a.ldk / VE;
@@ -142,8 +154,7 @@ __global__ void __launch_bounds__(kDecThreads) mix_attn_decode_kernel(const MixA
     }
     __syncthreads();
 
-    // weighted sum of V: a thread owns 16 bytes of the row for every ks-th key
-    const int nvv = a.ldv / VE, ks = kDecThreads / nvv, vec = tid % nvv, slice = tid / nvv;
+    // weighted sum of V
     const int prow = a.ldv + 4;                 // weighted sums, maximum, sum of exponentials; whole 16-byte lines
     float *part = j.partial + ((((size_t)b * a.KVH + g) * gridDim.x + sp) * rep) * prow;
     TO *out = reinterpret_cast<TO *>(j.out) + (size_t)b * j.ldo;
@@ -151,11 +162,9 @@ __global__ void __launch_bounds__(kDecThreads) mix_attn_decode_kernel(const MixA
         const int nr = min(4, rep - r0);
         float acc[4][VE] = {};
         if (slice < ks) {
-            const CT *vr = vc + (size_t)key0 * a.ldv + vec * VE;
-#pragma unroll 4
-            for (int k = slice; k < nk; k += ks) {
+            auto add = [&](int k, const uint4 &raw) {
                 float vv[VE];
-                Vec<CT>::load(vr + (size_t)k * a.ldv, vv);
+                Vec<CT>::unpack(raw, vv);
 #pragma unroll
                 for (int r = 0; r < 4; r++) {
                     if (r < nr) {
@@ -164,7 +173,11 @@ __global__ void __launch_bounds__(kDecThreads) mix_attn_decode_kernel(const MixA
                         for (int e = 0; e < VE; e++) acc[r][e] = fmaf(w, vv[e], acc[r][e]);
                     }
                 }
-            }
+            };
+#pragma unroll
+            for (int u = 0; u < PV; u++)
+                if (slice + u * ks < nk) add(slice + u * ks, pv[u]);
+            for (int k = slice + PV * ks; k < nk; k += ks) add(k, *reinterpret_cast<const uint4 *>(vr + (size_t)k * a.ldv));
 #pragma unroll
             for (int r = 0; r < 4; r++)
                 if (r < nr)
