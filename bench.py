@@ -20,7 +20,8 @@ are seeded synthetic GGUF blocks (no model file is needed or read).  Prints ONE 
 With N > 1 every rank decodes its own replica of the 8B model (no exchange step on this path): weak scaling; the
 headline stays that.  A `tp` object is added: the 70B-shaped model of config C4 split over the N ranks (tensor
 parallel, one process per GPU), its per-token all-reduce cost, and the same model on one GPU.
---workload c1 / c3 / qgemm / qrows / prefill-2layer run only that part (small cases for profiler captures among them).
+--workload c1 / c3 / qgemm / qrows / prefill-2layer / mukutar / mukutar-3layer run only that part (small cases for profiler captures
+among them; mukutar: the layered models of tl_b200/csrc/layered.cu beside a Llama model of the same sizes).
 """
 import argparse
 import json

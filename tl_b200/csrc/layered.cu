@@ -44,10 +44,10 @@ struct LayeredModel {
     std::vector<Storage *> stores;
     std::vector<RotTable> rots;
     // rows of the batch: projections, mixer output, up projection (f32); activation rows of the batch path
-    float *proj = nullptr, *mix = nullptr, *up = nullptr, *partial = nullptr, *dly = nullptr;
+    float *proj = nullptr, *mix = nullptr, *up = nullptr, *partial = nullptr;
     void *act = nullptr;
     int *counters = nullptr;
-    int ldp = 0, ldm = 0, ldu = 0, lda = 0, ldd = 0;
+    int ldp = 0, ldm = 0, ldu = 0, lda = 0;
     uint64_t weight_bytes = 0;
 };
 
@@ -320,7 +320,7 @@ tlb_status layered_create(LayeredModel **out, const ModelDesc &desc, tlb_map *m,
         TLB_TRY(ld.vec("final.norm", &lm->final_norm, W));
         size_t part = 1;
         int kvh = 1;
-        lm->ldp = lm->ldm = lm->ldu = lm->ldd = 8;
+        lm->ldp = lm->ldm = lm->ldu = 8;
         lm->lda = act_ld(W);
         for (const Layer &L : lm->layers) {
             lm->ldp = std::max(lm->ldp, act_ld(L.in.n));
