@@ -7,6 +7,7 @@
 //   dense_gemm_f32_kernel many rows, f32 activations: plain f32 multiply-adds (no tensor core rounds the operands).
 #include <algorithm>
 
+#include "act.cuh"
 #include "layered_kernels.h"
 #include "tc05.cuh"
 
@@ -41,6 +42,21 @@ struct DenseMvParams {
     float *out;
     const float *resid_scale;
     int tiles;
+    float softcap;
+    int groups;
+    const float *y, *y_gate, *post_w;
+    float *h_out;
+    int act;
+    float *state;
+    size_t parity_stride;
+    const int *pos;
+    RouteDesc route;
+    const float *logits;
+    int *sel;
+    float *weight;
+    const __nv_bfloat16 *shared_w;
+    int shared_k, shared_ld, seg_nch;      // seg_nch: chunks of one expert
+    const float *shared_x, *shared_gate;
 };
 
 // Shared position of activation element e: inside a chunk of 256 the first four of every eight come first, so that a lane's
@@ -70,20 +86,26 @@ template <int PRO, int WK>
 __global__ void __launch_bounds__(kMvThreads, 4) dense_matvec_kernel(const DenseMvParams p)
 {
     constexpr int GROUPS = kMvWarps / WK, TILE = GROUPS * kMvRows;
+    constexpr bool GNORM = PRO == DPRO_GNORM, EXPERT = PRO == DPRO_EXPERT, EXPERTS = PRO == DPRO_EXPERTS;
     extern __shared__ __align__(16) float xs[];
-    __shared__ float red[kMvWarps * 3];
+    __shared__ float red[GNORM ? 2 * kMaxNormGroups : kMvWarps * 3];
     __shared__ float fold[2][GROUPS][WK][kMvRows];
+    __shared__ int s_sel[EXPERT ? kMaxTop : 1];
+    __shared__ float s_weight[EXPERT ? kMaxTop : 1];
+    __shared__ const __nv_bfloat16 *s_base[EXPERTS ? kMaxTop + 1 : 1];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, wk = warp % WK, wg = warp / WK;
 
     // what the first tile reads does not depend on the launch before: ask L2 for it before waiting
-    {
+    if (!EXPERT) {
         const int r0 = blockIdx.x * TILE + wg * kMvRows;
-        for (int r = 0; r < kMvRows; r++) {
+        const __nv_bfloat16 *w0 = EXPERTS ? p.shared_w : p.w;         // which experts' rows is not known yet
+        const int ld = EXPERTS ? p.shared_ld : p.ld, nch = EXPERTS ? (p.shared_ld + kMvChunk - 1) / kMvChunk : p.nch;
+        for (int r = 0; r < kMvRows && w0; r++) {
             const int row = min(r0 + r, p.n - 1);
-            const __nv_bfloat16 *src = p.w + (size_t)row * p.ld;
-            for (int c = wk + (lane >> 2) * WK; c < p.nch; c += 8 * WK) {
+            const __nv_bfloat16 *src = w0 + (size_t)row * ld;
+            for (int c = wk + (lane >> 2) * WK; c < nch; c += 8 * WK) {
                 const int e = c * kMvChunk + (lane & 3) * 64;
-                if (e < p.ld) asm volatile("prefetch.global.L2 [%0];" ::"l"(src + e));
+                if (e < ld) asm volatile("prefetch.global.L2 [%0];" ::"l"(src + e));
             }
         }
     }
@@ -91,8 +113,18 @@ __global__ void __launch_bounds__(kMvThreads, 4) dense_matvec_kernel(const Dense
     pdl_launch_dependents();
 
     const int kp = p.nch * kMvChunk;
-    if (PRO == DPRO_PLAIN) {
+    const __nv_bfloat16 *wbase = p.w;
+    float *outp = p.out;
+    if (PRO == DPRO_PLAIN || EXPERT) {
         for (int e = tid; e < kp; e += kMvThreads) xs[xs_at(e)] = e < p.k ? __ldcg(p.x + e) : 0.f;
+        if (EXPERT) {
+            route_token(p.logits, p.route, xs + kp, s_sel, s_weight);
+            const int slot = blockIdx.y;
+            wbase += (size_t)s_sel[slot] * p.n * p.ld;
+            outp += (size_t)slot * p.n;
+            if (blockIdx.x == 0 && slot == 0)
+                for (int i = tid; i < p.route.top; i += kMvThreads) { p.sel[i] = s_sel[i]; p.weight[i] = s_weight[i]; }
+        }
     } else if (PRO == DPRO_NORM) {
         const __nv_bfloat16 *er = p.emb ? p.emb + (size_t)*p.token * p.emb_ld : nullptr;
         float ss[1] = {0.f};
@@ -108,6 +140,67 @@ __global__ void __launch_bounds__(kMvThreads, 4) dense_matvec_kernel(const Dense
             float *s = xs + xs_at(e);
             *s = e < p.k ? *s * inv * (p.norm_w[e] + p.norm_offset) : 0.f;
         }
+    } else if (GNORM) {
+        const __nv_bfloat16 *er = p.emb ? p.emb + (size_t)*p.token * p.emb_ld : nullptr;
+        const int len = p.k / p.groups;
+        float *inv = red + kMaxNormGroups;
+        auto at = [&](int e) { return xs[xs_at(e)]; };
+        if (p.y) {
+            for (int e = tid; e < p.k; e += kMvThreads) {
+                const float v = __ldcg(p.y + e);
+                xs[xs_at(e)] = p.y_gate ? v * sigmoidf(__ldcg(p.y_gate + e)) : v;
+            }
+            __syncthreads();
+            group_inv_rms(at, p.k, p.groups, p.eps, red, inv);
+            for (int e = tid; e < p.k; e += kMvThreads) {
+                float *s = xs + xs_at(e);
+                const float v = __ldcg(p.x + e) + *s * inv[e / len] * (p.post_w[e] + p.norm_offset);
+                *s = v;
+                if (blockIdx.x == 0) p.x_out[e] = v;
+            }
+        } else {
+            for (int e = tid; e < p.k; e += kMvThreads) {
+                const float v = er ? __bfloat162float(er[e]) : __ldcg(p.x + e);
+                xs[xs_at(e)] = v;
+                if (er && blockIdx.x == 0) p.x_out[e] = v;
+            }
+        }
+        __syncthreads();
+        group_inv_rms(at, p.k, p.groups, p.eps, red, inv);
+        for (int e = tid; e < kp; e += kMvThreads) {
+            float *s = xs + xs_at(e);
+            *s = e < p.k ? *s * inv[e / len] * (p.norm_w[e] + p.norm_offset) : 0.f;
+            if (p.h_out && blockIdx.x == 0 && e < p.k) p.h_out[e] = *s;
+        }
+    } else if (PRO == DPRO_GLU) {
+        for (int e = tid; e < kp; e += kMvThreads) xs[xs_at(e)] = e < p.k ? glu_act(p.act, __ldcg(p.x + e), __ldcg(p.x + p.k + e)) : 0.f;
+    } else if (PRO == DPRO_GRU) {
+        const int pos = __ldcg(p.pos);
+        const float *sin = p.state + (size_t)(pos & 1) * p.parity_stride;
+        float *sout = p.state + (size_t)((pos & 1) ^ 1) * p.parity_stride;
+        for (int e = tid; e < kp; e += kMvThreads) {
+            float v = 0.f;
+            if (e < p.k) {
+                const float z = sigmoidf(__ldcg(p.x + e)), c = gru_candidate(__ldcg(p.x + p.k + e)), old = pos > 0 ? __ldcg(sin + e) : 0.f;
+                const float st = (1.f - z) * old + z * c;
+                if (blockIdx.x == 0) sout[e] = st;
+                v = st * siluf(__ldcg(p.x + 2 * p.k + e));
+            }
+            xs[xs_at(e)] = v;
+        }
+    } else if (EXPERTS) {
+        const int top = p.route.top;
+        for (int s = 0; s < top; s++) {
+            const float w = __ldcg(p.weight + s);
+            const float *x = p.x + (size_t)s * 2 * p.k;
+            float *dst = xs + s * p.seg_nch * kMvChunk;
+            for (int e = tid; e < p.seg_nch * kMvChunk; e += kMvThreads) dst[xs_at(e)] = e < p.k ? w * glu_act(p.act, __ldcg(x + e), __ldcg(x + p.k + e)) : 0.f;
+        }
+        const int first = top * p.seg_nch * kMvChunk;
+        const float w = p.shared_gate ? sigmoidf(__ldcg(p.shared_gate)) : 1.f;
+        for (int e = tid; e < kp - first; e += kMvThreads)
+            xs[first + xs_at(e)] = e < p.shared_k ? w * glu_act(p.act, __ldcg(p.shared_x + e), __ldcg(p.shared_x + p.shared_k + e)) : 0.f;
+        for (int s = tid; s <= top; s += kMvThreads) s_base[s] = s < top ? p.w + (size_t)__ldcg(p.sel + s) * p.n * p.ld : p.shared_w;
     } else {
         float ss[3] = {0.f, 0.f, 0.f};
         for (int e = tid; e < p.k; e += kMvThreads) {
@@ -132,12 +225,20 @@ __global__ void __launch_bounds__(kMvThreads, 4) dense_matvec_kernel(const Dense
         const int r0 = tile * TILE + wg * kMvRows;
         const uint4 *rows[kMvRows];
 #pragma unroll
-        for (int r = 0; r < kMvRows; r++) rows[r] = reinterpret_cast<const uint4 *>(p.w + (size_t)min(r0 + r, p.n - 1) * p.ld) + lane;
+        for (int r = 0; r < kMvRows; r++) rows[r] = reinterpret_cast<const uint4 *>(wbase + (size_t)min(r0 + r, p.n - 1) * p.ld) + lane;
         float acc[kMvRows] = {0.f, 0.f, 0.f, 0.f};
         auto load = [&](int c, uint4 (&v)[kMvRows]) {
-            const bool in = c < p.nch && c * kMvChunk + lane * 8 < p.ld;
+            if constexpr (EXPERTS) {
+                const int seg = min(c / p.seg_nch, p.route.top), col = (c - seg * p.seg_nch) * kMvChunk + lane * 8, ld = seg < p.route.top ? p.ld : p.shared_ld;
+                const bool in = c < p.nch && col < ld;
 #pragma unroll
-            for (int r = 0; r < kMvRows; r++) v[r] = in ? __ldcs(rows[r] + c * (kMvChunk / 8)) : make_uint4(0u, 0u, 0u, 0u);
+                for (int r = 0; r < kMvRows; r++)
+                    v[r] = in ? __ldcs(reinterpret_cast<const uint4 *>(s_base[seg] + (size_t)min(r0 + r, p.n - 1) * ld + col)) : make_uint4(0u, 0u, 0u, 0u);
+            } else {
+                const bool in = c < p.nch && c * kMvChunk + lane * 8 < p.ld;
+#pragma unroll
+                for (int r = 0; r < kMvRows; r++) v[r] = in ? __ldcs(rows[r] + c * (kMvChunk / 8)) : make_uint4(0u, 0u, 0u, 0u);
+            }
         };
         auto mul = [&](int c, const uint4 (&v)[kMvRows]) {
             if (c >= p.nch) return;
@@ -175,8 +276,9 @@ __global__ void __launch_bounds__(kMvThreads, 4) dense_matvec_kernel(const Dense
         const int row = r0 + lane;
         if (wk == 0 && lane < kMvRows && row < p.n) {
             if (p.bias) y += p.bias[row];
-            if (p.resid_scale) p.out[row] = __ldcg(p.out + row) + p.resid_scale[row] * y;
-            else p.out[row] = y;
+            if (p.softcap > 0.f) y = p.softcap * tanhf(y / p.softcap);
+            if (p.resid_scale) outp[row] = __ldcg(outp + row) + p.resid_scale[row] * y;
+            else outp[row] = y;
         }
     }
 }
@@ -191,6 +293,12 @@ struct DenseTcParams {
     int n, T, ldo, nt, kt, stages;
     uint32_t tmem_cols;
     int *err;
+    float softcap;
+    int per;
+    size_t block_stride;
+    __half *out_h;
+    const int4 *tiles;
+    uint32_t type_bits;                    // operand types in the instruction descriptor
 };
 
 // One CTA: 128 weight rows (lanes of the accumulator) x nt tokens (its columns).  Warps 0-3 write out (a warp's 32 lanes are 32
@@ -207,7 +315,13 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_cons
     const uint32_t xbytes = (uint32_t)p.nt * (kTcK * 2), stage = kTcWBytes + xbytes;
     const uint32_t bars = base + (uint32_t)p.stages * stage;
     const uint32_t full = bars, empty = bars + 8u * p.stages, done = bars + 16u * p.stages;
-    const int t0 = blockIdx.x * p.nt, n0 = blockIdx.y * kTcRows;
+    const int n0 = blockIdx.y * kTcRows;
+    int t0 = blockIdx.x * p.nt, t_end = p.T, wrow0 = n0;
+    if (p.tiles) {                         // rows of one of several stacked weights
+        const int4 tile = p.tiles[blockIdx.x];
+        if (tile.z <= 0) return;
+        t0 = tile.y; t_end = tile.y + tile.z; wrow0 = tile.x * p.n + n0;
+    }
 
     if (tid == 0) {
         abort_word = 0;
@@ -231,14 +345,24 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_cons
             const int row = n0 + warp * 32 + lane;
             const bool in = row < p.n;
             const float bias = in && p.bias ? p.bias[row] : 0.f, rs = in && p.resid_scale ? p.resid_scale[row] : 0.f;
-            for (int c0 = 0; c0 < p.nt && t0 + c0 < p.T; c0 += 32) {
+            const size_t place = (size_t)(row / p.per) * p.block_stride + row % p.per;
+            for (int c0 = 0; c0 < p.nt && t0 + c0 < t_end; c0 += 32) {
                 uint32_t v[32];
                 tmem_ld32(tmem + ((uint32_t)(warp * 32) << 16) + (uint32_t)c0, v);
                 tmem_wait_ld();
                 if (!in) continue;
-                float *dst = p.out + (size_t)(t0 + c0) * p.ldo + row;
-                const int m = min(32, p.T - t0 - c0);
-                if (p.resid_scale) {
+                float *dst = p.out + (size_t)(t0 + c0) * p.ldo + place;
+                const int m = min(32, t_end - t0 - c0);
+                if (p.out_h) {
+                    __half *dh = p.out_h + (size_t)(t0 + c0) * p.ldo + place;
+#pragma unroll
+                    for (int i = 0; i < 32; i++)
+                        if (i < m) dh[(size_t)i * p.ldo] = __float2half_rn(fminf(fmaxf(__uint_as_float(v[i]) + bias, -65504.f), 65504.f));
+                } else if (p.softcap > 0.f) {
+#pragma unroll 4
+                    for (int i = 0; i < 32; i++)
+                        if (i < m) dst[(size_t)i * p.ldo] = p.softcap * tanhf((__uint_as_float(v[i]) + bias) / p.softcap);
+                } else if (p.resid_scale) {
                     float r[32];
 #pragma unroll
                     for (int i = 0; i < 32; i++) r[i] = i < m ? dst[(size_t)i * p.ldo] : 0.f;
@@ -259,7 +383,7 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_cons
                 const int s = k % p.stages;
                 if (k >= p.stages && !mbar_wait(empty + 8 * s, (uint32_t)(k / p.stages - 1) & 1u, abort_flag, p.err, 62)) break;
                 mbar_expect_tx(full + 8 * s, stage);
-                tma_load_2d(base + (uint32_t)s * stage, &wmap, k * kTcK, n0, full + 8 * s);
+                tma_load_2d(base + (uint32_t)s * stage, &wmap, k * kTcK, wrow0, full + 8 * s);
                 tma_load_2d(base + (uint32_t)s * stage + kTcWBytes, &xmap, k * kTcK, t0, full + 8 * s);
                 issued = k + 1;
             }
@@ -267,8 +391,8 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_cons
                 for (int k = max(0, issued - p.stages); k < issued; k++) mbar_wait_drain(full + 8 * (k % p.stages), (uint32_t)(k / p.stages) & 1u);
         }
     } else if (lane == 0) {
-        // f32 accumulator, bf16 operands, both K-major, M 128, N nt
-        const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(p.nt >> 3) << 17) | ((uint32_t)(kTcRows >> 4) << 24);
+        // f32 accumulator, operands of one 16-bit type, both K-major, M 128, N nt
+        const uint32_t idesc = (1u << 4) | p.type_bits | ((uint32_t)(p.nt >> 3) << 17) | ((uint32_t)(kTcRows >> 4) << 24);
         for (int k = 0; k < p.kt; k++) {
             const int s = k % p.stages;
             if (!mbar_wait(full + 8 * s, (uint32_t)(k / p.stages) & 1u, abort_flag, p.err, 63)) break;
@@ -296,20 +420,31 @@ struct DenseF32Params {
     const float *bias, *x, *resid_scale;
     int ldx, T, ldo;
     float *out;
+    float softcap;
+    int per;
+    size_t block_stride;
+    const int4 *tiles;
 };
-constexpr int kSgT = 64, kSgN = 64, kSgK = 16;
+constexpr int kSgT = kF32GemmRows, kSgN = 64, kSgK = 16;
 
 __global__ void __launch_bounds__(256) dense_gemm_f32_kernel(const DenseF32Params p)
 {
     __shared__ float sx[kSgK][kSgT + 4], sw[kSgK][kSgN + 4];
-    const int tid = threadIdx.x, n0 = blockIdx.y * kSgN, t0 = blockIdx.x * kSgT;
+    const int tid = threadIdx.x, n0 = blockIdx.y * kSgN;
     const int tn = tid & 15, tt = tid >> 4;
+    int t0 = blockIdx.x * kSgT, t_end = p.T;
+    const __nv_bfloat16 *w = p.w;
+    if (p.tiles) {
+        const int4 tile = p.tiles[blockIdx.x];
+        if (tile.z <= 0) return;
+        t0 = tile.y; t_end = tile.y + tile.z; w += (size_t)tile.x * p.n * p.ld;
+    }
     float acc[4][4] = {};
     for (int k0 = 0; k0 < p.k; k0 += kSgK) {
         for (int i = tid; i < kSgT * kSgK; i += 256) {
             const int r = i / kSgK, c = i % kSgK;
-            sx[c][r] = t0 + r < p.T && k0 + c < p.k ? p.x[(size_t)(t0 + r) * p.ldx + k0 + c] : 0.f;
-            sw[c][r] = n0 + r < p.n && k0 + c < p.k ? __bfloat162float(p.w[(size_t)(n0 + r) * p.ld + k0 + c]) : 0.f;
+            sx[c][r] = t0 + r < t_end && k0 + c < p.k ? p.x[(size_t)(t0 + r) * p.ldx + k0 + c] : 0.f;
+            sw[c][r] = n0 + r < p.n && k0 + c < p.k ? __bfloat162float(w[(size_t)(n0 + r) * p.ld + k0 + c]) : 0.f;
         }
         __syncthreads();
 #pragma unroll
@@ -328,10 +463,11 @@ __global__ void __launch_bounds__(256) dense_gemm_f32_kernel(const DenseF32Param
 #pragma unroll
         for (int j = 0; j < 4; j++) {
             const int t = t0 + tt * 4 + i, n = n0 + tn * 4 + j;
-            if (t >= p.T || n >= p.n) continue;
-            float *o = p.out + (size_t)t * p.ldo + n;
-            if (p.resid_scale) *o = fmaf(p.resid_scale[n], acc[i][j], *o);
-            else *o = acc[i][j] + (p.bias ? p.bias[n] : 0.f);
+            if (t >= t_end || n >= p.n) continue;
+            float *o = p.out + (size_t)t * p.ldo + (size_t)(n / p.per) * p.block_stride + n % p.per;
+            if (p.resid_scale) { *o = fmaf(p.resid_scale[n], acc[i][j], *o); continue; }
+            const float y = acc[i][j] + (p.bias ? p.bias[n] : 0.f);
+            *o = p.softcap > 0.f ? p.softcap * tanhf(y / p.softcap) : y;
         }
 }
 
@@ -446,6 +582,12 @@ __global__ void pack_rows_kernel(const __nv_bfloat16 *__restrict__ src, int k, _
     for (int i = threadIdx.x; i < k; i += blockDim.x) dst[(size_t)blockIdx.x * ld + i] = src[(size_t)blockIdx.x * k + i];
 }
 
+__global__ void pack_rows_f16_kernel(const __nv_bfloat16 *__restrict__ src, int k, __half *__restrict__ dst, int ld)
+{
+    for (int i = threadIdx.x; i < ld; i += blockDim.x)
+        dst[(size_t)blockIdx.x * ld + i] = i < k ? __float2half_rn(fminf(fmaxf(__bfloat162float(src[(size_t)blockIdx.x * k + i]), -65504.f), 65504.f)) : __float2half_rn(0.f);
+}
+
 tlb_status launched(const char *what)
 {
     cudaError_t e = cudaGetLastError();
@@ -458,15 +600,15 @@ template <int PRO, int WK>
 tlb_status run_matvec(const DenseMvParams &p, bool pdl)
 {
     Context *c = ctx();
-    const size_t smem = (size_t)p.nch * kMvChunk * sizeof(float);
+    const size_t smem = ((size_t)p.nch * kMvChunk + (PRO == DPRO_EXPERT ? route_scratch_floats(p.route) : 0)) * sizeof(float);
     static size_t allowed = 48 << 10;
     if (smem > allowed) {
         TLB_CUDA(cudaFuncSetAttribute(dense_matvec_kernel<PRO, WK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         allowed = smem;
     }
     const int per_sm = std::max(1, std::min(4, (int)(((size_t)220 << 10) / (smem + 2048))));
-    const int grid = std::min(p.tiles, c->sm_count * per_sm);
-    TLB_CUDA(launch_chained(dense_matvec_kernel<PRO, WK>, dim3(grid), dim3(kMvThreads), smem, pdl, p));
+    const int slots = PRO == DPRO_EXPERT ? p.route.top : 1, grid = std::min(p.tiles, std::max(1, c->sm_count * per_sm / slots));
+    TLB_CUDA(launch_chained(dense_matvec_kernel<PRO, WK>, dim3(grid, slots), dim3(kMvThreads), smem, pdl, p));
     count_launch();
     return TLB_OK;
 }
@@ -477,7 +619,8 @@ tlb_status pick_matvec(DenseMvParams p, bool pdl)
     // the fewest warps per row group that still give every SM two tiles
     int wk = 1;
     auto tiles = [&](int w) { return (p.n + kMvWarps / w * kMvRows - 1) / (kMvWarps / w * kMvRows); };
-    while (wk < 8 && tiles(wk) < 2 * ctx()->sm_count && wk * 2 <= p.nch) wk *= 2;
+    const int slots = PRO == DPRO_EXPERT ? p.route.top : 1;
+    while (wk < 8 && tiles(wk) * slots < 2 * ctx()->sm_count && wk * 2 <= p.nch) wk *= 2;
     p.tiles = tiles(wk);
     switch (wk) {
     case 1: return run_matvec<PRO, 1>(p, pdl);
@@ -491,6 +634,12 @@ tlb_status pick_matvec(DenseMvParams p, bool pdl)
 
 bool dense_matvec_supported(int k) { return k >= 1 && k <= 48 * 1024; }
 
+bool experts_matvec_supported(const RouteDesc &r, int ff, int shared_ff)
+{
+    const int nch = r.top * ((ff + kMvChunk - 1) / kMvChunk) + (shared_ff + kMvChunk - 1) / kMvChunk;
+    return r.top >= 1 && r.top <= kMaxTop && r.experts <= kMaxExperts && nch <= 48 * 1024 / kMvChunk;
+}
+
 tlb_status launch_dense_matvec(const DenseMatvecJob &j)
 {
     if (!ctx()) return TLB_ERR_DEVICE;
@@ -499,6 +648,19 @@ tlb_status launch_dense_matvec(const DenseMatvecJob &j)
     p.w = j.w.w; p.n = j.w.n; p.k = j.w.k; p.ld = j.w.ld; p.nch = (j.w.ld + kMvChunk - 1) / kMvChunk;
     p.bias = j.w.bias; p.x = j.x; p.emb = j.emb; p.emb_ld = act_ld(j.w.k); p.token = j.token; p.x_out = j.x_out;
     p.norm_w = j.norm_w; p.norm_offset = j.norm_offset; p.eps = j.eps; p.poly = j.poly; p.out = j.out; p.resid_scale = j.resid_scale;
+    p.softcap = j.softcap; p.groups = j.groups; p.y = j.y; p.y_gate = j.y_gate; p.post_w = j.post_w; p.h_out = j.h_out; p.act = j.act;
+    p.state = j.state; p.parity_stride = j.parity_stride; p.pos = j.pos;
+    p.route = j.route; p.logits = j.logits; p.sel = j.sel; p.weight = j.weight;
+    if (j.pro == DPRO_EXPERTS) {
+        p.seg_nch = p.nch;
+        p.shared_w = j.shared.w; p.shared_k = j.shared.k; p.shared_ld = j.shared.ld; p.shared_x = j.shared_x; p.shared_gate = j.shared_gate;
+        p.nch = j.route.top * p.seg_nch + (j.shared.ld + kMvChunk - 1) / kMvChunk;
+        return pick_matvec<DPRO_EXPERTS>(p, j.pdl);
+    }
+    if (j.pro == DPRO_GNORM) return pick_matvec<DPRO_GNORM>(p, j.pdl);
+    if (j.pro == DPRO_GLU) return pick_matvec<DPRO_GLU>(p, j.pdl);
+    if (j.pro == DPRO_GRU) return pick_matvec<DPRO_GRU>(p, j.pdl);
+    if (j.pro == DPRO_EXPERT) return pick_matvec<DPRO_EXPERT>(p, j.pdl);
     if (j.pro == DPRO_NORM) return pick_matvec<DPRO_NORM>(p, j.pdl);
     if (j.pro == DPRO_POLY) return pick_matvec<DPRO_POLY>(p, j.pdl);
     return pick_matvec<DPRO_PLAIN>(p, j.pdl);
@@ -509,16 +671,20 @@ tlb_status launch_dense_gemm(const DenseGemmJob &j, bool f32)
     Context *c = ctx();
     if (!c) return TLB_ERR_DEVICE;
     if (j.T < 1) return TLB_OK;
+    const int per = j.per > 0 ? j.per : j.w.n;
     if (f32) {
         DenseF32Params p;
+        p.softcap = j.softcap; p.per = per; p.block_stride = j.block_stride; p.tiles = j.tiles;
         p.w = j.w.w; p.n = j.w.n; p.k = j.w.k; p.ld = j.w.ld; p.bias = j.w.bias; p.x = (const float *)j.x; p.resid_scale = j.resid_scale;
         p.ldx = j.ldx; p.T = j.T; p.ldo = j.ldo; p.out = j.out;
-        dense_gemm_f32_kernel<<<dim3((j.T + kSgT - 1) / kSgT, (j.w.n + kSgN - 1) / kSgN), 256, 0, c->stream>>>(p);
+        dense_gemm_f32_kernel<<<dim3(j.tiles ? j.n_tiles : (j.T + kSgT - 1) / kSgT, (j.w.n + kSgN - 1) / kSgN), 256, 0, c->stream>>>(p);
         return launched("f32 GEMM launch");
     }
     DenseTcParams p;
     p.out = j.out; p.bias = j.w.bias; p.resid_scale = j.resid_scale; p.n = j.w.n; p.T = j.T; p.ldo = j.ldo;
-    p.nt = std::min(256, (j.T + 31) / 32 * 32);
+    p.softcap = j.softcap; p.per = per; p.block_stride = j.block_stride; p.out_h = j.out_h; p.tiles = j.tiles;
+    p.type_bits = j.w.f16 ? 0u : (1u << 7) | (1u << 10);
+    p.nt = j.tiles ? j.tile_rows : std::min(256, (j.T + 31) / 32 * 32);
     p.tmem_cols = 32;
     while (p.tmem_cols < (uint32_t)p.nt) p.tmem_cols *= 2;
     p.kt = (j.w.k + kTcK - 1) / kTcK;
@@ -526,8 +692,9 @@ tlb_status launch_dense_gemm(const DenseGemmJob &j, bool f32)
     p.stages = (int)std::min<size_t>(8, ((size_t)216 << 10) / stage);
     p.err = c->err_flag;
     CUtensorMap wmap, xmap;
-    if (!encode_f16_map(&wmap, j.w.w, (uint64_t)j.w.k, (uint64_t)j.w.n, (uint64_t)j.w.ld * 2, kTcK, kTcRows, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16) ||
-        !encode_f16_map(&xmap, j.x, (uint64_t)j.w.k, (uint64_t)j.T, (uint64_t)j.ldx * 2, kTcK, (uint32_t)p.nt, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16))
+    const CUtensorMapDataType type = j.w.f16 ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
+    if (!encode_f16_map(&wmap, j.w.w, (uint64_t)j.w.k, (uint64_t)j.w.n * j.n_weights, (uint64_t)j.w.ld * 2, kTcK, kTcRows, type) ||
+        !encode_f16_map(&xmap, j.x, (uint64_t)j.w.k, (uint64_t)j.T, (uint64_t)j.ldx * 2, kTcK, (uint32_t)p.nt, type))
         return fail(TLB_ERR_DEVICE, "GEMM: cuTensorMapEncodeTiled failed or is not available");
     const size_t smem = (size_t)p.stages * stage + 16 * p.stages + 8 + 1024;
     static size_t allowed = 0;
@@ -535,7 +702,7 @@ tlb_status launch_dense_gemm(const DenseGemmJob &j, bool f32)
         TLB_CUDA(cudaFuncSetAttribute(dense_gemm_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         allowed = smem;
     }
-    dense_gemm_tc_kernel<<<dim3((j.T + p.nt - 1) / p.nt, (j.w.n + kTcRows - 1) / kTcRows), kTcThreads, smem, c->stream>>>(wmap, xmap, p);
+    dense_gemm_tc_kernel<<<dim3(j.tiles ? j.n_tiles : (j.T + p.nt - 1) / p.nt, (j.w.n + kTcRows - 1) / kTcRows), kTcThreads, smem, c->stream>>>(wmap, xmap, p);
     return launched("GEMM launch");
 }
 
@@ -568,6 +735,12 @@ tlb_status launch_gather_rows(const float *x, int width, const int *idx, int n, 
 tlb_status launch_pack_rows(const __nv_bfloat16 *src, int n, int k, __nv_bfloat16 *dst, int ld, int col0)
 {
     pack_rows_kernel<<<n, 256, 0, ctx()->stream>>>(src, k, dst + col0, ld);
+    return launched("weight packing launch");
+}
+
+tlb_status launch_pack_rows_f16(const __nv_bfloat16 *src, int n, int k, void *dst, int ld)
+{
+    pack_rows_f16_kernel<<<n, 256, 0, ctx()->stream>>>(src, k, (__half *)dst, ld);
     return launched("weight packing launch");
 }
 

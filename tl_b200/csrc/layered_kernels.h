@@ -13,11 +13,25 @@ struct DenseW {
     const __nv_bfloat16 *w = nullptr;
     int n = 0, k = 0, ld = 0;
     const float *bias = nullptr;
+    bool f16 = false;                     // w holds f16 instead of bf16 (GEMM over f16 rows only)
 };
 inline int act_ld(int k) { return (k + 7) / 8 * 8; }   // pitch of an activation row that feeds a [.., k] weight
 
 // What the rows of a linear layer's input are made from.
-enum DensePro { DPRO_PLAIN = 0, DPRO_NORM = 1, DPRO_POLY = 2 };
+enum DensePro {
+    DPRO_PLAIN = 0,
+    DPRO_NORM = 1,      // x / rms * weight
+    DPRO_POLY = 2,      // PolyNorm
+    DPRO_GNORM = 3,     // residual step of the sublayer before, then the norm in groups
+    DPRO_GLU = 4,       // act(gate) * up
+    DPRO_GRU = 5,       // gated recurrence: new state * silu(gate)
+    DPRO_EXPERT = 6,    // plain x; the weight is the expert the router gave this launch's blockIdx.y
+    DPRO_EXPERTS = 7,   // act(gate) * up of the chosen experts and the shared one, each times its weight, side by side
+};
+enum GluAct { GLU_SILU = 0, GLU_GELU_TANH = 1 };
+// Router of a mixture of experts: the `top` best of the experts of the `keep` best groups; weights are scores over their sum * scale.
+struct RouteDesc { int experts = 0, groups = 1, keep = 1, top = 0; float scale = 1.f; };
+constexpr int kMaxTop = 64, kMaxExperts = 1024;
 // One row through one weight (f32 activation, f32 accumulation): out = W pro(x) [+ bias], or with resid_scale
 // out[i] += resid_scale[i] * (W pro(x))[i].
 struct DenseMatvecJob {
@@ -32,10 +46,31 @@ struct DenseMatvecJob {
     const float *poly = nullptr;          // POLY: four numbers
     float *out = nullptr;
     const float *resid_scale = nullptr;
+    float softcap = 0.f;                  // > 0: out = softcap * tanh(. / softcap)
+    // GNORM: the norms are taken over `groups` equal parts.  With y the residual moves on first: x + norm(y * sigmoid(y_gate)) *
+    // (post_w + norm_offset); CTA 0 stores it to x_out (not x itself) and, if asked, the normed row to h_out.
+    int groups = 1;
+    const float *y = nullptr, *y_gate = nullptr, *post_w = nullptr;
+    float *h_out = nullptr;
+    int act = GLU_SILU;                   // GLU, EXPERTS: x = gate [k] | up [k]
+    // GRU: x = z | u | gate, each [k]; state of position p at state + (p & 1) * parity_stride, the next one in the other half
+    float *state = nullptr;
+    size_t parity_stride = 0;
+    const int *pos = nullptr;
+    // EXPERT: w.n rows per expert, experts stacked; slot s of the choice goes to out + s * w.n.  The choice is stored to sel / weight.
+    // EXPERTS: w [experts * w.n, ff]; x [top][2 ff]; the shared expert (shared.w may be null) has gate | up at shared_x and the logit
+    // of its weight at shared_gate (null: one)
+    RouteDesc route;
+    const float *logits = nullptr;
+    int *sel = nullptr;
+    float *weight = nullptr;
+    DenseW shared;
+    const float *shared_x = nullptr, *shared_gate = nullptr;
     bool pdl = true;
 };
 tlb_status launch_dense_matvec(const DenseMatvecJob &j);
 bool dense_matvec_supported(int k);
+bool experts_matvec_supported(const RouteDesc &r, int ff, int shared_ff);
 
 // T rows: x [T, ldx] in the model's activation type (bf16 or f32)
 struct DenseGemmJob {
@@ -45,8 +80,17 @@ struct DenseGemmJob {
     float *out = nullptr;                 // [T, ldo]
     int ldo = 0;
     const float *resid_scale = nullptr;   // out[t][i] += resid_scale[i] * y instead of out = y + bias
+    float softcap = 0.f;
+    // columns in blocks of `per` (0: all), block b at out + b * block_stride; out_h: f16 output at the same places
+    int per = 0;
+    size_t block_stride = 0;
+    __half *out_h = nullptr;
+    // several weights [.., k] of w.n rows each, stacked: tile i covers rows y .. y + z - 1 of x and multiplies them with weight x
+    const int4 *tiles = nullptr;
+    int n_tiles = 0, tile_rows = 0, n_weights = 1;
 };
 tlb_status launch_dense_gemm(const DenseGemmJob &j, bool f32);
+constexpr int kF32GemmRows = 64;          // rows of a tile of the 32-bit GEMM
 
 // rows in the activation type, pitch ld
 tlb_status launch_norm_rows(const float *x, int T, int width, const float *w, float offset, float eps, void *out, int ld, bool f32);
@@ -54,6 +98,49 @@ tlb_status launch_poly_rows(const float *z, int T, int ff, int ldz, const float 
 tlb_status launch_embed_bf16(const int *tokens, const __nv_bfloat16 *table, int width, int ld, float *x, int T);
 tlb_status launch_gather_rows(const float *x, int width, const int *idx, int n, float *out);
 tlb_status launch_pack_rows(const __nv_bfloat16 *src, int n, int k, __nv_bfloat16 *dst, int ld, int col0);
+tlb_status launch_pack_rows_f16(const __nv_bfloat16 *src, int n, int k, void *dst, int ld);      // values as f16
+
+// ---------------------------------------------------------------- row_kernels.cu
+// act(gate) * up of rows z: gate at column 0, up at column ff
+tlb_status launch_glu_rows(const float *z, int T, int ff, int ldz, int act, void *out, int ld, bool f32);
+// What a mixture of experts leaves per token: y = sum over the choice of weight * part[slot] + sigmoid(shared_gate) * shared.
+struct MoeRows {
+    int top = 0;
+    const int *slot = nullptr;            // [T][top] rows of part
+    const float *weight = nullptr, *part = nullptr, *shared = nullptr, *shared_gate = nullptr;
+    int ld_shared_gate = 0;
+};
+// Rows of the residual: x += norm(y * sigmoid(gate)) * (post_w + offset), both norms over `groups` parts; then, if norm_w is given,
+// out = norm(x) * (norm_w + offset) in the activation type.  y null and moe null: the second step alone.
+struct ResidNormJob {
+    float *x = nullptr;
+    int T = 0, width = 0, groups = 1;
+    float offset = 0.f, eps = 0.f;
+    const float *y = nullptr;             // [T, width]
+    const MoeRows *moe = nullptr;
+    const float *gate = nullptr;          // row 0; null: none
+    int ld_gate = 0;
+    const float *post_w = nullptr, *norm_w = nullptr;
+    void *out = nullptr;
+    int ldo = 0;
+};
+tlb_status launch_resid_norm_rows(const ResidNormJob &j, bool f32);
+// out [T, ld] = rows of n values at x, each over its root mean square, times w
+tlb_status launch_rms_cols(const float *x, int T, int n, int ldx, const float *w, float eps, void *out, int ld, bool f32);
+
+// ---------------------------------------------------------------- moe.cu
+// The choice of T tokens and the order their rows take behind one another, expert by expert.
+struct MoePlan {
+    int *sel = nullptr, *place = nullptr;   // [T][top]: expert; row within the expert's part, then the row over all experts
+    float *weight = nullptr;                // [T][top]
+    int *count = nullptr;                   // [2 * experts]: rows per expert, first row
+    int4 *tiles = nullptr;                  // (expert, first row, rows, 0), moe_max_tiles of them; rows 0: nothing to do
+};
+int moe_tile_rows(const RouteDesc &r, int T, bool f32);
+int moe_max_tiles(const RouteDesc &r, int T, bool f32);
+tlb_status launch_moe_plan(const RouteDesc &r, const float *logits, int ldl, int T, const MoePlan &p, bool f32);
+// rows of act (pitch ld, activation type) to the places of their choices
+tlb_status launch_moe_gather(const RouteDesc &r, const MoePlan &p, const void *act, int T, int ld, void *out, bool f32);
 
 // ---------------------------------------------------------------- mix_attention.cu
 // Softmax attention with optional window, per-head bias by distance and sink.
@@ -69,6 +156,8 @@ struct MixAttn {
     // rows of projections: q at column 0, k at H * D, v at H * D + KVH * D
     const float *proj;
     int ldp;
+    const float *gate;                    // prompts: [T, ld_gate] logits of a gate on every output element, or null
+    int ld_gate;
 };
 // One new token per sequence (rows of proj), at *pos: append and attend.  out: rows of H * DV in the activation type (out_f32: f32), pitch ldo.
 struct MixAttnDecode {
@@ -85,6 +174,7 @@ size_t mix_attn_decode_partial_floats(const MixAttn &a, int batch);
 tlb_status launch_mix_attn_decode(const MixAttnDecode &j);
 // T tokens of sequence seq at rows pos0 ..: append, then attend.
 tlb_status launch_mix_attn_prefill(const MixAttn &a, int seq, int T, int pos0, void *out, int ldo, bool f32);
+tlb_status launch_mix_attn_prompt(const MixAttn &a, int seq, int T, int pos0, void *out, int ldo, bool f32);      // rows already appended
 bool mix_attn_supported(int D, int DV);
 tlb_status launch_mix_attn_prefill_tc(const MixAttn &a, int seq, int T, int pos0, void *out, int ldo);   // mix_attention_tc.cu: f16 cache
 bool mix_attn_prefill_tc_supported(int D, int DV);
@@ -128,6 +218,62 @@ int scan_look_ld(int T);
 tlb_status launch_delta_prefill(const MixRecur &m, int seq, int T, int pos0, float *decay, float2 *look, float *o, void *out, int ldo, bool f32);
 // tanh of the first step of the decay's projection as two activation-type terms (value and remainder): out [T, 2 * ldh]
 tlb_status launch_tanh_split(const float *x, int T, int rank, int ldx, void *out, int ldh, bool f32);
+
+// ---------------------------------------------------------------- mix_latent.cu
+// Latent attention: the cache holds, per token, a normed latent of R values and one rotated key part of RD values that all heads
+// share (row pitch ld).  Keys and values of a head are W_uk c and W_uv c.  Rows of queries are attended in the latent space: W_uk goes
+// to the query, W_uv to the weighted sum of latents; long portions of a prompt expand the visible keys and values instead.
+struct MixLatent {
+    int H, D, RD, DV, R, ld;              // D: unrotated dimensions of a head's query, which is [D | RD]
+    int max_seq, window;
+    float scale, eps;
+    int rot;                              // leading dimensions of the RD that turn, in pairs of neighbours
+    const float *rot_cos, *rot_sin;       // [position][rot / 2]
+    const float *c_norm;                  // [R]
+    DenseW uk, uv;                        // [H * D, R], [H * DV, R] bf16
+    DenseW uk16, uv16;                    // the same as f16 (16-bit sessions)
+    void *cache;                          // [seq][max_seq][ld], f32 or f16
+    size_t seq_stride;
+    float *q;                             // rows of queries [H][D + RD], pitch ldq
+    int ldq;
+    const float *kv;                      // rows of W_dkv h [R + RD], pitch ldkv
+    int ldkv;
+    const float *gate;                    // rows of H * DV logits, pitch ld_gate, or null
+    int ld_gate;
+};
+// `rows` queries, each the newest token of its sequence or of those before it in a portion: row i of sequence seq0 + i * seq_step at
+// position pos[i] (or pos0 + i), angles of rope_pos[i] (or rope0 + i * rope_step).  Appends, attends, writes gated rows [H * DV].
+struct MixLatentRows {
+    MixLatent m;
+    int rows, seq0, seq_step;
+    const int *pos, *rope_pos;
+    int pos0, rope0, rope_step;
+    void *qa;                             // scratch: rows * H * ld activations of the cache type
+    float *partial;                       // scratch: latent_partial_floats
+    void *out;
+    int ldo;
+    bool f32, out_f32, pdl;               // f32: cache and scores' operands
+};
+size_t latent_partial_floats(const MixLatent &m, int rows);
+tlb_status launch_latent_rows(const MixLatentRows &j);
+bool latent_supported(const MixLatent &m, bool f32);
+int latent_ld(int R, int RD);
+// portions with at least this many tokens expand keys and values
+bool latent_expands(const MixLatent &m, int T);
+tlb_status launch_latent_prompt(const MixLatent &m, int seq, int T, int pos0, int rope0, int rope_step, void *out, int ldo, bool f32);
+
+// ---------------------------------------------------------------- mix_gru.cu
+// Gated recurrence per channel, S <- (1 - z) S + z candidate(u); rows z | u | gate logits, each `width` wide; out = S * silu(gate).
+// The state of a sequence at position p lies at state + (p & 1) * parity_stride.
+struct MixGru {
+    int width;
+    float *state;                         // [2][seq][width]
+    size_t parity_stride;
+    const float *proj;
+    int ldp;
+};
+tlb_status launch_gru_rows(const MixGru &m, int batch, const int *pos, void *out, int ldo, bool f32);
+tlb_status launch_gru_prefill(const MixGru &m, int seq, int T, int pos0, void *out, int ldo, bool f32);
 
 // launch with programmatic dependent launch (the kernel calls griddepcontrol.wait before it touches what precedes it)
 template <typename... KArgs, typename... Args>

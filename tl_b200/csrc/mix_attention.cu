@@ -7,6 +7,7 @@
 // score(i, j) = q_i . k_j * scale - bias[i - j];   weights = exp(score) / (sum exp(score) + exp(sink)).
 #include <algorithm>
 
+#include "act.cuh"
 #include "layered_kernels.h"
 #include "qmv_common.cuh"
 
@@ -336,9 +337,12 @@ __global__ void __launch_bounds__(kRowWarps * 32) mix_attn_rows_kernel(const Mix
         }
     }
     const float inv = 1.f / l;
+    const float *gate = a.gate ? a.gate + (size_t)t * a.ld_gate + (size_t)h * a.DV : nullptr;
 #pragma unroll
-    for (int i = 0; i < kMaxHeadDim / 32; i++)
-        if (lane + 32 * i < a.DV) store_act(out + (size_t)t * ldo + (size_t)h * a.DV + lane + 32 * i, o[i] * inv);
+    for (int i = 0; i < kMaxHeadDim / 32; i++) {
+        const int d = lane + 32 * i;
+        if (d < a.DV) store_act(out + (size_t)t * ldo + (size_t)h * a.DV + d, gate ? o[i] * inv * sigmoidf(gate[d]) : o[i] * inv);
+    }
 }
 
 int decode_splits(const MixAttn &a) { return (std::min(a.window, a.max_seq) + kDecKeys - 1) / kDecKeys; }
@@ -380,6 +384,12 @@ tlb_status launch_mix_attn_prefill(const MixAttn &a, int seq, int T, int pos0, v
     else mix_attn_append_kernel<__half><<<T, 256, 0, c->stream>>>(a, seq, pos0);
     count_launch();
     TLB_CUDA(cudaGetLastError());
+    return launch_mix_attn_prompt(a, seq, T, pos0, out, ldo, f32);
+}
+
+tlb_status launch_mix_attn_prompt(const MixAttn &a, int seq, int T, int pos0, void *out, int ldo, bool f32)
+{
+    Context *c = ctx();
     if (!f32 && mix_attn_prefill_tc5_supported(a.D, a.DV, T)) return launch_mix_attn_prefill_tc5(a, seq, T, pos0, out, ldo);
     if (!f32 && mix_attn_prefill_tc_supported(a.D, a.DV)) return launch_mix_attn_prefill_tc(a, seq, T, pos0, out, ldo);
     const dim3 grid((T + kRowWarps - 1) / kRowWarps, a.H);

@@ -5,6 +5,7 @@
 // The bias is a table by distance; a tile needs 127 consecutive entries of it, staged beside the keys.
 #include <algorithm>
 
+#include "act.cuh"
 #include "layered_kernels.h"
 #include "qmv_common.cuh"
 
@@ -217,7 +218,10 @@ mix_attn_tc_kernel(const MixAttn a, int seq, int T, int pos0, __nv_bfloat16 *__r
 #pragma unroll
             for (int e = 0; e < 2; e++) {
                 const int d = nb * 8 + 2 * c + e;
-                if (d < a.DV) dst[d] = __float2bfloat16_rn(o[nb][2 * r + e] * inv);
+                if (d >= a.DV) continue;
+                float v = o[nb][2 * r + e] * inv;
+                if (a.gate) v *= sigmoidf(a.gate[(size_t)row * a.ld_gate + (size_t)h * a.DV + d]);
+                dst[d] = __float2bfloat16_rn(v);
             }
         }
     }

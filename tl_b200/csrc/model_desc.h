@@ -14,6 +14,14 @@ enum class MixerKind {
     Attention,      // softmax attention over a KV cache
     Retention,      // linear attention with a fixed decay per head
     GeneralDelta,   // generalised delta rule: decay per key channel, removal along the unit key
+    Latent,         // softmax attention over a cache of latents and one shared rotated key part per token
+    MinGru,         // gated recurrence per channel whose gates read only the current token
+};
+
+// Slower angles for pairs that turn seldom within `original` positions (YaRN); factor 0: none.
+struct RotScaling {
+    double factor = 0.0, original = 0.0, fast = 0.0, slow = 0.0;
+    bool operator==(const RotScaling &o) const { return factor == o.factor && original == o.original && fast == o.fast && slow == o.slow; }
 };
 
 struct MixerDesc {
@@ -25,25 +33,40 @@ struct MixerDesc {
     bool qkv_bias = false;      // q, k, v projections have biases
     bool log_distance_bias = false;   // score -= r1[h] * ln(1 + r2[h] * distance)
     bool sink = false;          // exp(sink[h]) joins the softmax denominator
-    // Retention
-    int rot_dims = 0;           // leading dimensions of q and k that are rotated (rotate-half pairs); 0: none
+    // Retention (rotate-half pairs), Latent (pairs of neighbours)
+    int rot_dims = 0;           // leading dimensions of q and k (Latent: of the rotated part) that turn; 0: none
     double rot_base = 0.0;
-    std::vector<float> decay;   // per head
+    RotScaling rot_scaling;
+    std::vector<float> decay;   // Retention: per head
     // GeneralDelta
     int rank = 0;               // inner size of the decay's two-step projection (from the tensor's shape)
+    // Latent: `dim` unrotated and `rot_dim` shared rotated key dimensions; also scale and window above
+    int rot_dim = 0, kv_rank = 0;
+    int q_rank = 0;             // size of the latent the queries go through; 0: projected directly
+    bool out_gate = false;      // every output element times a sigmoid of a projection
+    // MinGru
+    int width = 0;
 };
 
-enum class FfnAct { PolyNorm };
+enum class FfnAct { PolyNorm, SiluGlu, GeluTanhGlu };
 
 struct FfnDesc {
-    int ff = 0;                 // 0: the layer has no feed-forward
+    int ff = 0;                 // 0: the layer has no feed-forward; mixture of experts: of one expert
     FfnAct act = FfnAct::PolyNorm;
+    // mixture of experts
+    int experts = 0;            // 0: dense
+    int top = 0, groups = 1, keep = 1;
+    float router_scale = 1.f;
+    int shared_ff = 0;          // 0: no shared expert
 };
 
 struct LayerDesc {
     MixerDesc mix;
     FfnDesc ffn;
     bool layer_scale = false;   // per-channel factors on what the mixer and the feed-forward add to the residual
+    bool post_norm = false;     // a second norm on what the mixer and the feed-forward add
+    bool resid_gate = false;    // ... which is first multiplied by a sigmoid of a projection of the sublayer's input
+    int weights_of = -1;        // the layer whose tensors this one uses (with a cache or state of its own)
 };
 
 struct ModelDesc {
@@ -51,6 +74,8 @@ struct ModelDesc {
     int vocab = 0, width = 0;
     float eps = 0.f;
     float norm_offset = 0.f;    // added to the stored weight of the width norms (1: stored around zero)
+    int norm_groups = 1;        // equal parts of the width, each over its own root mean square
+    float logit_softcap = 0.f;  // > 0: logits go through cap * tanh(. / cap)
     std::vector<LayerDesc> layers;
 };
 

@@ -16,12 +16,13 @@
 // Warp roles: 0-3 softmax / write-out, 4 TMA (lane 0), 5 MMA issue (lane 0) and tensor-memory allocation.
 // The MIX form serves the attention of layered models (launch_mix_attn_prefill_tc5): a sliding window (only tiles with a visible
 // key are visited), a bias by distance taken off the scores (consecutive table entries per tile, staged in shared memory), a sink in
-// the denominator, head sizes up to 128 (zero-filled to 128 by TMA), and weights kept in 32 bits: P goes into tensor memory as
-// two f16 terms, value and remainder, and P V is the sum of both products.
+// the denominator, an output gate, key sizes up to 192 and value sizes up to 128 (zero-filled to whole 64-column boxes by TMA), and
+// weights kept in 32 bits: P goes into tensor memory as two f16 terms, value and remainder, and P V is the sum of both products.
 // Every mbarrier wait is bounded (qmv_common.cuh: mbar_wait): when one runs out the CTA sets the context's error word,
 // lets its copies land, frees its tensor memory and returns.
 #include <algorithm>
 
+#include "act.cuh"
 #include "layered_kernels.h"
 #include "tc05.cuh"
 
@@ -33,6 +34,8 @@ constexpr int kAtQ = 128, kAtK = 128, kAtD = 128;
 constexpr int kAtThreads = 192;
 constexpr int kBoxBytes = 128 * 128;            // one TMA box: 128 rows x 64 f16
 constexpr int kTileBytes = 2 * kBoxBytes;       // a 128 x 128 f16 operand = two boxes
+// shared memory: Q, two stages of K (KB boxes each) and of V^T, barriers, alignment
+constexpr size_t at_smem_bytes(int KB) { return (size_t)(3 * KB + 4) * kBoxBytes + 1024 + 128; }
 // tensor memory columns
 constexpr uint32_t kColS = 0, kColO = 256, kColP = 384, kColPRest = 448;
 
@@ -45,6 +48,8 @@ struct AtParams {
     int DV, ldo, window, bias_n, vt_first;    // vt_first: the key V^T's column 0 holds
     const float *bias, *sink;
     __nv_bfloat16 *out16;  // [T, ldo], head h at column h * DV
+    const float *gate;     // [T, ld_gate] logits, or null
+    int ld_gate;
 };
 constexpr float kLog2eAt = 1.4426950408889634f;
 
@@ -60,7 +65,8 @@ __device__ __forceinline__ uint32_t pack_h2(float a, float b)
     return *reinterpret_cast<uint32_t *>(&h);
 }
 
-template <bool MIX>
+// KB: 64-column boxes of a query or key row
+template <bool MIX, int KB>
 __global__ void __launch_bounds__(kAtThreads, 1)
 prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_constant__ CUtensorMap kmap,
                             const __grid_constant__ CUtensorMap vtmap, const AtParams p)
@@ -71,7 +77,8 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __gr
     volatile int *abort_flag = &abort_word;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const uint32_t base = (smem_u32(at_smem) + 1023u) & ~1023u;
-    const uint32_t sQ = base, sK = base + kTileBytes, sV = sK + 2 * kTileBytes;     // K and V^T: two stages each
+    constexpr uint32_t kKeyBytes = KB * kBoxBytes;
+    const uint32_t sQ = base, sK = base + kKeyBytes, sV = sK + 2 * kKeyBytes;       // K and V^T: two stages each
     const uint32_t bars = sV + 2 * kTileBytes;
     const uint32_t q_full = bars, kv_full = bars + 8, kv_empty = bars + 24, s_full = bars + 40, p_full = bars + 56, o_full = bars + 64;
 
@@ -202,6 +209,12 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __gr
                 if constexpr (MIX) {
                     if (q < p.T) {
                         __nv_bfloat16 *d16 = p.out16 + (size_t)q * p.ldo + (size_t)h * p.DV + c * 32;
+                        if (p.gate) {
+                            const float *gt = p.gate + (size_t)q * p.ld_gate + (size_t)h * p.DV + c * 32;
+#pragma unroll
+                            for (int i = 0; i < 32; i++)
+                                if (c * 32 + i < p.DV) o[i] = __float_as_uint(__uint_as_float(o[i]) * sigmoidf(gt[i]));
+                        }
                         if (p.DV % 8 == 0 && p.ldo % 8 == 0) {
 #pragma unroll
                             for (int i = 0; i < 32; i += 8) {
@@ -231,17 +244,17 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __gr
     } else if (warp == 4) {
         // ------------------------------------------------ TMA: Q once, then K and V^T tiles two ahead
         if (lane == 0) {
-            mbar_expect_tx(q_full, kTileBytes);
-            tma_load_2d(sQ, &qmap, h * kAtD, q0, q_full);
-            tma_load_2d(sQ + kBoxBytes, &qmap, h * kAtD + 64, q0, q_full);
+            mbar_expect_tx(q_full, kKeyBytes);
+#pragma unroll
+            for (int j = 0; j < KB; j++) tma_load_2d(sQ + j * kBoxBytes, &qmap, (h * KB + j) * 64, q0, q_full);
             int issued = 0;
             for (int t = 0; t < n_tiles; t++) {
                 const int st = t & 1;
                 if (t >= 2 && !mbar_wait(kv_empty + 8 * st, (uint32_t)((t - 2) >> 1) & 1u, abort_flag, p.err, 44)) break;
-                mbar_expect_tx(kv_full + 8 * st, 2 * kTileBytes);
+                mbar_expect_tx(kv_full + 8 * st, kKeyBytes + kTileBytes);
                 const int key0 = (tile0 + t) * kAtK, vt0 = MIX ? p.vt_first : 0;
-                tma_load_2d(sK + st * kTileBytes, &kmap, 0, kvh * p.max_seq + key0, kv_full + 8 * st);
-                tma_load_2d(sK + st * kTileBytes + kBoxBytes, &kmap, 64, kvh * p.max_seq + key0, kv_full + 8 * st);
+#pragma unroll
+                for (int j = 0; j < KB; j++) tma_load_2d(sK + st * kKeyBytes + j * kBoxBytes, &kmap, j * 64, kvh * p.max_seq + key0, kv_full + 8 * st);
                 tma_load_2d(sV + st * kTileBytes, &vtmap, key0 - vt0, kvh * kAtD, kv_full + 8 * st);
                 tma_load_2d(sV + st * kTileBytes + kBoxBytes, &vtmap, key0 - vt0 + 64, kvh * kAtD, kv_full + 8 * st);
                 issued = t + 1;
@@ -261,8 +274,8 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __gr
                 if (!mbar_wait(kv_full + 8 * st, (uint32_t)(t >> 1) & 1u, abort_flag, p.err, 46)) return false;
                 tc_fence_after();
 #pragma unroll
-                for (int j = 0; j < 2; j++) {
-                    const uint64_t ad = smem_desc_sw128(sQ + j * kBoxBytes), bd = smem_desc_sw128(sK + st * kTileBytes + j * kBoxBytes);
+                for (int j = 0; j < KB; j++) {
+                    const uint64_t ad = smem_desc_sw128(sQ + j * kBoxBytes), bd = smem_desc_sw128(sK + st * kKeyBytes + j * kBoxBytes);
 #pragma unroll
                     for (int k16 = 0; k16 < 4; k16++) umma_f16_ss(tmem + kColS + (uint32_t)(st * 128), ad + 2u * k16, bd + 2u * k16, idesc, (j | k16) != 0);
                 }
@@ -332,15 +345,16 @@ __global__ void __launch_bounds__(256) v_transpose_kernel(const __half *__restri
         if (k0 + tx < keys_ld) dst[(size_t)(d0 + j) * keys_ld + k0 + tx] = tile[tx][j];
 }
 
-// queries of the projection rows as f16, every head padded to 128 columns
+// queries of the projection rows as f16, every head padded to QD columns
+template <int QD>
 __global__ void __launch_bounds__(256) mix_q_to_f16_kernel(const float *__restrict__ proj, int ldp, int H, int D, __half *__restrict__ qh)
 {
     const float *row = proj + (size_t)blockIdx.x * ldp;
-    for (int i = threadIdx.x; i < H * kAtD / 2; i += blockDim.x) {
-        const int h = i / (kAtD / 2), d = (i % (kAtD / 2)) * 2;
+    for (int i = threadIdx.x; i < H * QD / 2; i += blockDim.x) {
+        const int h = i / (QD / 2), d = (i % (QD / 2)) * 2;
         const float *q = row + (size_t)h * D + d;
         const float a = d < D ? q[0] : 0.f, b = d + 1 < D ? q[1] : 0.f;
-        reinterpret_cast<uint32_t *>(qh)[(size_t)blockIdx.x * (H * kAtD / 2) + i] = pack_h2(fminf(fmaxf(a, -65504.f), 65504.f), fminf(fmaxf(b, -65504.f), 65504.f));
+        reinterpret_cast<uint32_t *>(qh)[(size_t)blockIdx.x * (H * QD / 2) + i] = pack_h2(fminf(fmaxf(a, -65504.f), 65504.f), fminf(fmaxf(b, -65504.f), 65504.f));
     }
 }
 // cache rows key_first .. of V as V^T [KV head][128][keys_ld] (columns counted from key_first, rows past DV zero)
@@ -361,25 +375,27 @@ __global__ void __launch_bounds__(256) mix_v_transpose_kernel(const __half *__re
 }  // namespace
 
 // Head sizes that fill most of the 128 columns, and enough queries for a tile.
-bool mix_attn_prefill_tc5_supported(int D, int DV, int T) { return std::max(D, DV) > 64 && D <= kAtD && DV <= kAtD && T >= 64; }
+bool mix_attn_prefill_tc5_supported(int D, int DV, int T) { return std::max(D, DV) > 64 && D <= 192 && DV <= kAtD && T >= 64; }
 
-// MixAttn over an f16 cache: T tokens of sequence seq whose rows are in the cache already.
-tlb_status launch_mix_attn_prefill_tc5(const MixAttn &a, int seq, int T, int pos0, void *out, int ldo)
+namespace {
+
+template <int KB>
+tlb_status run_mix_tc5(const MixAttn &a, int seq, int T, int pos0, void *out, int ldo)
 {
     Context *c = ctx();
-    if (!c) return TLB_ERR_DEVICE;
+    constexpr int QD = KB * 64;
     // cache rows some query sees, from a tile border on
     const int key_first = std::max(0, pos0 - a.window + 1) / kAtK * kAtK, n_keys = pos0 + T - key_first, keys_ld = (n_keys + 127) / 128 * 128;
-    Storage *qh = storage_alloc((size_t)T * a.H * kAtD * sizeof(__half));
+    Storage *qh = storage_alloc((size_t)T * a.H * QD * sizeof(__half));
     Storage *vt = storage_alloc((size_t)a.KVH * kAtD * keys_ld * sizeof(__half));
     if (!qh || !vt) { if (qh) storage_release(qh); if (vt) storage_release(vt); return TLB_ERR_ALLOC; }
     auto done = [&](tlb_status st) { storage_release(qh); storage_release(vt); return st; };
     const __half *kc = (const __half *)a.kcache + (size_t)seq * a.seq_stride_k, *vc = (const __half *)a.vcache + (size_t)seq * a.seq_stride_v;
-    mix_q_to_f16_kernel<<<T, 256, 0, c->stream>>>(a.proj, a.ldp, a.H, a.D, (__half *)qh->ptr);
+    mix_q_to_f16_kernel<QD><<<T, 256, 0, c->stream>>>(a.proj, a.ldp, a.H, a.D, (__half *)qh->ptr);
     mix_v_transpose_kernel<<<dim3(kAtD / 32, (unsigned)(keys_ld / 32), (unsigned)a.KVH), 256, 0, c->stream>>>(vc, (__half *)vt->ptr, a.max_seq, a.ldv, key_first, n_keys, keys_ld);
     count_launch(2);
     CUtensorMap qmap, kmap, vtmap;
-    if (!encode_f16_map(&qmap, qh->ptr, (uint64_t)a.H * kAtD, (uint64_t)T, (uint64_t)a.H * kAtD * 2, 64, 128) ||
+    if (!encode_f16_map(&qmap, qh->ptr, (uint64_t)a.H * QD, (uint64_t)T, (uint64_t)a.H * QD * 2, 64, 128) ||
         !encode_f16_map(&kmap, kc, (uint64_t)a.ldk, (uint64_t)a.KVH * a.max_seq, (uint64_t)a.ldk * 2, 64, 128) ||
         !encode_f16_map(&vtmap, vt->ptr, (uint64_t)keys_ld, (uint64_t)a.KVH * kAtD, (uint64_t)keys_ld * 2, 64, 128))
         return done(fail(TLB_ERR_DEVICE, "prompt attention: cuTensorMapEncodeTiled failed or is not available"));
@@ -389,18 +405,28 @@ tlb_status launch_mix_attn_prefill_tc5(const MixAttn &a, int seq, int T, int pos
     p.err = c->err_flag;
     p.DV = a.DV; p.ldo = ldo; p.window = a.window; p.bias_n = a.bias_n; p.bias = a.bias; p.sink = a.sink; p.out16 = (__nv_bfloat16 *)out;
     p.vt_first = key_first;
-    const size_t smem = (size_t)5 * kTileBytes + 1024 + 128;
+    p.gate = a.gate; p.ld_gate = a.ld_gate;
+    constexpr size_t smem = at_smem_bytes(KB);
     static bool attr_set = false;
     if (!attr_set) {
-        cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<true, KB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return done(cuda_fail(e, "prompt attention attribute"));
         attr_set = true;
     }
-    prefill_attention_tc_kernel<true><<<dim3((unsigned)((T + kAtQ - 1) / kAtQ), (unsigned)a.H), kAtThreads, smem, c->stream>>>(qmap, kmap, vtmap, p);
+    prefill_attention_tc_kernel<true, KB><<<dim3((unsigned)((T + kAtQ - 1) / kAtQ), (unsigned)a.H), kAtThreads, smem, c->stream>>>(qmap, kmap, vtmap, p);
     count_launch();
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return done(cuda_fail(e, "prompt attention launch"));
     return done(TLB_OK);
+}
+
+}  // namespace
+
+// MixAttn over an f16 cache: T tokens of sequence seq whose rows are in the cache already.
+tlb_status launch_mix_attn_prefill_tc5(const MixAttn &a, int seq, int T, int pos0, void *out, int ldo)
+{
+    if (!ctx()) return TLB_ERR_DEVICE;
+    return a.D > 128 ? run_mix_tc5<3>(a, seq, T, pos0, out, ldo) : run_mix_tc5<2>(a, seq, T, pos0, out, ldo);
 }
 
 bool prefill_attention_tc_supported(int D, int kv_f16, int n_tokens) { return D == 128 && kv_f16 && n_tokens >= 64; }
@@ -429,15 +455,15 @@ tlb_status launch_prefill_attention_tc(const float *q, const void *kcache, const
     p.out = out; p.T = T; p.H = H; p.KVH = KVH; p.max_seq = max_seq; p.pos0 = pos0; p.vt_rows = keys_ld;
     p.scale2 = scale * 1.4426950408889634f;
     p.err = c->err_flag;
-    const size_t smem = (size_t)5 * kTileBytes + 1024 + 128;
+    constexpr size_t smem = at_smem_bytes(2);
     static bool attr_set = false;
     if (!attr_set) {
-        cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<false, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return done(cuda_fail(e, "prompt attention attribute"));
         attr_set = true;
     }
     dim3 grid((unsigned)((T + kAtQ - 1) / kAtQ), (unsigned)H);
-    prefill_attention_tc_kernel<false><<<grid, kAtThreads, smem, c->stream>>>(qmap, kmap, vtmap, p);
+    prefill_attention_tc_kernel<false, 2><<<grid, kAtThreads, smem, c->stream>>>(qmap, kmap, vtmap, p);
     count_launch();
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return done(cuda_fail(e, "prompt attention launch"));
