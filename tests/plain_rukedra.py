@@ -67,6 +67,16 @@ def choose_experts(logits, top, groups, keep, scale):
     return pick, s[pick] / (np.sum(s[pick]) + 1e-20) * scale
 
 
+def choice_margin(logits, top, groups, keep):
+    """How far a token is from another choice: the gap behind the last group kept and the last expert chosen."""
+    s = sigmoid(logits)
+    parts = np.sort(s.reshape(groups, -1), axis=1)
+    g = np.sort(parts[:, -2:].sum(axis=1))[::-1]
+    kept = np.argsort(-parts[:, -2:].sum(axis=1), kind="stable")[:keep]
+    e = np.sort(s.reshape(groups, -1)[kept].reshape(-1))[::-1]
+    return min(g[keep - 1] - g[keep] if keep < groups else 1.0, e[top - 1] - e[top] if top < len(e) else 1.0)
+
+
 def gated(W, p, h, act):
     return W[p + "down"] @ (act(W[p + "gate"] @ h) * (W[p + "up"] @ h))
 
@@ -76,6 +86,7 @@ class PlainRukedra:
         self.cfg = cfg
         self.w = {k: np.asarray(v, dtype=np.float64) for k, v in weights.items()}
         self.eps, self.groups = cfg["norm"]["eps"], cfg["norm"]["groups"]
+        self.margins = []                   # of every choice of experts made so far
 
     def new_state(self):
         return {"pos": 0, "layers": [dict() for _ in self.cfg["layers"]]}
@@ -115,7 +126,10 @@ class PlainRukedra:
         if m["kind"] == "dense":
             return gated(self.w, p, h, gelu_tanh)
         r = m["router"]
-        pick, weight = choose_experts(self.w[p + "router"] @ h, r["top"], r["groups"]["count"], r["groups"]["keep"], r["scale"])
+        groups = r.get("groups") or {"count": 1, "keep": 1}
+        z = self.w[p + "router"] @ h
+        self.margins.append(choice_margin(z, r["top"], groups["count"], groups["keep"]))
+        pick, weight = choose_experts(z, r["top"], groups["count"], groups["keep"], r["scale"])
         y = sum(w * gated(self.w, "%se%d." % (p, e), h, silu) for e, w in zip(pick, weight))
         if m.get("shared"):
             y = y + sigmoid(self.w[p + "shared.sg"] @ h) * gated(self.w, p + "shared.", h, silu)
@@ -141,8 +155,9 @@ class PlainRukedra:
             if layers_out is not None:
                 layers_out[i].append(x)
         state["pos"] += 1
-        cap = self.cfg["logit_softcap"]
-        return cap * np.tanh(self.w["head"] @ self.norm(x, "final.norm") / cap)
+        logits = self.w["head"] @ self.norm(x, "final.norm")
+        cap = self.cfg.get("logit_softcap")
+        return cap * np.tanh(logits / cap) if cap else logits
 
     def forward(self, tokens, state, layers_out=None):
         return np.stack([self.token(int(t), state, layers_out) for t in tokens])

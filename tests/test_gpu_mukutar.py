@@ -7,8 +7,10 @@ import json
 import numpy as np
 import pytest
 
+import layered_session as S
 import plain_layers as P
 import tl_b200 as tl
+from layered_session import decode, err, greedy, run_portions, toks
 from tl_b200 import synth
 
 pytestmark = pytest.mark.gpu
@@ -40,59 +42,16 @@ def config(layers, width=72, ff=100, vocab=131, eps=1e-5, mlps=None):
 MIXED = [retention(), attention(), delta(), attention(heads=4, kv=1, dim=40, vdim=24, window=70), retention(heads=2, dim=40, vdim=16, dims=40), delta(heads=2, dim=64)]
 
 
-class Model:
+class Model(S.Model):
     def __init__(self, cfg, seed=1, rank=11, edit=None):
-        self.cfg = cfg
-        vals = {n: synth.mukutar_tensor(n, s, seed) for n, s in synth.mukutar_specs(cfg, rank).items()}
-        if edit:
-            edit(vals)
-        self.bits = {n: synth.to_bf16(v) for n, v in vals.items()}
-        self.plain = P.Plain(cfg, {n: synth.from_bf16(b) for n, b in self.bits.items()})
-        self.map = tl.TensorMap.new()
-        for n, b in self.bits.items():
-            self.map.add(n, synth.BF16, b.shape, b)
-        self.map.set_config(json.dumps(cfg))
-
-    def dec(self, f32, max_seq=256, **kw):
-        return tl.Decoder(None, self.map, max_seq=max_seq, f32=f32, **kw)
-
-    def ref(self, tokens):
-        return self.plain.forward(tokens, self.plain.new_state())
-
-
-def toks(n, vocab=131, seed=0):
-    return [int(t) for t in np.random.default_rng(seed).integers(0, vocab, n)]
-
-
-def err(a, b):
-    a, b = np.atleast_2d(a), np.atleast_2d(b)
-    d = a - b
-    return float(np.max(np.sqrt(np.mean(d * d, axis=1)) / np.sqrt(np.mean(b * b))))
+        super().__init__(cfg, synth.mukutar_specs(cfg, rank), synth.mukutar_tensor, P.Plain, seed, edit)
 
 
 def close(a, b, f32):
     """Every row within the tolerance; with bf16 operands all but 3 % of them (at least one): a head's output over its own root mean
     square jumps where it crosses zero - on a sequence's first token it is little more than the sign of one dot product."""
-    d = np.atleast_2d(a) - np.atleast_2d(b)
-    e = np.sqrt(np.mean(d * d, axis=1)) / np.sqrt(np.mean(np.square(b)))
+    e = S.row_errors(a, b)
     return int(np.sum(e >= TOL[f32])) <= (0 if f32 else max(1, int(0.03 * len(e))))
-
-
-def decode(d, tokens, pos):
-    out = []
-    for i, t in enumerate(tokens):
-        d.step(t, pos + i, read=False)
-        out.append(d.logits())
-    return np.stack(out)
-
-
-def run_portions(d, tokens, sizes, seq=0):
-    out, at, i = [], 0, 0
-    while at < len(tokens):
-        n = min(sizes[i % len(sizes)], len(tokens) - at)
-        out.append(d.prefill_logits(tokens[at:at + n], at, seq=seq))
-        at, i = at + n, i + 1
-    return np.concatenate(out)
 
 
 # ---- mechanisms alone, at sizes that are multiples of nothing and at ones that coincide or are 1
@@ -336,18 +295,6 @@ def test_prompt_longer_than_a_chunk(f32):
 
 
 # ---- generation through the session's own entry points
-def greedy(m, prompt, n):
-    st = m.plain.new_state()
-    lg = m.plain.forward(prompt, st)[-1]
-    out, gaps = [], []
-    for _ in range(n):
-        top = np.sort(lg)[-2:]
-        gaps.append(top[1] - top[0])
-        out.append(int(np.argmax(lg)))
-        lg = m.plain.forward([out[-1]], st)[-1]
-    return out, min(gaps) / np.sqrt(np.mean(lg * lg))
-
-
 def test_greedy_generation():
     m = Model(config(MIXED), seed=15)
     prompt = toks(45, seed=5)

@@ -237,6 +237,63 @@ def mukutar_tensors(cfg, seed, rank=64):
     return {n: to_bf16(mukutar_tensor(n, s, seed)) for n, s in mukutar_specs(cfg, rank).items()}
 
 
+def rukedra_specs(cfg):
+    """Name -> shape of every tensor of a Rukedra model with this config.json."""
+    W = cfg["width"]
+    s = {"embed": (cfg["vocab"], W), "head": (cfg["vocab"], W), "final.norm": (W,)}
+
+    def gated(p, ff):
+        s[p + "gate"] = s[p + "up"] = (ff, W)
+        s[p + "down"] = (W, ff)
+
+    for i, lay in enumerate(cfg["layers"]):
+        if lay.get("weights_of") is not None:
+            continue
+        p, m = "l%d." % i, lay["mixer"]
+        q = p + "mix."
+        for n in ("1", "2") if lay.get("mlp") else ("1",):
+            s[p + "norm" + n] = s[p + "norm%sb" % n] = s[p + "rg%s.b" % n] = (W,)
+            s[p + "rg" + n] = (W, W)
+        if lay["type"] == "mingru":
+            D = m["width"]
+            s[q + "z"] = s[q + "x"] = s[q + "g"] = (D, W)
+            s[q + "z.b"] = s[q + "x.b"] = (D,)
+            s[q + "o"] = (W, D)
+        else:
+            H, hd, R = m["heads"], m["dim"] + m["rot_dim"], m["kv_rank"]
+            if lay["type"] == "latent_attention":
+                s[q + "dq"], s[q + "dq.norm"], s[q + "uq"] = (m["q_rank"], W), (m["q_rank"],), (H * hd, m["q_rank"])
+                s[q + "g"] = (H * m["vdim"], W)
+            else:
+                s[q + "q"] = (H * hd, W)
+            s[q + "dkv"], s[q + "dkv.norm"] = (R + m["rot_dim"], W), (R,)
+            s[q + "uk"], s[q + "uv"], s[q + "o"] = (H * m["dim"], R), (H * m["vdim"], R), (W, H * m["vdim"])
+        f = lay.get("mlp")
+        if f and f["kind"] == "dense":
+            gated(p + "mlp.", f["ff"])
+        elif f:
+            for e in range(f["router"]["experts"]):
+                gated(p + "mlp.e%d." % e, f["expert"]["ff"])
+            s[p + "mlp.router"] = (f["router"]["experts"], W)
+            if f.get("shared"):
+                gated(p + "mlp.shared.", f["shared"]["ff"])
+                s[p + "mlp.shared.sg"] = (1, W)
+    return s
+
+
+def rukedra_tensor(name, shape, seed):
+    """Seeded f32 values of one tensor, of a size a trained model's could have; rounded to bf16 they are the stored ones."""
+    x = _rng(seed, name).standard_normal(int(np.prod(shape)), dtype=np.float32).reshape(shape)
+    if len(shape) == 2:
+        return x if name == "embed" else x * np.float32((3.0 if name.endswith("router") else 1.0) * shape[1] ** -0.5)
+    return 0.5 * x if name.endswith(".b") else 1.0 + 0.2 * x
+
+
+def rukedra_tensors(cfg, seed):
+    """Name -> bf16 bits (uint16) of a whole model."""
+    return {n: to_bf16(rukedra_tensor(n, s, seed)) for n, s in rukedra_specs(cfg).items()}
+
+
 def write_model_dir(path, cfg, tensors):
     """A model folder: config.json and model.safetensors (bf16 bits as uint16, int32 and float32 arrays)."""
     import json
