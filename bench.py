@@ -20,8 +20,8 @@ are seeded synthetic GGUF blocks (no model file is needed or read).  Prints ONE 
 With N > 1 every rank decodes its own replica of the 8B model (no exchange step on this path): weak scaling; the
 headline stays that.  A `tp` object is added: the 70B-shaped model of config C4 split over the N ranks (tensor
 parallel, one process per GPU), its per-token all-reduce cost, and the same model on one GPU.
---workload c1 / c3 / qgemm / qrows / prefill-2layer / mukutar / mukutar-3layer run only that part (small cases for profiler captures
-among them; mukutar: the layered models of tl_b200/csrc/layered.cu beside a Llama model of the same sizes).
+--workload c1 / c3 / qgemm / qrows / prefill-2layer / mukutar / mukutar-3layer / rukedra / rukedra-3layer run only that part (small cases
+for profiler captures among them; mukutar, rukedra: the layered models of tl_b200/csrc/layered.cu beside a model of the same sizes).
 """
 import argparse
 import json
@@ -677,6 +677,8 @@ PARTS = {
     "per-op-4layer": "the TL chatbot's op sequence through the per-op entry points (native driver), Llama-3-8B shapes cut to 4 layers, 2048 cached rows, 3 steps",
     "mukutar": "Mukutar models (bf16 weights): decode and prompt throughput at two sizes, beside a Llama model (Q4_K) of the same sizes",
     "mukutar-3layer": "one layer of each mixer at width 4096 + head: a 2048-token prompt and 8 decode steps (small case for a launch list)",
+    "rukedra": "Rukedra models (bf16 weights): decode and prompt throughput at two sizes, beside a Mukutar model (bf16) of the same width, heads, layers and dense feed-forward",
+    "rukedra-3layer": "one layer of each Rukedra mixer (dense, expert and dense feed-forward) at width 4096 + head: a 2048-token prompt and 8 decode steps (small case for a launch list)",
     "prefill-2layer": "one 2048-token prompt through two Llama-3-8B-shaped layers + head, three times (small case for a profiler capture)",
 }
 
@@ -691,21 +693,50 @@ def mukutar_cfg(width, heads, kv_heads, ff, n_layers, vocab, window, dim=128):
             "layers": [{"type": order[i % 3], "mixer": mix[order[i % 3]], "mlp": {"kind": "dense", "ff": ff}} for i in range(n_layers)]}
 
 
-def build_mukutar_map(tl, cfg, seed=77):
+def rukedra_cfg(width, heads, ff, expert_ff, n_layers, vocab, window, q_rank, experts=64, top=6):
+    """Direct and windowed latent attention (heads of 128 + 64, latents of 512) and the gated recurrence in turn; dense and expert
+    feed-forwards by turns."""
+    scaling = dict(factor=8.0, original=4096, fast=32.0, slow=1.0)
+    lat = dict(heads=heads, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5, rot=dict(base=10000.0, dims=64, scaling=scaling))
+    mix = {"latent_attention_2": lat, "latent_attention": dict(lat, q_rank=q_rank, mask=dict(size=window)), "mingru": dict(width=width)}
+    order = ["latent_attention_2", "latent_attention", "mingru"]
+    ffn = [dict(kind="dense", ff=ff), dict(kind="moe", expert=dict(ff=expert_ff), shared=dict(ff=2 * expert_ff), router=dict(experts=experts, top=top, scale=2.5, groups=dict(count=8, keep=3)))]
+    return {"architecture": "Rukedra", "vocab": vocab, "width": width, "norm": {"eps": 1e-6, "groups": 2}, "logit_softcap": 30.0,
+            "layers": [{"type": order[i % 3], "mixer": mix[order[i % 3]], "mlp": ffn[i % 2]} for i in range(n_layers)]}
+
+
+def build_layered_map(tl, cfg, seed=77):
     """Seeded random weights; large matrices repeat a block of random values, generated once (the arithmetic does not depend on them)."""
     from tl_b200 import synth
     block = synth.to_bf16(np.random.default_rng(seed).standard_normal(1 << 22, dtype=np.float32))
     m = tl.TensorMap.new()
-    for name, shape in synth.mukutar_specs(cfg, rank=128).items():
+    specs, value = (synth.mukutar_specs(cfg, rank=128), synth.mukutar_tensor) if cfg["architecture"] == "Mukutar" else (synth.rukedra_specs(cfg), synth.rukedra_tensor)
+    for name, shape in specs.items():
         n = int(np.prod(shape))
         if n < block.size:
-            bits = synth.to_bf16(synth.mukutar_tensor(name, shape, seed))
+            bits = synth.to_bf16(value(name, shape, seed))
         else:
             scale = np.float32(1.0 if name == "embed" else shape[1] ** -0.5)
             bits = np.resize(synth.to_bf16(synth.from_bf16(block) * scale), n)
         m.add(name, synth.BF16, shape, bits)
     m.set_config(json.dumps(cfg))
     return m
+
+
+def layered_linear_flops(cfg):
+    """Multiply-adds times two of one token's linear layers (the chosen experts; not the head, nor the latents' expansion)."""
+    from tl_b200 import synth
+    specs = synth.mukutar_specs(cfg, rank=128) if cfg["architecture"] == "Mukutar" else synth.rukedra_specs(cfg)
+    total = 0.0
+    for name, shape in specs.items():
+        if len(shape) != 2 or name in ("embed", "head") or name.endswith((".mix.uk", ".mix.uv")):
+            continue
+        part = 1.0
+        if ".mlp.e" in name:
+            r = cfg["layers"][int(name[1:name.index(".")])]["mlp"]["router"]
+            part = r["top"] / r["experts"]
+        total += 2.0 * shape[0] * shape[1] * part
+    return total
 
 
 def time_events(tl, ev, fn, n):
@@ -719,40 +750,55 @@ def time_events(tl, ev, fn, n):
     return _elapsed_ms(tl, ev[0], ev[1]) / n
 
 
-def measure_mukutar(tl, ev, peaks, width, heads, kv_heads, ff, n_layers=6, vocab=32768, window=4096, prompt=2048, steps=32):
-    """Decode (batch 1, behind a prompt of `prompt` tokens) and prompt throughput of a Mukutar model, and of a Llama model of the same
-    width, heads, feed-forward size, layers and vocabulary (Q4_K, three feed-forward matrices against two).  Weights exceed L2."""
+def measure_session(tl, ev, peaks, dec, toks, lin, steps):
+    """Prompt and decode (batch 1, behind the prompt) throughput; lin: floating-point operations of a token's linear layers."""
+    prompt = len(toks)
+    for _ in range(3):
+        dec.prefill(toks, 0, read=False)
+    ms = time_events(tl, ev, lambda: dec.prefill(toks, 0, read=False), 5)
+    tf = lin * prompt / ms / 1e9
+    r = {"prefill_ms": round(ms, 3), "prefill_tokens_per_s": round(prompt / ms * 1e3), "prefill_linear_tflops": round(tf, 1), "prefill_frac_bf16": round(tf / peaks.get("bf16_tflops", 1590.0), 4)}
+    dec.generate(1, prompt, 8, read=False)
+    ms = time_events(tl, ev, lambda: dec.generate(1, prompt + 8, steps, read=False), 1) / steps
+    st = dec.stats(prompt + 8)
+    gbs = (st["weight_bytes"] + st["kv_bytes"]) / ms / 1e6
+    r.update({"decode_ms": round(ms, 4), "decode_tokens_per_s": round(1e3 / ms, 1), "decode_GBs": round(gbs, 1), "decode_frac_hbm": round(gbs / peaks["hbm_gbs"], 4),
+              "weight_MB": round(st["weight_bytes"] / 1e6, 1), "kernels_per_step": st["kernels_per_step"]})
+    return r
+
+
+def measure_layered(tl, ev, peaks, cfg, beside, shape, prompt=2048, steps=32):
+    """A layered model and the models beside it: (name, config of a layered model or of a Llama model in Q4_K).  Weights exceed L2."""
     from tl_b200 import synth
-    toks = [int(t) for t in np.random.default_rng(6).integers(0, vocab, prompt)]
-    out = {"width": width, "heads": heads, "kv_heads": kv_heads, "ff": ff, "layers": n_layers, "vocab": vocab, "window": window, "prompt": prompt}
-    cfg = mukutar_cfg(width, heads, kv_heads, ff, n_layers, vocab, window)
-    lcfg = dict(n_layers=n_layers, d_model=width, n_heads=heads, n_kv_heads=kv_heads, head_dim=128, ffn=ff, vocab=vocab, eps=1e-5, rope_base=10000.0, attn_scale=0.08839)
-    for name in ("mukutar", "llama_q4k"):
-        if name == "mukutar":
-            wmap = build_mukutar_map(tl, cfg)
+    toks = [int(t) for t in np.random.default_rng(6).integers(0, cfg["vocab"], prompt)]
+    out = dict(shape, layers=len(cfg["layers"]), vocab=cfg["vocab"], prompt=prompt)
+    for name, c in [(cfg["architecture"].lower(), cfg)] + beside:
+        if "architecture" in c:
+            wmap = build_layered_map(tl, c)
             dec = tl.Decoder(None, wmap, max_seq=prompt + 256)
-            per_kind = {"retention": 4, "general_delta": 5, "attention": 2}      # input matrices of heads * 128 rows (attention: q, and k | v)
-            lin = sum(2.0 * width * heads * 128 * (per_kind[l["type"]] + 1) + (4.0 * width * kv_heads * 128 - 2.0 * width * heads * 128 if l["type"] == "attention" else 0.0) + 4.0 * width * ff
-                      for l in cfg["layers"])
+            lin = layered_linear_flops(c)
         else:
-            wmap = tl.map_from_tensors(synth.llama_tensors(lcfg, 1, 12, 12))
-            dec = tl.Decoder(lcfg, wmap, kv_f16=True, max_seq=prompt + 256)
-            lin = n_layers * (2.0 * width * (2 * heads + 2 * kv_heads) * 128 + 6.0 * width * ff)
-        for _ in range(2):
-            dec.prefill(toks, 0, read=False)
-        ms = time_events(tl, ev, lambda: dec.prefill(toks, 0, read=False), 3)
-        tf = lin * prompt / ms / 1e9
-        r = {"prefill_ms": round(ms, 3), "prefill_tokens_per_s": round(prompt / ms * 1e3), "prefill_linear_tflops": round(tf, 1), "prefill_frac_bf16": round(tf / peaks.get("bf16_tflops", 1590.0), 4)}
-        dec.generate(1, prompt, 8, read=False)
-        ms = time_events(tl, ev, lambda: dec.generate(1, prompt + 8, steps, read=False), 1) / steps
-        st = dec.stats(prompt + 8)
-        gbs = (st["weight_bytes"] + st["kv_bytes"]) / ms / 1e6
-        r.update({"decode_ms": round(ms, 4), "decode_tokens_per_s": round(1e3 / ms, 1), "decode_GBs": round(gbs, 1), "decode_frac_hbm": round(gbs / peaks["hbm_gbs"], 4),
-                  "weight_MB": round(st["weight_bytes"] / 1e6, 1), "kernels_per_step": st["kernels_per_step"]})
-        out[name] = r
+            wmap = tl.map_from_tensors(synth.llama_tensors(c, 1, 12, 12))
+            dec = tl.Decoder(c, wmap, kv_f16=True, max_seq=prompt + 256)
+            lin = c["n_layers"] * (2.0 * c["d_model"] * (2 * c["n_heads"] + 2 * c["n_kv_heads"]) * 128 + 6.0 * c["d_model"] * c["ffn"])
+        out[name] = measure_session(tl, ev, peaks, dec, toks, lin, steps)
         dec.destroy()
         wmap.free()
     return out
+
+
+def measure_mukutar(tl, ev, peaks, width, heads, kv_heads, ff, n_layers=6, vocab=32768, window=4096):
+    """A Mukutar model, and a Llama model of the same width, heads, feed-forward size, layers and vocabulary (Q4_K, three feed-forward
+    matrices against two)."""
+    lcfg = dict(n_layers=n_layers, d_model=width, n_heads=heads, n_kv_heads=kv_heads, head_dim=128, ffn=ff, vocab=vocab, eps=1e-5, rope_base=10000.0, attn_scale=0.08839)
+    return measure_layered(tl, ev, peaks, mukutar_cfg(width, heads, kv_heads, ff, n_layers, vocab, window), [("llama_q4k", lcfg)],
+                           {"width": width, "heads": heads, "kv_heads": kv_heads, "ff": ff, "window": window})
+
+
+def measure_rukedra(tl, ev, peaks, width, heads, ff, expert_ff, q_rank, n_layers=6, vocab=32768, window=4096):
+    """A Rukedra model, and a Mukutar model of the same width, heads, layers, vocabulary and dense feed-forward size."""
+    return measure_layered(tl, ev, peaks, rukedra_cfg(width, heads, ff, expert_ff, n_layers, vocab, window, q_rank), [("mukutar", mukutar_cfg(width, heads, heads // 4, ff, n_layers, vocab, window))],
+                           {"width": width, "heads": heads, "ff": ff, "expert_ff": expert_ff, "experts": "6 of 64", "q_rank": q_rank, "kv_rank": 512, "window": window})
 
 
 def run_part(args):
@@ -832,8 +878,12 @@ def run_part(args):
         clk = ClockSampler(0)
         sizes = [measure_mukutar(tl, ev, peaks, 2048, 16, 4, 5632), measure_mukutar(tl, ev, peaks, 4096, 32, 8, 14336)]
         line.update({"sizes": sizes, "value": sizes[1]["mukutar"]["decode_tokens_per_s"], "unit": "tokens/s (width 4096, 6 layers + head, batch 1)", "higher_is_better": True, "clocks": clk.stop()})
-    elif name == "mukutar-3layer":
-        wmap = build_mukutar_map(tl, mukutar_cfg(4096, 32, 8, 14336, 3, 32768, 4096))
+    elif name == "rukedra":
+        clk = ClockSampler(0)
+        sizes = [measure_rukedra(tl, ev, peaks, 2048, 16, 5632, 1408, 1536), measure_rukedra(tl, ev, peaks, 4096, 32, 14336, 1792, 1536)]
+        line.update({"sizes": sizes, "value": sizes[1]["rukedra"]["decode_tokens_per_s"], "unit": "tokens/s (width 4096, 6 layers + head, batch 1)", "higher_is_better": True, "clocks": clk.stop()})
+    elif name in ("mukutar-3layer", "rukedra-3layer"):
+        wmap = build_layered_map(tl, mukutar_cfg(4096, 32, 8, 14336, 3, 32768, 4096) if name == "mukutar-3layer" else rukedra_cfg(4096, 32, 14336, 1792, 3, 32768, 4096, 1536))
         dec = tl.Decoder(None, wmap, max_seq=2304)
         toks = [int(t) for t in np.random.default_rng(6).integers(0, 32768, 2048)]
         for _ in range(2):
