@@ -411,7 +411,7 @@ def test_step_statistics():
     layer = [sum(size(n) for n in shapes if n.startswith("l%d." % i) and ".mlp.e" not in n) for i in (0, 1)]
     experts = f["router"]["top"] * 3 * f["expert"]["ff"] * W * 2
     assert st["weight_bytes"] == 2 * (layer[0] + experts) + layer[1] + (V + 1) * W * 2 + W * 4
-    assert st["kv_bytes"] == 2 * 19 * (44 + 12) * 2 + 2 * 52 * 4 and st["kernels_per_step"] == 9 + 2 + 9 + 1 + 1
+    assert st["kv_bytes"] == 2 * 19 * (44 + 12) * 2 + 2 * 52 * 4 and st["kernels_per_step"] == 9 + 3 + 9 + 1 + 1
 
 
 def test_model_folder_loads_to_the_same_model(tmp_path):

@@ -8,10 +8,11 @@ namespace tlb {
 
 __device__ __forceinline__ float sigmoidf(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float siluf(float x) { return x / (1.f + expf(-x)); }
+// z / 2 (1 + tanh(c)) = z sigmoid(2 c)
 __device__ __forceinline__ float gelu_tanhf(float z)
 {
-    constexpr float kRoot = 0.79788456080286535588f;         // sqrt(2 / pi)
-    return 0.5f * z * (1.f + tanhf(kRoot * fmaf(0.044715f * z * z, z, z)));
+    constexpr float kRoot2 = 2.f * 0.79788456080286535588f;  // 2 sqrt(2 / pi)
+    return z / (1.f + expf(-kRoot2 * fmaf(0.044715f * z * z, z, z)));
 }
 __device__ __forceinline__ float glu_act(int act, float gate, float up) { return (act == GLU_SILU ? siluf(gate) : gelu_tanhf(gate)) * up; }
 // value that enters a gated recurrence without a normaliser: positive, continuous, slope one above zero
@@ -29,6 +30,7 @@ __device__ __forceinline__ void group_inv_rms(F value, int n, int groups, float 
         const int g = u / per, s = u - g * per;
         const int beg = g * len + (int)((long long)len * s / per), end = g * len + (int)((long long)len * (s + 1) / per);
         float ss = 0.f;
+#pragma unroll 4
         for (int e = beg + lane; e < end; e += 32) { const float v = value(e); ss += v * v; }
 #pragma unroll
         for (int o = 16; o; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
@@ -42,6 +44,9 @@ __device__ __forceinline__ void group_inv_rms(F value, int n, int groups, float 
     }
     __syncthreads();
 }
+
+// part of element e (below 2^22) when a part has 1 / inv_len elements
+__device__ __forceinline__ int group_of(int e, float inv_len) { return (int)(((float)e + 0.5f) * inv_len); }
 
 // Chooses the experts of one token; all threads of the block call.  Scores are sigmoids of the logits; with several groups only
 // the `keep` groups whose two best scores sum highest take part (ties: the lower index).  sel / weight [top] and the scratch

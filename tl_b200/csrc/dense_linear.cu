@@ -46,10 +46,8 @@ struct DenseMvParams {
     int groups;
     const float *y, *y_gate, *post_w;
     float *h_out;
-    int act;
-    float *state;
-    size_t parity_stride;
-    const int *pos;
+    float *act_out;
+    int glu, act, ldx;
     RouteDesc route;
     const float *logits;
     int *sel;
@@ -91,7 +89,7 @@ __global__ void __launch_bounds__(kMvThreads, 4) dense_matvec_kernel(const Dense
     __shared__ float red[GNORM ? 2 * kMaxNormGroups : kMvWarps * 3];
     __shared__ float fold[2][GROUPS][WK][kMvRows];
     __shared__ int s_sel[EXPERT ? kMaxTop : 1];
-    __shared__ float s_weight[EXPERT ? kMaxTop : 1];
+    __shared__ float s_weight[EXPERT || EXPERTS ? kMaxTop + 1 : 1];
     __shared__ const __nv_bfloat16 *s_base[EXPERTS ? kMaxTop + 1 : 1];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, wk = warp % WK, wg = warp / WK;
 
@@ -109,19 +107,25 @@ __global__ void __launch_bounds__(kMvThreads, 4) dense_matvec_kernel(const Dense
             }
         }
     }
+    if (GNORM) {
+        for (int e = tid * 32; e < p.k; e += kMvThreads * 32) {
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(p.norm_w + e));
+            if (p.post_w) asm volatile("prefetch.global.L2 [%0];" ::"l"(p.post_w + e));
+        }
+    }
     pdl_wait();
     pdl_launch_dependents();
 
     const int kp = p.nch * kMvChunk;
     const __nv_bfloat16 *wbase = p.w;
-    float *outp = p.out;
+    float *actp = p.act_out;
     if (PRO == DPRO_PLAIN || EXPERT) {
         for (int e = tid; e < kp; e += kMvThreads) xs[xs_at(e)] = e < p.k ? __ldcg(p.x + e) : 0.f;
         if (EXPERT) {
             route_token(p.logits, p.route, xs + kp, s_sel, s_weight);
             const int slot = blockIdx.y;
             wbase += (size_t)s_sel[slot] * p.n * p.ld;
-            outp += (size_t)slot * p.n;
+            actp += (size_t)slot * (p.n / 2);
             if (blockIdx.x == 0 && slot == 0)
                 for (int i = tid; i < p.route.top; i += kMvThreads) { p.sel[i] = s_sel[i]; p.weight[i] = s_weight[i]; }
         }
@@ -142,9 +146,63 @@ __global__ void __launch_bounds__(kMvThreads, 4) dense_matvec_kernel(const Dense
         }
     } else if (GNORM) {
         const __nv_bfloat16 *er = p.emb ? p.emb + (size_t)*p.token * p.emb_ld : nullptr;
-        const int len = p.k / p.groups;
         float *inv = red + kMaxNormGroups;
         auto at = [&](int e) { return xs[xs_at(e)]; };
+        const float inv_len = (float)p.groups / (float)p.k;
+        auto scaled = [&](float4 v, float4 w, int e) {
+            return make_float4(v.x * inv[group_of(e, inv_len)] * (w.x + p.norm_offset), v.y * inv[group_of(e + 1, inv_len)] * (w.y + p.norm_offset),
+                               v.z * inv[group_of(e + 2, inv_len)] * (w.z + p.norm_offset), v.w * inv[group_of(e + 3, inv_len)] * (w.w + p.norm_offset));
+        };
+        constexpr int NV = 4;
+        if (!er && p.k % 4 == 0 && p.k <= NV * 4 * kMvThreads && (reinterpret_cast<uintptr_t>(p.y_gate) & 15) == 0) {
+            // 16 elements per thread: every load of the rows is on its way before the first is used
+            float4 v[NV], x[NV];
+            auto ld4 = [&](const float *src, int e) { return e < p.k ? __ldcg(reinterpret_cast<const float4 *>(src + e)) : make_float4(0.f, 0.f, 0.f, 0.f); };
+            auto slot = [&](int e) { return reinterpret_cast<float4 *>(xs + xs_at(e)); };
+            if (p.y) {
+                float4 g[NV];
+#pragma unroll
+                for (int i = 0; i < NV; i++) v[i] = ld4(p.y, (tid + i * kMvThreads) * 4);
+#pragma unroll
+                for (int i = 0; i < NV; i++) g[i] = p.y_gate ? ld4(p.y_gate, (tid + i * kMvThreads) * 4) : make_float4(INFINITY, INFINITY, INFINITY, INFINITY);
+#pragma unroll
+                for (int i = 0; i < NV; i++) x[i] = ld4(p.x, (tid + i * kMvThreads) * 4);
+#pragma unroll
+                for (int i = 0; i < NV; i++) {
+                    const int e = (tid + i * kMvThreads) * 4;
+                    v[i].x *= sigmoidf(g[i].x); v[i].y *= sigmoidf(g[i].y); v[i].z *= sigmoidf(g[i].z); v[i].w *= sigmoidf(g[i].w);
+                    if (e < p.k) *slot(e) = v[i];
+                }
+                __syncthreads();
+                group_inv_rms(at, p.k, p.groups, p.eps, red, inv);
+#pragma unroll
+                for (int i = 0; i < NV; i++) {
+                    const int e = (tid + i * kMvThreads) * 4;
+                    if (e < p.k) {
+                        const float4 a = scaled(*slot(e), *reinterpret_cast<const float4 *>(p.post_w + e), e);
+                        x[i].x += a.x; x[i].y += a.y; x[i].z += a.z; x[i].w += a.w;
+                        *slot(e) = x[i];
+                        if (blockIdx.x == 0) *reinterpret_cast<float4 *>(p.x_out + e) = x[i];
+                    }
+                }
+            } else {
+#pragma unroll
+                for (int i = 0; i < NV; i++) x[i] = ld4(p.x, (tid + i * kMvThreads) * 4);
+#pragma unroll
+                for (int i = 0; i < NV; i++)
+                    if ((tid + i * kMvThreads) * 4 < p.k) *slot((tid + i * kMvThreads) * 4) = x[i];
+            }
+            __syncthreads();
+            group_inv_rms(at, p.k, p.groups, p.eps, red, inv);
+#pragma unroll
+            for (int i = 0; i < NV; i++) {
+                const int e = (tid + i * kMvThreads) * 4;
+                if (e >= kp) continue;
+                const float4 a = e < p.k ? scaled(x[i], *reinterpret_cast<const float4 *>(p.norm_w + e), e) : make_float4(0.f, 0.f, 0.f, 0.f);
+                *slot(e) = a;
+                if (p.h_out && blockIdx.x == 0 && e < p.k) *reinterpret_cast<float4 *>(p.h_out + e) = a;
+            }
+        } else {
         if (p.y) {
             for (int e = tid; e < p.k; e += kMvThreads) {
                 const float v = __ldcg(p.y + e);
@@ -154,7 +212,7 @@ __global__ void __launch_bounds__(kMvThreads, 4) dense_matvec_kernel(const Dense
             group_inv_rms(at, p.k, p.groups, p.eps, red, inv);
             for (int e = tid; e < p.k; e += kMvThreads) {
                 float *s = xs + xs_at(e);
-                const float v = __ldcg(p.x + e) + *s * inv[e / len] * (p.post_w[e] + p.norm_offset);
+                const float v = __ldcg(p.x + e) + *s * inv[group_of(e, inv_len)] * (p.post_w[e] + p.norm_offset);
                 *s = v;
                 if (blockIdx.x == 0) p.x_out[e] = v;
             }
@@ -169,38 +227,26 @@ __global__ void __launch_bounds__(kMvThreads, 4) dense_matvec_kernel(const Dense
         group_inv_rms(at, p.k, p.groups, p.eps, red, inv);
         for (int e = tid; e < kp; e += kMvThreads) {
             float *s = xs + xs_at(e);
-            *s = e < p.k ? *s * inv[e / len] * (p.norm_w[e] + p.norm_offset) : 0.f;
+            *s = e < p.k ? *s * inv[group_of(e, inv_len)] * (p.norm_w[e] + p.norm_offset) : 0.f;
             if (p.h_out && blockIdx.x == 0 && e < p.k) p.h_out[e] = *s;
         }
-    } else if (PRO == DPRO_GLU) {
-        for (int e = tid; e < kp; e += kMvThreads) xs[xs_at(e)] = e < p.k ? glu_act(p.act, __ldcg(p.x + e), __ldcg(p.x + p.k + e)) : 0.f;
-    } else if (PRO == DPRO_GRU) {
-        const int pos = __ldcg(p.pos);
-        const float *sin = p.state + (size_t)(pos & 1) * p.parity_stride;
-        float *sout = p.state + (size_t)((pos & 1) ^ 1) * p.parity_stride;
-        for (int e = tid; e < kp; e += kMvThreads) {
-            float v = 0.f;
-            if (e < p.k) {
-                const float z = sigmoidf(__ldcg(p.x + e)), c = gru_candidate(__ldcg(p.x + p.k + e)), old = pos > 0 ? __ldcg(sin + e) : 0.f;
-                const float st = (1.f - z) * old + z * c;
-                if (blockIdx.x == 0) sout[e] = st;
-                v = st * siluf(__ldcg(p.x + 2 * p.k + e));
-            }
-            xs[xs_at(e)] = v;
         }
     } else if (EXPERTS) {
-        const int top = p.route.top;
-        for (int s = 0; s < top; s++) {
-            const float w = __ldcg(p.weight + s);
-            const float *x = p.x + (size_t)s * 2 * p.k;
-            float *dst = xs + s * p.seg_nch * kMvChunk;
-            for (int e = tid; e < p.seg_nch * kMvChunk; e += kMvThreads) dst[xs_at(e)] = e < p.k ? w * glu_act(p.act, __ldcg(x + e), __ldcg(x + p.k + e)) : 0.f;
+        const int top = p.route.top, seg = p.seg_nch * kMvChunk, first = top * seg;
+        for (int s = tid; s <= top; s += kMvThreads) {
+            s_weight[s] = s < top ? __ldcg(p.weight + s) : (p.shared_gate ? sigmoidf(__ldcg(p.shared_gate)) : 1.f);
+            s_base[s] = s < top ? p.w + (size_t)__ldcg(p.sel + s) * p.n * p.ld : p.shared_w;
         }
-        const int first = top * p.seg_nch * kMvChunk;
-        const float w = p.shared_gate ? sigmoidf(__ldcg(p.shared_gate)) : 1.f;
-        for (int e = tid; e < kp - first; e += kMvThreads)
-            xs[first + xs_at(e)] = e < p.shared_k ? w * glu_act(p.act, __ldcg(p.shared_x + e), __ldcg(p.shared_x + p.shared_k + e)) : 0.f;
-        for (int s = tid; s <= top; s += kMvThreads) s_base[s] = s < top ? p.w + (size_t)__ldcg(p.sel + s) * p.n * p.ld : p.shared_w;
+        __syncthreads();
+        for (int s = 0; s < top; s++) {
+            const float w = s_weight[s];
+            const float *x = p.x + (size_t)s * p.ldx;
+#pragma unroll 8
+            for (int e = tid; e < seg; e += kMvThreads) xs[s * seg + xs_at(e)] = e < p.k ? w * __ldcg(x + e) : 0.f;
+        }
+        const float w = s_weight[top];
+#pragma unroll 8
+        for (int e = tid; e < kp - first; e += kMvThreads) xs[first + xs_at(e)] = e < p.shared_k ? w * __ldcg(p.shared_x + e) : 0.f;
     } else {
         float ss[3] = {0.f, 0.f, 0.f};
         for (int e = tid; e < p.k; e += kMvThreads) {
@@ -273,12 +319,19 @@ __global__ void __launch_bounds__(kMvThreads, 4) dense_matvec_kernel(const Dense
                 for (int i = 0; i < WK; i++) y += fold[flip][wg][i][lane];
             }
         }
-        const int row = r0 + lane;
-        if (wk == 0 && lane < kMvRows && row < p.n) {
-            if (p.bias) y += p.bias[row];
-            if (p.softcap > 0.f) y = p.softcap * tanhf(y / p.softcap);
-            if (p.resid_scale) outp[row] = __ldcg(outp + row) + p.resid_scale[row] * y;
-            else outp[row] = y;
+        if (wk == 0) {
+            const int row = r0 + lane;
+            const bool in = lane < kMvRows && row < p.n;
+            if (in && p.bias) y += p.bias[row];
+            if (r0 < p.glu) {                                  // two gates and their ups
+                const float up = __shfl_down_sync(0xffffffffu, y, 2);
+                if (lane < 2) actp[(r0 >> 1) + lane] = glu_act(p.act, y, up);
+            } else if (in) {
+                if (p.softcap > 0.f) y = p.softcap * tanhf(y / p.softcap);
+                float *o = p.out + (row - p.glu);
+                if (p.resid_scale) *o = __ldcg(o) + p.resid_scale[row] * y;
+                else *o = y;
+            }
         }
     }
 }
@@ -296,8 +349,10 @@ struct DenseTcParams {
     float softcap;
     int per;
     size_t block_stride;
-    __half *out_h;
+    __half *out_h, *out_t;
     const int4 *tiles;
+    int glu, act, ld_act;
+    __nv_bfloat16 *act_out;
     uint32_t type_bits;                    // operand types in the instruction descriptor
 };
 
@@ -345,12 +400,41 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_cons
             const int row = n0 + warp * 32 + lane;
             const bool in = row < p.n;
             const float bias = in && p.bias ? p.bias[row] : 0.f, rs = in && p.resid_scale ? p.resid_scale[row] : 0.f;
-            const size_t place = (size_t)(row / p.per) * p.block_stride + row % p.per;
+            const int col = row - p.glu;
+            const size_t place = (size_t)(col / p.per) * p.block_stride + col % p.per;
+            if (p.out_t) t_end = (t_end + 127) / 128 * 128;        // rows past T came as zeros
             for (int c0 = 0; c0 < p.nt && t0 + c0 < t_end; c0 += 32) {
                 uint32_t v[32];
                 tmem_ld32(tmem + ((uint32_t)(warp * 32) << 16) + (uint32_t)c0, v);
                 tmem_wait_ld();
-                if (!in) continue;
+                if (n0 + warp * 32 < p.glu) {
+                    // lanes (0, 1), (2, 3) of four hold gates and ups of two units: the former take tokens 0 .. 15, the latter 16 .. 31
+                    const bool hi = lane & 2;
+                    const float mine = bias, theirs = __shfl_xor_sync(0xffffffffu, bias, 2);
+                    __nv_bfloat16 *da = p.act_out + (size_t)(t0 + c0) * p.ld_act + (row >> 2) * 2 + (row & 1);
+#pragma unroll
+                    for (int i = 0; i < 16; i++) {
+                        const float other = __uint_as_float(__shfl_xor_sync(0xffffffffu, hi ? v[i] : v[i + 16], 2)) + theirs;
+                        const float own = __uint_as_float(hi ? v[i + 16] : v[i]) + mine;
+                        const int t = hi ? i + 16 : i;
+                        if (row < p.glu && t0 + c0 + t < t_end) da[(size_t)t * p.ld_act] = __float2bfloat16_rn(hi ? glu_act(p.act, other, own) : glu_act(p.act, own, other));
+                    }
+                }
+                if (!in || row < p.glu) continue;
+                if (p.out_t) {
+                    __half *dt = p.out_t + (size_t)(col / p.per) * p.block_stride + (size_t)(col % p.per) * p.ldo + t0 + c0;
+#pragma unroll
+                    for (int i = 0; i < 32; i += 8) {
+                        uint32_t w[4];
+#pragma unroll
+                        for (int k = 0; k < 4; k++) {
+                            const __half2 h = __floats2half2_rn(fminf(fmaxf(__uint_as_float(v[i + 2 * k]), -65504.f), 65504.f), fminf(fmaxf(__uint_as_float(v[i + 2 * k + 1]), -65504.f), 65504.f));
+                            w[k] = *reinterpret_cast<const uint32_t *>(&h);
+                        }
+                        *reinterpret_cast<uint4 *>(dt + i) = make_uint4(w[0], w[1], w[2], w[3]);
+                    }
+                    continue;
+                }
                 float *dst = p.out + (size_t)(t0 + c0) * p.ldo + place;
                 const int m = min(32, t_end - t0 - c0);
                 if (p.out_h) {
@@ -392,7 +476,8 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_cons
         }
     } else if (lane == 0) {
         // f32 accumulator, operands of one 16-bit type, both K-major, M 128, N nt
-        const uint32_t idesc = (1u << 4) | p.type_bits | ((uint32_t)(p.nt >> 3) << 17) | ((uint32_t)(kTcRows >> 4) << 24);
+        const int cols = p.tiles ? (t_end - t0 + 15) / 16 * 16 : p.nt;       // a tile that is not full multiplies fewer columns
+        const uint32_t idesc = (1u << 4) | p.type_bits | ((uint32_t)(cols >> 3) << 17) | ((uint32_t)(kTcRows >> 4) << 24);
         for (int k = 0; k < p.kt; k++) {
             const int s = k % p.stages;
             if (!mbar_wait(full + 8 * s, (uint32_t)(k / p.stages) & 1u, abort_flag, p.err, 63)) break;
@@ -424,6 +509,8 @@ struct DenseF32Params {
     int per;
     size_t block_stride;
     const int4 *tiles;
+    int glu, act, ld_act;
+    float *act_out;
 };
 constexpr int kSgT = kF32GemmRows, kSgN = 64, kSgK = 16;
 
@@ -458,13 +545,27 @@ __global__ void __launch_bounds__(256) dense_gemm_f32_kernel(const DenseF32Param
         }
         __syncthreads();
     }
+    if (n0 + tn * 4 < p.glu) {                 // this thread's four columns: two gates and their ups
+        const int n = n0 + tn * 4;
+        float b[4];
+#pragma unroll
+        for (int j = 0; j < 4; j++) b[j] = p.bias ? p.bias[n + j] : 0.f;
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            const int t = t0 + tt * 4 + i;
+            if (t >= t_end) continue;
+#pragma unroll
+            for (int j = 0; j < 2; j++) p.act_out[(size_t)t * p.ld_act + n / 2 + j] = glu_act(p.act, acc[i][j] + b[j], acc[i][j + 2] + b[j + 2]);
+        }
+        return;
+    }
 #pragma unroll
     for (int i = 0; i < 4; i++)
 #pragma unroll
         for (int j = 0; j < 4; j++) {
-            const int t = t0 + tt * 4 + i, n = n0 + tn * 4 + j;
+            const int t = t0 + tt * 4 + i, n = n0 + tn * 4 + j, col = n - p.glu;
             if (t >= t_end || n >= p.n) continue;
-            float *o = p.out + (size_t)t * p.ldo + (size_t)(n / p.per) * p.block_stride + n % p.per;
+            float *o = p.out + (size_t)t * p.ldo + (size_t)(col / p.per) * p.block_stride + col % p.per;
             if (p.resid_scale) { *o = fmaf(p.resid_scale[n], acc[i][j], *o); continue; }
             const float y = acc[i][j] + (p.bias ? p.bias[n] : 0.f);
             *o = p.softcap > 0.f ? p.softcap * tanhf(y / p.softcap) : y;
@@ -582,6 +683,12 @@ __global__ void pack_rows_kernel(const __nv_bfloat16 *__restrict__ src, int k, _
     for (int i = threadIdx.x; i < k; i += blockDim.x) dst[(size_t)blockIdx.x * ld + i] = src[(size_t)blockIdx.x * k + i];
 }
 
+__global__ void pack_glu_rows_kernel(const __nv_bfloat16 *__restrict__ src, int k, __nv_bfloat16 *__restrict__ dst, int ld)
+{
+    const int i = blockIdx.x;
+    for (int e = threadIdx.x; e < k; e += blockDim.x) dst[(size_t)((i >> 1) * 4 + (i & 1)) * ld + e] = src[(size_t)i * k + e];
+}
+
 __global__ void pack_rows_f16_kernel(const __nv_bfloat16 *__restrict__ src, int k, __half *__restrict__ dst, int ld)
 {
     for (int i = threadIdx.x; i < ld; i += blockDim.x)
@@ -648,8 +755,8 @@ tlb_status launch_dense_matvec(const DenseMatvecJob &j)
     p.w = j.w.w; p.n = j.w.n; p.k = j.w.k; p.ld = j.w.ld; p.nch = (j.w.ld + kMvChunk - 1) / kMvChunk;
     p.bias = j.w.bias; p.x = j.x; p.emb = j.emb; p.emb_ld = act_ld(j.w.k); p.token = j.token; p.x_out = j.x_out;
     p.norm_w = j.norm_w; p.norm_offset = j.norm_offset; p.eps = j.eps; p.poly = j.poly; p.out = j.out; p.resid_scale = j.resid_scale;
-    p.softcap = j.softcap; p.groups = j.groups; p.y = j.y; p.y_gate = j.y_gate; p.post_w = j.post_w; p.h_out = j.h_out; p.act = j.act;
-    p.state = j.state; p.parity_stride = j.parity_stride; p.pos = j.pos;
+    p.softcap = j.softcap; p.groups = j.groups; p.y = j.y; p.y_gate = j.y_gate; p.post_w = j.post_w; p.h_out = j.h_out;
+    p.glu = j.w.glu; p.act = j.w.glu_act; p.act_out = j.act_out; p.ldx = j.ldx;
     p.route = j.route; p.logits = j.logits; p.sel = j.sel; p.weight = j.weight;
     if (j.pro == DPRO_EXPERTS) {
         p.seg_nch = p.nch;
@@ -658,8 +765,6 @@ tlb_status launch_dense_matvec(const DenseMatvecJob &j)
         return pick_matvec<DPRO_EXPERTS>(p, j.pdl);
     }
     if (j.pro == DPRO_GNORM) return pick_matvec<DPRO_GNORM>(p, j.pdl);
-    if (j.pro == DPRO_GLU) return pick_matvec<DPRO_GLU>(p, j.pdl);
-    if (j.pro == DPRO_GRU) return pick_matvec<DPRO_GRU>(p, j.pdl);
     if (j.pro == DPRO_EXPERT) return pick_matvec<DPRO_EXPERT>(p, j.pdl);
     if (j.pro == DPRO_NORM) return pick_matvec<DPRO_NORM>(p, j.pdl);
     if (j.pro == DPRO_POLY) return pick_matvec<DPRO_POLY>(p, j.pdl);
@@ -675,6 +780,7 @@ tlb_status launch_dense_gemm(const DenseGemmJob &j, bool f32)
     if (f32) {
         DenseF32Params p;
         p.softcap = j.softcap; p.per = per; p.block_stride = j.block_stride; p.tiles = j.tiles;
+        p.glu = j.w.glu; p.act = j.w.glu_act; p.ld_act = j.ld_act; p.act_out = (float *)j.act_out;
         p.w = j.w.w; p.n = j.w.n; p.k = j.w.k; p.ld = j.w.ld; p.bias = j.w.bias; p.x = (const float *)j.x; p.resid_scale = j.resid_scale;
         p.ldx = j.ldx; p.T = j.T; p.ldo = j.ldo; p.out = j.out;
         dense_gemm_f32_kernel<<<dim3(j.tiles ? j.n_tiles : (j.T + kSgT - 1) / kSgT, (j.w.n + kSgN - 1) / kSgN), 256, 0, c->stream>>>(p);
@@ -682,9 +788,10 @@ tlb_status launch_dense_gemm(const DenseGemmJob &j, bool f32)
     }
     DenseTcParams p;
     p.out = j.out; p.bias = j.w.bias; p.resid_scale = j.resid_scale; p.n = j.w.n; p.T = j.T; p.ldo = j.ldo;
-    p.softcap = j.softcap; p.per = per; p.block_stride = j.block_stride; p.out_h = j.out_h; p.tiles = j.tiles;
+    p.softcap = j.softcap; p.per = per; p.block_stride = j.block_stride; p.out_h = j.out_h; p.out_t = j.out_t; p.tiles = j.tiles;
+    p.glu = j.w.glu; p.act = j.w.glu_act; p.ld_act = j.ld_act; p.act_out = (__nv_bfloat16 *)j.act_out;
     p.type_bits = j.w.f16 ? 0u : (1u << 7) | (1u << 10);
-    p.nt = j.tiles ? j.tile_rows : std::min(256, (j.T + 31) / 32 * 32);
+    p.nt = j.tiles ? j.tile_rows : (j.out_t ? 128 : std::min(256, (j.T + 31) / 32 * 32));
     p.tmem_cols = 32;
     while (p.tmem_cols < (uint32_t)p.nt) p.tmem_cols *= 2;
     p.kt = (j.w.k + kTcK - 1) / kTcK;
@@ -735,6 +842,12 @@ tlb_status launch_gather_rows(const float *x, int width, const int *idx, int n, 
 tlb_status launch_pack_rows(const __nv_bfloat16 *src, int n, int k, __nv_bfloat16 *dst, int ld, int col0)
 {
     pack_rows_kernel<<<n, 256, 0, ctx()->stream>>>(src, k, dst + col0, ld);
+    return launched("weight packing launch");
+}
+
+tlb_status launch_pack_glu_rows(const __nv_bfloat16 *src, int ff, int k, __nv_bfloat16 *dst, int ld, bool up)
+{
+    pack_glu_rows_kernel<<<ff, 256, 0, ctx()->stream>>>(src, k, dst + (up ? (size_t)2 * ld : 0), ld);
     return launched("weight packing launch");
 }
 

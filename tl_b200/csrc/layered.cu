@@ -24,7 +24,7 @@ struct Layer {
     RouteDesc route;
     tlb_tensor *norm1 = nullptr, *norm2 = nullptr, *post1 = nullptr, *post2 = nullptr, *ls1 = nullptr, *ls2 = nullptr, *act = nullptr;
     tlb_tensor *sink = nullptr, *onorm = nullptr, *w0 = nullptr, *qnorm = nullptr, *cnorm = nullptr;
-    // columns of the stacked projections (-1: absent): latent, output gate, residual gate; shared expert's gate | up is first of `up`
+    // columns of the stacked projections (-1: absent), those of `up` behind its gated activations
     int c_kv = -1, c_gate = -1, c_rg1 = -1, u_rg2 = -1, u_router = -1, u_sg = -1;
     uint64_t step_bytes = 0;               // weights one decoded token reads
     float *bias = nullptr;                 // by distance, [heads][bias_n]
@@ -41,11 +41,11 @@ struct RotTable { int dims; double base; RotScaling scaling; float *cos_t, *sin_
 struct RowBufs {
     float *x = nullptr, *proj = nullptr, *u = nullptr, *o = nullptr, *y = nullptr, *q = nullptr, *dly = nullptr;
     float2 *look = nullptr;
-    void *act = nullptr, *th = nullptr;
+    void *act = nullptr, *hid = nullptr, *th = nullptr;
     // mixture of experts: T * top rows
     MoePlan plan;
-    float *hp = nullptr, *yp = nullptr, *ysh = nullptr;
-    void *xp = nullptr;
+    float *yp = nullptr, *ysh = nullptr;
+    void *xp = nullptr, *hp = nullptr;
     // latent attention, rows of queries in the latent space
     void *qa = nullptr;
     float *partial = nullptr;
@@ -72,7 +72,7 @@ struct LayeredModel {
     RowBufs batch_rows;                    // of a session with several sequences (x: the session's)
     // one token: projections (a layer's residual gate is read while the next layer writes: two), mixer output, up projection
     float *proj[2] = {nullptr, nullptr}, *mix = nullptr, *up = nullptr, *partial = nullptr;
-    float *x2 = nullptr, *y = nullptr, *h = nullptr, *q = nullptr, *ex = nullptr, *weight = nullptr;
+    float *x2 = nullptr, *y = nullptr, *h = nullptr, *q = nullptr, *hid = nullptr, *ex = nullptr, *weight = nullptr;
     void *qa = nullptr;
     int *counters = nullptr, *sel = nullptr;
     int ldp = 0, ldm = 0, ldu = 0, lda = 0, ldq = 0;
@@ -131,13 +131,18 @@ struct Loader {
     }
     // several [n_i, k] matrices as one, rows one after the other; a single matrix whose rows are whole 16-byte lines stays where it is
     struct Part { std::string name; int n; bool bias; };
-    tlb_status stack(DenseW *w, const std::vector<Part> &parts, int k)
+    // the two [ff, k] matrices of a gated activation; they come first, in pairs (DenseW::glu)
+    struct Glu { std::string gate, up; int ff; };
+    static int glu_rows(int ff) { return 2 * ((ff + 1) / 2 * 2); }
+    tlb_status stack(DenseW *w, const std::vector<Part> &parts, int k, const std::vector<Glu> &pairs = {}, int act = 0)
     {
-        int n = 0;
+        int n = 0, glu = 0;
         bool any_bias = false;
+        for (const Glu &g : pairs) glu += glu_rows(g.ff);
         for (const Part &p : parts) { n += p.n; any_bias |= p.bias; }
-        w->n = n; w->k = k; w->ld = act_ld(k);
-        if (parts.size() == 1 && w->ld == k) {
+        n += glu;
+        w->n = n; w->k = k; w->ld = act_ld(k); w->glu = glu; w->glu_act = act;
+        if (parts.size() == 1 && !glu && w->ld == k) {
             const tlb_tensor *t;
             TLB_TRY(matrix(parts[0].name, &t, n, k));
             tlb_tensor_retain(const_cast<tlb_tensor *>(t));
@@ -145,8 +150,18 @@ struct Loader {
             w->w = (const __nv_bfloat16 *)t->data();
         } else {
             __nv_bfloat16 *dst;
-            TLB_TRY(alloc(lm, &dst, (size_t)n * w->ld, w->ld != k));
+            bool odd = false;
+            for (const Glu &g : pairs) odd |= g.ff % 2 != 0;
+            TLB_TRY(alloc(lm, &dst, (size_t)n * w->ld, w->ld != k || odd));
             int at = 0;
+            for (const Glu &g : pairs) {
+                for (int up = 0; up < 2; up++) {
+                    const tlb_tensor *t;
+                    TLB_TRY(matrix(up ? g.up : g.gate, &t, g.ff, k));
+                    TLB_TRY(launch_pack_glu_rows((const __nv_bfloat16 *)t->data(), g.ff, k, dst + (size_t)at * w->ld, w->ld, up));
+                }
+                at += glu_rows(g.ff);
+            }
             for (const Part &p : parts) {
                 const tlb_tensor *t;
                 TLB_TRY(matrix(p.name, &t, p.n, k));
@@ -158,7 +173,7 @@ struct Loader {
         if (any_bias) {
             float *b;
             TLB_TRY(alloc(lm, &b, n));
-            int at = 0;
+            int at = glu;
             for (const Part &p : parts) {
                 if (p.bias) {
                     tlb_tensor *t;
@@ -320,13 +335,15 @@ struct Loader {
             const FfnDesc &f = d.ffn;
             in.clear();
             n_in = 0;
+            std::vector<Glu> pairs;
+            const int act = f.act == FfnAct::SiluGlu ? GLU_SILU : GLU_GELU_TANH;
             if (f.act == FfnAct::PolyNorm) {
                 add(p + "mlp.up", f.ff, false);
                 TLB_TRY(vec(p + "mlp.act", &L->act, 4));
             } else if (!f.experts) {
-                add(p + "mlp.gate", f.ff, false); add(p + "mlp.up", f.ff, false);
+                pairs.push_back({p + "mlp.gate", p + "mlp.up", f.ff});
             } else if (f.shared_ff) {
-                add(p + "mlp.shared.gate", f.shared_ff, false); add(p + "mlp.shared.up", f.shared_ff, false);
+                pairs.push_back({p + "mlp.shared.gate", p + "mlp.shared.up", f.shared_ff});
             }
             if (d.resid_gate) L->u_rg2 = add(p + "rg2", W, true);
             if (f.experts) {
@@ -337,21 +354,22 @@ struct Loader {
                     L->u_sg = add(p + "mlp.shared.sg", 1, false);
                     TLB_TRY(stack(&L->sdown, {{p + "mlp.shared.down", W, false}}, f.shared_ff));
                 }
-                std::vector<Part> eu, ed;
+                std::vector<Glu> eu;
+                std::vector<Part> ed;
                 for (int e = 0; e < f.experts; e++) {
                     const std::string ep = p + "mlp.e" + std::to_string(e) + ".";
-                    eu.push_back({ep + "gate", f.ff, false}); eu.push_back({ep + "up", f.ff, false});
+                    eu.push_back({ep + "gate", ep + "up", f.ff});
                     ed.push_back({ep + "down", W, false});
                 }
                 const uint64_t b0 = lm->weight_bytes;
-                TLB_TRY(stack(&L->eup, eu, W));
+                TLB_TRY(stack(&L->eup, {}, W, eu, act));
                 TLB_TRY(stack(&L->edown, ed, f.ff));
-                L->eup.n = 2 * f.ff; L->edown.n = W;         // rows of one expert
+                L->eup.n = L->eup.glu = glu_rows(f.ff); L->edown.n = W;         // rows of one expert
                 idle = (lm->weight_bytes - b0) / f.experts * (f.experts - f.top);
             } else {
                 TLB_TRY(stack(&L->down, {{p + "mlp.down", W, false}}, f.ff));
             }
-            TLB_TRY(stack(&L->up, in, W));
+            TLB_TRY(stack(&L->up, in, W, pairs, act));
             TLB_TRY(vec(p + "norm2", &L->norm2, W));
             if (d.post_norm) TLB_TRY(vec(p + "norm2b", &L->post2, W));
             if (d.layer_scale) TLB_TRY(vec(p + "ls2", &L->ls2, W));
@@ -376,7 +394,7 @@ struct Loader {
             if (!latent_supported(latent_args(lm, *L, nullptr, 0, nullptr, 0), lm->cfg.f32)) return fail(TLB_ERR_SHAPE, "layer %d: latent attention over %d + %d cached values is not supported", idx, x.kv_rank, x.rot_dim);
             return alloc(lm, (char **)&L->kcache, rows * latent_ld(x.kv_rank, x.rot_dim) * es);
         case MixerKind::MinGru:
-            return alloc(lm, &L->state, 2 * B * x.width);
+            return alloc(lm, &L->state, B * x.width);
         default:
             return alloc(lm, &L->state, B * x.heads * x.vdim * mix_recur_ld(x.dim));
         }
@@ -411,14 +429,10 @@ MixRecur recur_args(const LayeredModel *lm, const Layer &L, float *proj, int ldp
 
 MixGru gru_args(const LayeredModel *lm, const Layer &L, const float *proj, int ldp)
 {
-    const int w = L.d->mix.width;
-    return MixGru{w, L.state, (size_t)lm->cfg.batch * w, proj, ldp};
+    return MixGru{L.d->mix.width, L.state, proj, ldp};
 }
 
-int glu_act_of(const FfnDesc &f) { return f.act == FfnAct::SiluGlu ? GLU_SILU : GLU_GELU_TANH; }
-
-// The mixer of one token per sequence: projection rows in, gated / attended rows out.  (A MinGru of one token is part of the
-// output projection's launch.)
+// The mixer of one token per sequence: projection rows in, gated / attended rows out.
 tlb_status decode_mixer(LayeredModel *lm, const Layer &L, int batch, float *proj, float *q, void *qa, float *latent_partial, const int *pos, const int *rope_pos, void *out,
                         int ldo, bool out_f32, bool pdl)
 {
@@ -438,7 +452,7 @@ tlb_status decode_mixer(LayeredModel *lm, const Layer &L, int batch, float *proj
         return launch_latent_rows(j);
     }
     case MixerKind::MinGru:
-        return launch_gru_rows(gru_args(lm, L, proj, lm->ldp), batch, pos, out, ldo, out_f32);
+        return launch_gru_rows(gru_args(lm, L, proj, lm->ldp), batch, pos, out, ldo, out_f32, pdl);
     default: {
         MixRecurDecode j = {};
         j.m = recur_args(lm, L, proj, lm->ldp);
@@ -468,16 +482,17 @@ template <typename Get>
 tlb_status row_bufs(const LayeredModel *lm, int T, bool absorbed, RowBufs *b, Get get)
 {
     const size_t es = lm->cfg.f32 ? 4 : 2, W = lm->desc.width;
-    size_t n_dly = 0, n_th = 0, n_look = 0, n_y = 0, top = 0, experts = 0, ff = 0, ld_ff = 0, tiles = 0, shared = 0, n_qa = 0, n_part = 0;
+    size_t n_dly = 0, n_th = 0, n_look = 0, n_y = 0, top = 0, experts = 0, ld_ff = 0, ld_hid = 0, tiles = 0, shared = 0, n_qa = 0, n_part = 0;
     for (const Layer &L : lm->layers) {
         if (L.d->mix.kind == MixerKind::GeneralDelta) { n_dly = std::max(n_dly, (size_t)L.w2.n); n_th = std::max(n_th, (size_t)L.w2.k); n_look = std::max(n_look, (size_t)L.d->mix.heads); }
         if (L.d->post_norm) n_y = W;
         if (L.eup.w) {
             top = std::max(top, (size_t)L.route.top); experts = std::max(experts, (size_t)L.route.experts);
-            ff = std::max(ff, (size_t)L.route.top * L.eup.n); ld_ff = std::max(ld_ff, (size_t)act_ld(L.edown.k));
+            ld_ff = std::max(ld_ff, (size_t)act_ld(L.edown.k));
             tiles = std::max(tiles, (size_t)moe_max_tiles(L.route, T, lm->cfg.f32));
             if (L.sdown.w) shared = W;
         }
+        if (L.up.glu) ld_hid = std::max(ld_hid, (size_t)act_ld(L.up.glu / 2));
         if (absorbed && L.d->mix.kind == MixerKind::Latent) {
             const MixLatent m = latent_args(lm, L, nullptr, 0, nullptr, 0);
             n_qa = std::max(n_qa, (size_t)m.H * m.ld); n_part = std::max(n_part, latent_partial_floats(m, T));
@@ -499,17 +514,19 @@ tlb_status row_bufs(const LayeredModel *lm, int T, bool absorbed, RowBufs *b, Ge
     TLB_TRY(want(&b->plan.weight, t * top * 4));
     TLB_TRY(want(&b->plan.count, 2 * experts * 4));
     TLB_TRY(want(&b->plan.tiles, tiles * sizeof(int4)));
-    TLB_TRY(want(&b->hp, t * ff * 4));
+    TLB_TRY(want(&b->hid, t * ld_hid * es));
+    TLB_TRY(want(&b->hp, t * top * ld_ff * es));
     TLB_TRY(want(&b->yp, t * top * W * 4));
-    TLB_TRY(want(&b->xp, t * top * std::max((size_t)act_ld((int)W), ld_ff) * es));
+    TLB_TRY(want(&b->xp, t * top * act_ld((int)W) * es));
     TLB_TRY(want(&b->ysh, t * shared * 4));
     TLB_TRY(want(&b->qa, t * n_qa * es));
     return want(&b->partial, n_part * 4);
 }
 
-tlb_status rows_gemm(const LayeredModel *lm, const DenseW &w, const void *x, int ldx, int T, float *out, int ldo, const tlb_tensor *scale, float softcap = 0.f)
+tlb_status rows_gemm(const LayeredModel *lm, const DenseW &w, const void *x, int ldx, int T, float *out, int ldo, const tlb_tensor *scale, float softcap = 0.f, void *hid = nullptr)
 {
     DenseGemmJob j;
+    j.act_out = hid; j.ld_act = act_ld(w.glu / 2);
     j.w = w; j.x = x; j.ldx = ldx; j.T = T; j.out = out; j.ldo = ldo; j.resid_scale = scale ? scale->f32() : nullptr; j.softcap = softcap;
     return launch_dense_gemm(j, lm->cfg.f32);
 }
@@ -558,25 +575,22 @@ tlb_status rows_mixer(LayeredModel *lm, const Layer &L, RowBufs &b, const RowCtx
     return TLB_OK;
 }
 
-// The mixture of experts over rows: normed rows in b.act, the first projection in b.u.
+// The mixture of experts over rows: normed rows in b.act, of the first projection the shared activations in b.hid, the rest in b.u.
 tlb_status rows_experts(LayeredModel *lm, const Layer &L, RowBufs &b, int T, MoeRows *out)
 {
     const bool f32 = lm->cfg.f32;
-    const int W = lm->desc.width, ff = L.edown.k, ldw = act_ld(W), ldf = act_ld(ff), P = T * L.route.top, act = glu_act_of(L.d->ffn);
+    const int W = lm->desc.width, ff = L.edown.k, ldw = act_ld(W), ldf = act_ld(ff), P = T * L.route.top;
     TLB_TRY(launch_moe_plan(L.route, b.u + L.u_router, lm->ldu, T, b.plan, f32));
     TLB_TRY(launch_moe_gather(L.route, b.plan, b.act, T, ldw, b.xp, f32));
     DenseGemmJob j;
     j.tiles = b.plan.tiles; j.n_tiles = moe_max_tiles(L.route, T, f32); j.tile_rows = moe_tile_rows(L.route, T, f32); j.n_weights = L.route.experts; j.T = P;
-    j.w = L.eup; j.x = b.xp; j.ldx = ldw; j.out = b.hp; j.ldo = 2 * ff;
+    j.w = L.eup; j.x = b.xp; j.ldx = ldw; j.act_out = b.hp; j.ld_act = ldf;
     TLB_TRY(launch_dense_gemm(j, f32));
-    TLB_TRY(launch_glu_rows(b.hp, P, ff, 2 * ff, act, b.xp, ldf, f32));
-    j.w = L.edown; j.ldx = ldf; j.out = b.yp; j.ldo = W;
+    j.w = L.edown; j.x = b.hp; j.ldx = ldf; j.out = b.yp; j.ldo = W;
     TLB_TRY(launch_dense_gemm(j, f32));
     out->top = L.route.top; out->slot = b.plan.place; out->weight = b.plan.weight; out->part = b.yp;
     if (L.sdown.w) {
-        const int sf = L.sdown.k, lds = act_ld(sf);
-        TLB_TRY(launch_glu_rows(b.u, T, sf, lm->ldu, act, b.act, lds, f32));
-        TLB_TRY(rows_gemm(lm, L.sdown, b.act, lds, T, b.ysh, W, nullptr));
+        TLB_TRY(rows_gemm(lm, L.sdown, b.hid, act_ld(L.sdown.k), T, b.ysh, W, nullptr));
         out->shared = b.ysh; out->shared_gate = b.u + L.u_sg; out->ld_shared_gate = lm->ldu;
     }
     return TLB_OK;
@@ -608,15 +622,14 @@ tlb_status run_rows(LayeredModel *lm, RowBufs &b, const RowCtx &c)
         TLB_TRY(rows_gemm(lm, L.o, b.act, lda, T, post ? b.y : b.x, W, L.ls1));
         TLB_TRY(join(L, nullptr, L.c_rg1 >= 0 ? b.proj + L.c_rg1 : nullptr, lm->ldp, L.post1, L.up.w ? L.norm2 : next));
         if (!L.up.w) continue;
-        TLB_TRY(rows_gemm(lm, L.up, b.act, ldw, T, b.u, lm->ldu, nullptr));
+        TLB_TRY(rows_gemm(lm, L.up, b.act, ldw, T, b.u, lm->ldu, nullptr, 0.f, b.hid));
         MoeRows moe;
         if (L.eup.w) {
             TLB_TRY(rows_experts(lm, L, b, T, &moe));
         } else {
             const int ldf = act_ld(L.down.k);
             if (L.act) TLB_TRY(launch_poly_rows(b.u, T, L.down.k, lm->ldu, L.act->f32(), md.eps, b.act, ldf, f32));
-            else TLB_TRY(launch_glu_rows(b.u, T, L.down.k, lm->ldu, glu_act_of(L.d->ffn), b.act, ldf, f32));
-            TLB_TRY(rows_gemm(lm, L.down, b.act, ldf, T, post ? b.y : b.x, W, L.ls2));
+            TLB_TRY(rows_gemm(lm, L.down, L.act ? b.act : b.hid, ldf, T, post ? b.y : b.x, W, L.ls2));
         }
         TLB_TRY(join(L, L.eup.w ? &moe : nullptr, L.u_rg2 >= 0 ? b.u + L.u_rg2 : nullptr, lm->ldu, L.post2, next));
     }
@@ -638,6 +651,7 @@ struct Chain {
     {
         const ModelDesc &d = lm->desc;
         DenseMatvecJob j;
+        j.act_out = lm->hid;
         j.w = w; j.norm_w = norm->f32(); j.norm_offset = d.norm_offset; j.eps = d.eps; j.groups = d.norm_groups; j.out = out; j.h_out = h_out; j.softcap = softcap;
         j.pro = d.norm_groups > 1 || post || h_out ? DPRO_GNORM : DPRO_NORM;
         j.x = buf[cur];
@@ -691,7 +705,7 @@ tlb_status layered_create(LayeredModel **out, const ModelDesc &desc, tlb_map *m,
         for (size_t i = 0; i < desc.layers.size(); i++) { lm->layers[i].d = &lm->desc.layers[i]; TLB_TRY(ld.state(&lm->layers[i], lm->desc.layers[i], (int)i)); }
         TLB_TRY(ld.stack(&lm->head, {{"head", desc.vocab, false}}, W));
         TLB_TRY(ld.vec("final.norm", &lm->final_norm, W));
-        size_t part = 1, lpart = 0, qa = 0, ex = 0, top = 0, attn_part = 0;
+        size_t part = 1, lpart = 0, qa = 0, hid = 0, ex = 0, top = 0, attn_part = 0;
         int kvh = 1;
         lm->ldp = lm->ldm = lm->ldu = 8;
         lm->lda = act_ld(W);
@@ -699,7 +713,7 @@ tlb_status layered_create(LayeredModel **out, const ModelDesc &desc, tlb_map *m,
             const MixerDesc &x = L.d->mix;
             lm->ldp = std::max(lm->ldp, act_ld(L.in.n));
             lm->ldm = std::max(lm->ldm, act_ld(L.out_width));
-            lm->ldu = std::max(lm->ldu, act_ld(L.up.n));
+            lm->ldu = std::max(lm->ldu, act_ld(L.up.n - L.up.glu));
             for (int n : {L.out_width, L.down.k, L.sdown.k, x.q_rank}) lm->lda = std::max(lm->lda, act_ld(n));
             if (x.kind == MixerKind::Attention) {
                 attn_part = std::max(attn_part, mix_attn_decode_partial_floats(attn_args(lm, L, nullptr, 0), B));
@@ -710,7 +724,8 @@ tlb_status layered_create(LayeredModel **out, const ModelDesc &desc, tlb_map *m,
                 qa = std::max(qa, (size_t)m.H * m.ld);
                 if (x.q_rank) lm->ldq = std::max(lm->ldq, act_ld(L.uq.n));
             }
-            if (L.eup.w) { ex = std::max(ex, (size_t)L.route.top * L.eup.n); top = std::max(top, (size_t)L.route.top); }
+            hid = std::max(hid, (size_t)L.up.glu / 2);
+            if (L.eup.w) { ex = std::max(ex, (size_t)L.route.top * L.eup.n / 2); top = std::max(top, (size_t)L.route.top); }
         }
         part = std::max(part, std::max(attn_part, lpart));
         for (float *&p : lm->proj) TLB_TRY(alloc(lm, &p, lm->ldp));
@@ -720,6 +735,7 @@ tlb_status layered_create(LayeredModel **out, const ModelDesc &desc, tlb_map *m,
         TLB_TRY(alloc(lm, &lm->counters, (size_t)B * kvh));
         for (float **p : {&lm->x2, &lm->y, &lm->h}) TLB_TRY(alloc(lm, p, W));
         if (lm->ldq) TLB_TRY(alloc(lm, &lm->q, lm->ldq));
+        if (hid) TLB_TRY(alloc(lm, &lm->hid, hid));
         if (qa) TLB_TRY(alloc(lm, (char **)&lm->qa, qa * (cfg.f32 ? 4 : 2)));
         if (top) { TLB_TRY(alloc(lm, &lm->ex, ex)); TLB_TRY(alloc(lm, &lm->weight, top)); TLB_TRY(alloc(lm, &lm->sel, top)); }
         if (B > 1) TLB_TRY(row_bufs(lm, B, true, &lm->batch_rows, [&](void **p, size_t bytes) { return alloc(lm, (char **)p, bytes); }));
@@ -749,27 +765,21 @@ tlb_status layered_step(LayeredModel *lm, const int *token, const int *pos, cons
             j.w = L.uq; j.pro = DPRO_NORM; j.x = proj; j.norm_w = L.qnorm->f32(); j.eps = eps; j.out = lm->q;
             TLB_TRY(launch_dense_matvec(j));
         }
+        TLB_TRY(decode_mixer(lm, L, 1, proj, lm->q, lm->qa, lm->partial, pos, rope_pos, lm->mix, lm->ldm, true, true));
         DenseMatvecJob j;
-        j.w = L.o;
-        if (mx.kind == MixerKind::MinGru) {
-            j.pro = DPRO_GRU; j.x = proj; j.state = L.state; j.parity_stride = gru_args(lm, L, proj, 0).parity_stride; j.pos = pos;
-        } else {
-            TLB_TRY(decode_mixer(lm, L, 1, proj, lm->q, lm->qa, lm->partial, pos, rope_pos, lm->mix, lm->ldm, true, true));
-            j.x = lm->mix;
-        }
+        j.w = L.o; j.x = lm->mix;
         TLB_TRY(c.back(j, L, L.ls1, L.post1, L.c_rg1 >= 0 ? proj + L.c_rg1 : nullptr));
         if (!L.up.w) continue;
         TLB_TRY(c.front(L.up, L.norm2, lm->up, L.eup.w ? lm->h : nullptr));
         j = DenseMatvecJob();
         if (L.eup.w) {
-            j.w = L.eup; j.pro = DPRO_EXPERT; j.x = lm->h; j.route = L.route; j.logits = lm->up + L.u_router; j.sel = lm->sel; j.weight = lm->weight; j.out = lm->ex;
+            j.w = L.eup; j.pro = DPRO_EXPERT; j.x = lm->h; j.route = L.route; j.logits = lm->up + L.u_router; j.sel = lm->sel; j.weight = lm->weight; j.act_out = lm->ex;
             TLB_TRY(launch_dense_matvec(j));
-            j.w = L.edown; j.pro = DPRO_EXPERTS; j.x = lm->ex; j.act = glu_act_of(L.d->ffn);
-            if (L.sdown.w) { j.shared = L.sdown; j.shared_x = lm->up; j.shared_gate = lm->up + L.u_sg; }
+            j.w = L.edown; j.pro = DPRO_EXPERTS; j.x = lm->ex; j.ldx = L.eup.n / 2;
+            if (L.sdown.w) { j.shared = L.sdown; j.shared_x = lm->hid; j.shared_gate = lm->up + L.u_sg; }
         } else {
-            j.w = L.down; j.x = lm->up; j.eps = eps;
+            j.w = L.down; j.x = L.act ? lm->up : lm->hid; j.eps = eps;
             if (L.act) { j.pro = DPRO_POLY; j.poly = L.act->f32(); }
-            else { j.pro = DPRO_GLU; j.act = glu_act_of(L.d->ffn); }
         }
         TLB_TRY(c.back(j, L, L.ls2, L.post2, L.u_rg2 >= 0 ? lm->up + L.u_rg2 : nullptr));
     }
@@ -842,7 +852,7 @@ uint64_t layered_state_bytes(const LayeredModel *lm, int ctx_len)
         switch (x.kind) {
         case MixerKind::Attention: b += seen * x.kv_heads * (x.dim + x.vdim) * es; break;
         case MixerKind::Latent: b += seen * (x.kv_rank + x.rot_dim) * es; break;
-        case MixerKind::MinGru: b += 2ull * x.width * 4; break;                            // read and written
+        case MixerKind::MinGru: b += 2ull * x.width * 4; break;                  // read and written
         default: b += 2ull * x.heads * x.vdim * mix_recur_ld(x.dim) * 4;
         }
     }
@@ -854,7 +864,7 @@ int layered_kernels_per_step(const LayeredModel *lm)
     int n = 1;
     for (const Layer &L : lm->layers) {
         const MixerDesc &x = L.d->mix;
-        n += x.kind == MixerKind::MinGru ? 2 : (x.kind == MixerKind::Latent ? (x.q_rank ? 6 : 5) : 3);
+        n += x.kind == MixerKind::Latent ? (x.q_rank ? 6 : 5) : 3;
         n += !L.up.w ? 0 : (L.eup.w ? 3 : 2);
     }
     return n;

@@ -14,6 +14,9 @@ struct DenseW {
     int n = 0, k = 0, ld = 0;
     const float *bias = nullptr;
     bool f16 = false;                     // w holds f16 instead of bf16 (GEMM over f16 rows only)
+    // The first `glu` rows (a multiple of 4) are gate and up rows of a gated activation: rows 4 i, 4 i + 1 gates and 4 i + 2, 4 i + 3
+    // ups of units 2 i, 2 i + 1.  They yield act(gate) * up of glu / 2 units to act_out; `out` holds the other rows, from 0.
+    int glu = 0, glu_act = 0;
 };
 inline int act_ld(int k) { return (k + 7) / 8 * 8; }   // pitch of an activation row that feeds a [.., k] weight
 
@@ -23,10 +26,8 @@ enum DensePro {
     DPRO_NORM = 1,      // x / rms * weight
     DPRO_POLY = 2,      // PolyNorm
     DPRO_GNORM = 3,     // residual step of the sublayer before, then the norm in groups
-    DPRO_GLU = 4,       // act(gate) * up
-    DPRO_GRU = 5,       // gated recurrence: new state * silu(gate)
-    DPRO_EXPERT = 6,    // plain x; the weight is the expert the router gave this launch's blockIdx.y
-    DPRO_EXPERTS = 7,   // act(gate) * up of the chosen experts and the shared one, each times its weight, side by side
+    DPRO_EXPERT = 4,    // plain x; the weight is the expert the router gave this launch's blockIdx.y
+    DPRO_EXPERTS = 5,   // activations of the chosen experts and the shared one, each times its weight, side by side
 };
 enum GluAct { GLU_SILU = 0, GLU_GELU_TANH = 1 };
 // Router of a mixture of experts: the `top` best of the experts of the `keep` best groups; weights are scores over their sum * scale.
@@ -52,14 +53,12 @@ struct DenseMatvecJob {
     int groups = 1;
     const float *y = nullptr, *y_gate = nullptr, *post_w = nullptr;
     float *h_out = nullptr;
-    int act = GLU_SILU;                   // GLU, EXPERTS: x = gate [k] | up [k]
-    // GRU: x = z | u | gate, each [k]; state of position p at state + (p & 1) * parity_stride, the next one in the other half
-    float *state = nullptr;
-    size_t parity_stride = 0;
-    const int *pos = nullptr;
-    // EXPERT: w.n rows per expert, experts stacked; slot s of the choice goes to out + s * w.n.  The choice is stored to sel / weight.
-    // EXPERTS: w [experts * w.n, ff]; x [top][2 ff]; the shared expert (shared.w may be null) has gate | up at shared_x and the logit
-    // of its weight at shared_gate (null: one)
+    float *act_out = nullptr;             // w.glu
+    // EXPERT: w.n rows per expert (all of them gated activations), experts stacked; slot s of the choice goes to act_out + s * w.n / 2.
+    // The choice is stored to sel / weight.
+    // EXPERTS: w [experts * w.n, ff]; x [top] rows of pitch ldx; the shared expert (shared.w may be null) has its activations at
+    // shared_x and the logit of its weight at shared_gate (null: one)
+    int ldx = 0;
     RouteDesc route;
     const float *logits = nullptr;
     int *sel = nullptr;
@@ -81,10 +80,13 @@ struct DenseGemmJob {
     int ldo = 0;
     const float *resid_scale = nullptr;   // out[t][i] += resid_scale[i] * y instead of out = y + bias
     float softcap = 0.f;
-    // columns in blocks of `per` (0: all), block b at out + b * block_stride; out_h: f16 output at the same places
+    // columns in blocks of `per` (0: all), block b at out + b * block_stride; out_h: f16 output at the same places; out_t: f16 output
+    // transposed, column c of block b at out_t + b * block_stride + c * ldo, zeros behind the last row up to a multiple of 128
     int per = 0;
     size_t block_stride = 0;
-    __half *out_h = nullptr;
+    __half *out_h = nullptr, *out_t = nullptr;
+    void *act_out = nullptr;              // w.glu: rows in the activation type, pitch ld_act
+    int ld_act = 0;
     // several weights [.., k] of w.n rows each, stacked: tile i covers rows y .. y + z - 1 of x and multiplies them with weight x
     const int4 *tiles = nullptr;
     int n_tiles = 0, tile_rows = 0, n_weights = 1;
@@ -98,11 +100,11 @@ tlb_status launch_poly_rows(const float *z, int T, int ff, int ldz, const float 
 tlb_status launch_embed_bf16(const int *tokens, const __nv_bfloat16 *table, int width, int ld, float *x, int T);
 tlb_status launch_gather_rows(const float *x, int width, const int *idx, int n, float *out);
 tlb_status launch_pack_rows(const __nv_bfloat16 *src, int n, int k, __nv_bfloat16 *dst, int ld, int col0);
+// rows of a gated activation's gate (up: false) or up matrix to their places among the pairs (DenseW::glu)
+tlb_status launch_pack_glu_rows(const __nv_bfloat16 *src, int ff, int k, __nv_bfloat16 *dst, int ld, bool up);
 tlb_status launch_pack_rows_f16(const __nv_bfloat16 *src, int n, int k, void *dst, int ld);      // values as f16
 
 // ---------------------------------------------------------------- row_kernels.cu
-// act(gate) * up of rows z: gate at column 0, up at column ff
-tlb_status launch_glu_rows(const float *z, int T, int ff, int ldz, int act, void *out, int ld, bool f32);
 // What a mixture of experts leaves per token: y = sum over the choice of weight * part[slot] + sigmoid(shared_gate) * shared.
 struct MoeRows {
     int top = 0;
@@ -158,6 +160,9 @@ struct MixAttn {
     int ldp;
     const float *gate;                    // prompts: [T, ld_gate] logits of a gate on every output element, or null
     int ld_gate;
+    // tcgen05 prompt kernel, instead of proj and vcache: queries [T][H * mix_attn_tc5_qd(D)] padded with zeros, V^T [KVH][128][vt_ld]
+    const __half *q16, *vt;
+    int vt_ld;
 };
 // One new token per sequence (rows of proj), at *pos: append and attend.  out: rows of H * DV in the activation type (out_f32: f32), pitch ldo.
 struct MixAttnDecode {
@@ -180,6 +185,7 @@ tlb_status launch_mix_attn_prefill_tc(const MixAttn &a, int seq, int T, int pos0
 bool mix_attn_prefill_tc_supported(int D, int DV);
 tlb_status launch_mix_attn_prefill_tc5(const MixAttn &a, int seq, int T, int pos0, void *out, int ldo);  // prefill_attn_tc.cu: f16 cache, tcgen05
 bool mix_attn_prefill_tc5_supported(int D, int DV, int T);
+inline int mix_attn_tc5_qd(int D) { return D > 128 ? 192 : 128; }
 
 // ---------------------------------------------------------------- mix_recurrent.cu
 // Linear recurrences with a matrix state per head, S[value channel][key channel] (key channels padded to ld), f32.
@@ -264,15 +270,13 @@ tlb_status launch_latent_prompt(const MixLatent &m, int seq, int T, int pos0, in
 
 // ---------------------------------------------------------------- mix_gru.cu
 // Gated recurrence per channel, S <- (1 - z) S + z candidate(u); rows z | u | gate logits, each `width` wide; out = S * silu(gate).
-// The state of a sequence at position p lies at state + (p & 1) * parity_stride.
 struct MixGru {
     int width;
-    float *state;                         // [2][seq][width]
-    size_t parity_stride;
+    float *state;                         // [seq][width]
     const float *proj;
     int ldp;
 };
-tlb_status launch_gru_rows(const MixGru &m, int batch, const int *pos, void *out, int ldo, bool f32);
+tlb_status launch_gru_rows(const MixGru &m, int batch, const int *pos, void *out, int ldo, bool out_f32, bool pdl);
 tlb_status launch_gru_prefill(const MixGru &m, int seq, int T, int pos0, void *out, int ldo, bool f32);
 
 // launch with programmatic dependent launch (the kernel calls griddepcontrol.wait before it touches what precedes it)

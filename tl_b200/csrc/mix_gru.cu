@@ -2,15 +2,15 @@
 //   S_t = (1 - z) S_(t-1) + z candidate(u),  out = S_t * silu(gate)
 // A prompt is a linear recurrence with known coefficients: a CTA owns 32 channels (a lane each), its warps take consecutive runs of
 // tokens, compose their steps into one (factor, term) pair, and every warp starts from the state the runs before it leave.
-// One token at a time runs inside the output projection's matvec (DPRO_GRU); rows of a batch here.
 #include "act.cuh"
 #include "layered_kernels.h"
+#include "qmv_common.cuh"
 
 namespace tlb {
 
 namespace {
 
-constexpr int kGruWarps = 16, kGruRun = 8, kGruTile = kGruWarps * kGruRun;
+constexpr int kGruWarps = 32, kGruRun = 4, kGruTile = kGruWarps * kGruRun;
 
 template <typename TO>
 __global__ void __launch_bounds__(kGruWarps * 32) gru_scan_kernel(const MixGru m, int seq, int T, int pos0, TO *__restrict__ out, int ldo)
@@ -19,7 +19,7 @@ __global__ void __launch_bounds__(kGruWarps * 32) gru_scan_kernel(const MixGru m
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, c = blockIdx.x * 32 + lane;
     const bool live = c < m.width;
     const float *pz = m.proj + c, *pu = pz + m.width, *pg = pu + m.width;
-    float state = live && pos0 > 0 ? m.state[(size_t)(pos0 & 1) * m.parity_stride + (size_t)seq * m.width + c] : 0.f;
+    float state = live && pos0 > 0 ? m.state[(size_t)seq * m.width + c] : 0.f;
     float z[kGruRun], u[kGruRun], g[kGruRun];
     auto fetch = [&](int t0) {
 #pragma unroll
@@ -61,21 +61,23 @@ __global__ void __launch_bounds__(kGruWarps * 32) gru_scan_kernel(const MixGru m
             if (live && t < T) store_actv(out + (size_t)t * ldo + c, mine * w[i]);
         }
     }
-    if (live && warp == 0) m.state[(size_t)((pos0 + T) & 1) * m.parity_stride + (size_t)seq * m.width + c] = state;
+    if (live && warp == 0) m.state[(size_t)seq * m.width + c] = state;
 }
 
 template <typename TO>
-__global__ void __launch_bounds__(256) gru_rows_kernel(const MixGru m, const int *__restrict__ pos, TO *__restrict__ out, int ldo)
+__global__ void __launch_bounds__(128) gru_rows_kernel(const MixGru m, const int *__restrict__ pos, TO *__restrict__ out, int ldo)
 {
-    const int c = blockIdx.x * 256 + threadIdx.x, b = blockIdx.y;
-    if (c >= m.width) return;
-    const int p = pos[b];
-    const float *row = m.proj + (size_t)b * m.ldp;
-    const size_t at = (size_t)b * m.width + c;
-    const float z = sigmoidf(row[c]), old = p > 0 ? m.state[(size_t)(p & 1) * m.parity_stride + at] : 0.f;
-    const float st = (1.f - z) * old + z * gru_candidate(row[m.width + c]);
-    m.state[(size_t)((p & 1) ^ 1) * m.parity_stride + at] = st;
-    store_actv(out + (size_t)b * ldo + c, st * siluf(row[2 * m.width + c]));
+    const int c = blockIdx.x * 128 + threadIdx.x, b = blockIdx.y;
+    const bool live = c < m.width;
+    float *s = m.state + (size_t)b * m.width + c;
+    const float old = live && __ldcg(pos + b) > 0 ? *s : 0.f;       // both left by launches of an earlier step
+    pdl_wait();
+    pdl_launch_dependents();
+    if (!live) return;
+    const float *row = m.proj + (size_t)b * m.ldp + c;
+    const float z = sigmoidf(__ldcg(row)), st = (1.f - z) * old + z * gru_candidate(__ldcg(row + m.width));
+    *s = st;
+    store_actv(out + (size_t)b * ldo + c, st * siluf(__ldcg(row + 2 * m.width)));
 }
 
 tlb_status launched(const char *what)
@@ -88,12 +90,13 @@ tlb_status launched(const char *what)
 
 }  // namespace
 
-tlb_status launch_gru_rows(const MixGru &m, int batch, const int *pos, void *out, int ldo, bool f32)
+tlb_status launch_gru_rows(const MixGru &m, int batch, const int *pos, void *out, int ldo, bool out_f32, bool pdl)
 {
-    const dim3 grid((m.width + 255) / 256, batch);
-    if (f32) gru_rows_kernel<<<grid, 256, 0, ctx()->stream>>>(m, pos, (float *)out, ldo);
-    else gru_rows_kernel<<<grid, 256, 0, ctx()->stream>>>(m, pos, (__nv_bfloat16 *)out, ldo);
-    return launched("gated recurrence launch");
+    const dim3 grid((m.width + 127) / 128, batch);
+    if (out_f32) TLB_CUDA(launch_chained(gru_rows_kernel<float>, grid, dim3(128), 0, pdl, m, pos, (float *)out, ldo));
+    else TLB_CUDA(launch_chained(gru_rows_kernel<__nv_bfloat16>, grid, dim3(128), 0, pdl, m, pos, (__nv_bfloat16 *)out, ldo));
+    count_launch();
+    return TLB_OK;
 }
 
 tlb_status launch_gru_prefill(const MixGru &m, int seq, int T, int pos0, void *out, int ldo, bool f32)

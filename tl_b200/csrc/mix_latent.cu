@@ -10,6 +10,7 @@
 // Long portions expand the visible latents to keys and values (two GEMMs over cache rows) and take the prompt attention.
 // Scores, softmax weights (two f16 terms, value and remainder, on the tensor cores) and sums are 32-bit.
 #include <algorithm>
+#include <vector>
 
 #include "act.cuh"
 #include "layered_kernels.h"
@@ -371,9 +372,14 @@ __global__ void __launch_bounds__(kThreads) latent_value_kernel(const MixLatentR
 #pragma unroll
     for (int r = 0; r < 4; r++) {
         w[r] = m.uv.w + ((size_t)h * m.DV + min(j0 + r, m.DV - 1)) * m.uv.ld;
-        for (int e = lane * 64; e < m.uv.ld; e += 32 * 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(w[r] + e));
+        for (int e = 512 + lane * 64; e < m.uv.ld; e += 32 * 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(w[r] + e));
     }
     const Cut cut = cut_keys(row_pos(j, row), m.window, max_split);
+    uint4 pre[4][2];                                         // the weights' first 512 columns, ahead of the wait
+#pragma unroll
+    for (int r = 0; r < 4; r++)
+#pragma unroll
+        for (int i = 0; i < 2; i++) pre[r][i] = lane + 32 * i < nv ? *reinterpret_cast<const uint4 *>(w[r] + (lane + 32 * i) * 8) : make_uint4(0u, 0u, 0u, 0u);
     pdl_wait();
     pdl_launch_dependents();
     const int prow = part_row(m.R);
@@ -427,18 +433,29 @@ __global__ void __launch_bounds__(kThreads) latent_value_kernel(const MixLatentR
     for (int e = m.R + tid; e < (m.uv.ld + 3) / 4 * 4; e += kThreads) so[e] = 0.f;       // the weight's padding meets zeros
     __syncthreads();
     float acc[4] = {};
-    for (int v = lane; v < nv; v += 32) {
+    auto mul = [&](int v, const uint4 (&x)[4]) {
         const float4 a = *reinterpret_cast<const float4 *>(so + v * 8), b = *reinterpret_cast<const float4 *>(so + v * 8 + 4);
 #pragma unroll
         for (int r = 0; r < 4; r++) {
-            const uint4 x = *reinterpret_cast<const uint4 *>(w[r] + v * 8);
             float s = acc[r];
-            s = fmaf(bf_lo(x.x), a.x, s); s = fmaf(bf_hi(x.x), a.y, s);
-            s = fmaf(bf_lo(x.y), a.z, s); s = fmaf(bf_hi(x.y), a.w, s);
-            s = fmaf(bf_lo(x.z), b.x, s); s = fmaf(bf_hi(x.z), b.y, s);
-            s = fmaf(bf_lo(x.w), b.z, s); s = fmaf(bf_hi(x.w), b.w, s);
+            s = fmaf(bf_lo(x[r].x), a.x, s); s = fmaf(bf_hi(x[r].x), a.y, s);
+            s = fmaf(bf_lo(x[r].y), a.z, s); s = fmaf(bf_hi(x[r].y), a.w, s);
+            s = fmaf(bf_lo(x[r].z), b.x, s); s = fmaf(bf_hi(x[r].z), b.y, s);
+            s = fmaf(bf_lo(x[r].w), b.z, s); s = fmaf(bf_hi(x[r].w), b.w, s);
             acc[r] = s;
         }
+    };
+#pragma unroll
+    for (int i = 0; i < 2; i++)
+        if (lane + 32 * i < nv) {
+            const uint4 x[4] = {pre[0][i], pre[1][i], pre[2][i], pre[3][i]};
+            mul(lane + 32 * i, x);
+        }
+    for (int v = lane + 64; v < nv; v += 32) {
+        uint4 x[4];
+#pragma unroll
+        for (int r = 0; r < 4; r++) x[r] = *reinterpret_cast<const uint4 *>(w[r] + v * 8);
+        mul(v, x);
     }
 #pragma unroll
     for (int r = 0; r < 4; r++) acc[r] = warp_sum(acc[r]);
@@ -451,20 +468,32 @@ __global__ void __launch_bounds__(kThreads) latent_value_kernel(const MixLatentR
 }
 
 // ================================================================ long portions
-// rotates the queries of a token in place and appends its cache row
+// rotates the queries of a token in place (or, with q16, into f16 rows whose heads are padded to qd) and appends its cache row
 template <typename CT>
-__global__ void __launch_bounds__(kThreads) latent_prep_kernel(const MixLatent m, int seq, int pos0, int rope0, int rope_step)
+__global__ void __launch_bounds__(kThreads) latent_prep_kernel(const MixLatent m, int seq, int pos0, int rope0, int rope_step, __half *__restrict__ q16, int qd)
 {
     __shared__ float part[kWarps], inv[1];
     const int t = blockIdx.x, rope = rope0 + t * rope_step, half = m.rot / 2, hd = m.D + m.RD;
     const float *c = m.rot_cos + (size_t)rope * half, *s = m.rot_sin + (size_t)rope * half;
     float *q = m.q + (size_t)t * m.ldq;
-    for (int i = threadIdx.x; i < m.H * half; i += kThreads) {
-        const int h = i / half, k = i - h * half;
-        float *x = q + (size_t)h * hd + m.D + 2 * k;
-        const float u = x[0], v = x[1];
-        x[0] = u * c[k] - v * s[k];
-        x[1] = v * c[k] + u * s[k];
+    if (q16) {
+        __half2 *dst = reinterpret_cast<__half2 *>(q16 + (size_t)t * m.H * qd);
+        auto value = [&](const float *x, int d) { return d < m.D ? __ldcg(x + d) : (d < hd ? turned(x + m.D, d - m.D, m.rot, c, s) : 0.f); };
+        auto clamp = [](float v) { return fminf(fmaxf(v, -65504.f), 65504.f); };
+#pragma unroll 4
+        for (int i = threadIdx.x; i < m.H * qd / 2; i += kThreads) {
+            const int h = i / (qd / 2), d = (i - h * (qd / 2)) * 2;
+            const float *x = q + (size_t)h * hd;
+            dst[i] = __floats2half2_rn(clamp(value(x, d)), clamp(value(x, d + 1)));
+        }
+    } else {
+        for (int i = threadIdx.x; i < m.H * half; i += kThreads) {
+            const int h = i / half, k = i - h * half;
+            float *x = q + (size_t)h * hd + m.D + 2 * k;
+            const float u = x[0], v = x[1];
+            x[0] = u * c[k] - v * s[k];
+            x[1] = v * c[k] + u * s[k];
+        }
     }
     append_row<CT>(m, seq, pos0 + t, rope, m.kv + (size_t)t * m.ldkv, part, inv);
 }
@@ -510,14 +539,17 @@ template <typename CT, int RT>
 tlb_status run_query(const MixLatentRows &j)
 {
     const MixLatent &m = j.m;
-    const int vecs = m.uk.ld / 8, tc = vecs > 32 ? 64 : (vecs > 16 ? 32 : (vecs > 8 ? 16 : 8));
+    // few rows: narrow column chunks, so that a thread has all its weights in flight at once
+    const int vecs = m.uk.ld / 8, tiles = (j.rows + RT - 1) / RT;
+    int tc = 8;
+    while (tc < 64 && tc < vecs && (vecs / tc) * m.H * tiles > 4 * ctx()->sm_count) tc *= 2;
     const size_t smem = ((size_t)(RT * m.D + 3) / 4 * 4 + (size_t)kThreads * RT * 8) * sizeof(float);
     static size_t allowed = 48 << 10;
     if (smem > allowed) {
         TLB_CUDA(cudaFuncSetAttribute(latent_query_kernel<CT, RT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         allowed = smem;
     }
-    TLB_CUDA(launch_chained(latent_query_kernel<CT, RT>, dim3((vecs + tc - 1) / tc, m.H + 1, (j.rows + RT - 1) / RT), dim3(kThreads), smem, j.pdl, j, tc));
+    TLB_CUDA(launch_chained(latent_query_kernel<CT, RT>, dim3((vecs + tc - 1) / tc, m.H + 1, tiles), dim3(kThreads), smem, j.pdl, j, tc));
     count_launch();
     return TLB_OK;
 }
@@ -580,36 +612,49 @@ tlb_status launch_latent_prompt(const MixLatent &m, int seq, int T, int pos0, in
     Context *c = ctx();
     if (!c) return TLB_ERR_DEVICE;
     const size_t es = f32 ? 4 : 2;
-    if (f32) latent_prep_kernel<float><<<T, kThreads, 0, c->stream>>>(m, seq, pos0, rope0, rope_step);
-    else latent_prep_kernel<__half><<<T, kThreads, 0, c->stream>>>(m, seq, pos0, rope0, rope_step);
-    TLB_CUDA(cudaGetLastError());
-    count_launch();
     // the latents some query sees, from a tile border of the prompt attention on, as keys and values per head
     const int key_first = std::max(0, pos0 - m.window + 1) / 128 * 128, n_keys = pos0 + T - key_first;
-    const int hd = m.D + m.RD, ldk = act_ld(hd), ldv = act_ld(m.DV);
-    Storage *ks = storage_alloc((size_t)m.H * n_keys * ldk * es), *vs = storage_alloc((size_t)m.H * n_keys * ldv * es);
-    auto done = [&](tlb_status st) { if (ks) storage_release(ks); if (vs) storage_release(vs); return st; };
-    if (!ks || !vs) return done(TLB_ERR_ALLOC);
-    const char *cache = (const char *)m.cache + ((size_t)seq * m.seq_stride + (size_t)key_first * m.ld) * es;
-    auto expand = [&](const DenseW &w, Storage *dst, int per, int ld) {
-        DenseGemmJob j;
-        j.w = w; j.x = cache; j.ldx = m.ld; j.T = n_keys; j.ldo = ld; j.per = per; j.block_stride = (size_t)n_keys * ld;
-        if (f32) j.out = (float *)dst->ptr;
-        else j.out_h = (__half *)dst->ptr;
-        return launch_dense_gemm(j, f32);
+    const int hd = m.D + m.RD, ldk = act_ld(hd), ldv = act_ld(m.DV), qd = mix_attn_tc5_qd(hd), vt_ld = (n_keys + 127) / 128 * 128;
+    // the tcgen05 kernel takes f16 queries and V^T, which the kernels here write at once
+    const bool tc5 = !f32 && mix_attn_prefill_tc5_supported(hd, m.DV, T);
+    std::vector<Storage *> held;
+    auto done = [&](tlb_status st) { for (Storage *s : held) storage_release(s); return st; };
+    auto get = [&](size_t bytes) -> void * {
+        Storage *s = storage_alloc(bytes);
+        if (!s) return nullptr;
+        held.push_back(s);
+        return s->ptr;
     };
-    tlb_status st = expand(f32 ? m.uk : m.uk16, ks, m.D, ldk);
-    if (st == TLB_OK) st = expand(f32 ? m.uv : m.uv16, vs, m.DV, ldv);
-    if (st != TLB_OK) return done(st);
-    if (f32) latent_rot_kernel<float><<<n_keys, kThreads, 0, c->stream>>>(m, (const float *)cache, (float *)ks->ptr, n_keys, ldk);
-    else latent_rot_kernel<__half><<<n_keys, kThreads, 0, c->stream>>>(m, (const __half *)cache, (__half *)ks->ptr, n_keys, ldk);
+    void *keys = get((size_t)m.H * n_keys * ldk * es), *vals = get((size_t)m.H * (tc5 ? (size_t)128 * vt_ld : (size_t)n_keys * ldv) * es);
+    __half *q16 = tc5 ? (__half *)get((size_t)T * m.H * qd * 2) : nullptr;
+    if (!keys || !vals || (tc5 && !q16)) return done(TLB_ERR_ALLOC);
+    if (f32) latent_prep_kernel<float><<<T, kThreads, 0, c->stream>>>(m, seq, pos0, rope0, rope_step, nullptr, 0);
+    else latent_prep_kernel<__half><<<T, kThreads, 0, c->stream>>>(m, seq, pos0, rope0, rope_step, q16, qd);
     cudaError_t e = cudaGetLastError();
+    if (e != cudaSuccess) return done(cuda_fail(e, "latent preparation launch"));
+    const char *cache = (const char *)m.cache + ((size_t)seq * m.seq_stride + (size_t)key_first * m.ld) * es;
+    DenseGemmJob j;
+    j.x = cache; j.ldx = m.ld; j.T = n_keys;
+    j.w = f32 ? m.uk : m.uk16; j.per = m.D; j.ldo = ldk; j.block_stride = (size_t)n_keys * ldk;
+    (f32 ? (void *&)j.out : (void *&)j.out_h) = keys;
+    tlb_status st = launch_dense_gemm(j, f32);
+    if (st != TLB_OK) return done(st);
+    j.out = nullptr; j.out_h = nullptr;
+    j.w = f32 ? m.uv : m.uv16; j.per = m.DV;
+    if (tc5) { j.out_t = (__half *)vals; j.ldo = vt_ld; j.block_stride = (size_t)128 * vt_ld; }
+    else { (f32 ? (void *&)j.out : (void *&)j.out_h) = vals; j.ldo = ldv; j.block_stride = (size_t)n_keys * ldv; }
+    st = launch_dense_gemm(j, f32);
+    if (st != TLB_OK) return done(st);
+    if (f32) latent_rot_kernel<float><<<n_keys, kThreads, 0, c->stream>>>(m, (const float *)cache, (float *)keys, n_keys, ldk);
+    else latent_rot_kernel<__half><<<n_keys, kThreads, 0, c->stream>>>(m, (const __half *)cache, (__half *)keys, n_keys, ldk);
+    e = cudaGetLastError();
     if (e != cudaSuccess) return done(cuda_fail(e, "latent expansion launch"));
-    count_launch();
+    count_launch(2);
     MixAttn a = {};
     a.H = a.KVH = m.H; a.D = hd; a.DV = m.DV; a.ldk = ldk; a.ldv = ldv; a.max_seq = n_keys; a.window = m.window; a.scale = m.scale;
     a.bias_n = 1;
-    a.kcache = ks->ptr; a.vcache = vs->ptr; a.proj = m.q; a.ldp = m.ldq; a.gate = m.gate; a.ld_gate = m.ld_gate;
+    a.kcache = keys; a.vcache = vals; a.proj = m.q; a.ldp = m.ldq; a.gate = m.gate; a.ld_gate = m.ld_gate;
+    if (tc5) { a.q16 = q16; a.vt = (const __half *)vals; a.vt_ld = vt_ld; }
     return done(launch_mix_attn_prompt(a, 0, T, pos0 - key_first, out, ldo, f32));
 }
 

@@ -199,6 +199,19 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __gr
         // ------------------------------------------------ write-out: O / l
         if (ok && mbar_wait(o_full, (uint32_t)(n_tiles - 1) & 1u, abort_flag, p.err, 43)) {
             tc_fence_after();
+            // The gate of the warp's 32 rows goes through shared memory (the tiles are no longer read: every product has ended), so
+            // that its rows are read whole.
+            constexpr int kGatePitch = kAtD + 4;
+            float *s_gate = reinterpret_cast<float *>(at_smem + (sK - smem_u32(at_smem))) + warp * 32 * kGatePitch;
+            if (MIX && p.gate) {
+                const float *gt = p.gate + (size_t)(q0 + warp * 32) * p.ld_gate + (size_t)h * p.DV;
+                const int nr = min(32, p.T - (q0 + warp * 32));
+                for (int c = lane; c < p.DV; c += 32) {
+#pragma unroll 16
+                    for (int r = 0; r < nr; r++) s_gate[r * kGatePitch + c] = sigmoidf(__ldg(gt + (size_t)r * p.ld_gate + c));
+                }
+                __syncwarp();
+            }
             const float inv = 1.f / l_run;
             float *dst = p.out + (size_t)q * (p.H * kAtD) + h * kAtD;
 #pragma unroll
@@ -210,10 +223,15 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __gr
                     if (q < p.T) {
                         __nv_bfloat16 *d16 = p.out16 + (size_t)q * p.ldo + (size_t)h * p.DV + c * 32;
                         if (p.gate) {
-                            const float *gt = p.gate + (size_t)q * p.ld_gate + (size_t)h * p.DV + c * 32;
+                            const float4 *gt = reinterpret_cast<const float4 *>(s_gate + lane * kGatePitch + c * 32);
 #pragma unroll
-                            for (int i = 0; i < 32; i++)
-                                if (c * 32 + i < p.DV) o[i] = __float_as_uint(__uint_as_float(o[i]) * sigmoidf(gt[i]));
+                            for (int i = 0; i < 32; i += 4) {
+                                const float4 g = gt[i / 4];               // columns past DV: never stored
+                                o[i] = __float_as_uint(__uint_as_float(o[i]) * g.x);
+                                o[i + 1] = __float_as_uint(__uint_as_float(o[i + 1]) * g.y);
+                                o[i + 2] = __float_as_uint(__uint_as_float(o[i + 2]) * g.z);
+                                o[i + 3] = __float_as_uint(__uint_as_float(o[i + 3]) * g.w);
+                            }
                         }
                         if (p.DV % 8 == 0 && p.ldo % 8 == 0) {
 #pragma unroll
@@ -384,20 +402,30 @@ tlb_status run_mix_tc5(const MixAttn &a, int seq, int T, int pos0, void *out, in
 {
     Context *c = ctx();
     constexpr int QD = KB * 64;
-    // cache rows some query sees, from a tile border on
-    const int key_first = std::max(0, pos0 - a.window + 1) / kAtK * kAtK, n_keys = pos0 + T - key_first, keys_ld = (n_keys + 127) / 128 * 128;
-    Storage *qh = storage_alloc((size_t)T * a.H * QD * sizeof(__half));
-    Storage *vt = storage_alloc((size_t)a.KVH * kAtD * keys_ld * sizeof(__half));
-    if (!qh || !vt) { if (qh) storage_release(qh); if (vt) storage_release(vt); return TLB_ERR_ALLOC; }
-    auto done = [&](tlb_status st) { storage_release(qh); storage_release(vt); return st; };
+    // cache rows some query sees, from a tile border on; V^T that is given starts with row 0
+    const int key_first = a.vt ? 0 : std::max(0, pos0 - a.window + 1) / kAtK * kAtK, n_keys = pos0 + T - key_first, keys_ld = a.vt ? a.vt_ld : (n_keys + 127) / 128 * 128;
+    Storage *qh = nullptr, *vt = nullptr;
+    auto done = [&](tlb_status st) { if (qh) storage_release(qh); if (vt) storage_release(vt); return st; };
     const __half *kc = (const __half *)a.kcache + (size_t)seq * a.seq_stride_k, *vc = (const __half *)a.vcache + (size_t)seq * a.seq_stride_v;
-    mix_q_to_f16_kernel<QD><<<T, 256, 0, c->stream>>>(a.proj, a.ldp, a.H, a.D, (__half *)qh->ptr);
-    mix_v_transpose_kernel<<<dim3(kAtD / 32, (unsigned)(keys_ld / 32), (unsigned)a.KVH), 256, 0, c->stream>>>(vc, (__half *)vt->ptr, a.max_seq, a.ldv, key_first, n_keys, keys_ld);
-    count_launch(2);
+    const void *q16 = a.q16, *v16 = a.vt;
+    if (!q16) {
+        qh = storage_alloc((size_t)T * a.H * QD * sizeof(__half));
+        if (!qh) return done(TLB_ERR_ALLOC);
+        mix_q_to_f16_kernel<QD><<<T, 256, 0, c->stream>>>(a.proj, a.ldp, a.H, a.D, (__half *)qh->ptr);
+        count_launch();
+        q16 = qh->ptr;
+    }
+    if (!v16) {
+        vt = storage_alloc((size_t)a.KVH * kAtD * keys_ld * sizeof(__half));
+        if (!vt) return done(TLB_ERR_ALLOC);
+        mix_v_transpose_kernel<<<dim3(kAtD / 32, (unsigned)(keys_ld / 32), (unsigned)a.KVH), 256, 0, c->stream>>>(vc, (__half *)vt->ptr, a.max_seq, a.ldv, key_first, n_keys, keys_ld);
+        count_launch();
+        v16 = vt->ptr;
+    }
     CUtensorMap qmap, kmap, vtmap;
-    if (!encode_f16_map(&qmap, qh->ptr, (uint64_t)a.H * QD, (uint64_t)T, (uint64_t)a.H * QD * 2, 64, 128) ||
+    if (!encode_f16_map(&qmap, q16, (uint64_t)a.H * QD, (uint64_t)T, (uint64_t)a.H * QD * 2, 64, 128) ||
         !encode_f16_map(&kmap, kc, (uint64_t)a.ldk, (uint64_t)a.KVH * a.max_seq, (uint64_t)a.ldk * 2, 64, 128) ||
-        !encode_f16_map(&vtmap, vt->ptr, (uint64_t)keys_ld, (uint64_t)a.KVH * kAtD, (uint64_t)keys_ld * 2, 64, 128))
+        !encode_f16_map(&vtmap, v16, (uint64_t)keys_ld, (uint64_t)a.KVH * kAtD, (uint64_t)keys_ld * 2, 64, 128))
         return done(fail(TLB_ERR_DEVICE, "prompt attention: cuTensorMapEncodeTiled failed or is not available"));
     AtParams p = {};
     p.T = T; p.H = a.H; p.KVH = a.KVH; p.max_seq = a.max_seq; p.pos0 = pos0; p.vt_rows = keys_ld;

@@ -1,5 +1,5 @@
-// Row kernels of layered models: gated activations, and the residual step of designs that norm what a sublayer adds - gate, norm
-// in groups, addition and the next sublayer's norm in one pass over the row.
+// Row kernels of layered models: norms of part of a row, and the residual step of designs that norm what a sublayer adds - gate,
+// norm in groups, addition and the next sublayer's norm in one pass over the row.
 #include <algorithm>
 
 #include "act.cuh"
@@ -8,21 +8,6 @@
 namespace tlb {
 
 namespace {
-
-template <typename TA>
-__global__ void __launch_bounds__(256) glu_rows_kernel(const float *__restrict__ z, int ff, int ldz, int act, TA *__restrict__ out, int ld)
-{
-    const float *row = z + (size_t)blockIdx.x * ldz;
-    TA *o = out + (size_t)blockIdx.x * ld;
-    const int e = (blockIdx.y * 256 + threadIdx.x) * 4;
-    if (e >= ff) return;
-    if (ff % 4 == 0 && ldz % 4 == 0 && (reinterpret_cast<uintptr_t>(z) & 15) == 0) {
-        const float4 g = *reinterpret_cast<const float4 *>(row + e), u = *reinterpret_cast<const float4 *>(row + ff + e);
-        store_actv4(o + e, glu_act(act, g.x, u.x), glu_act(act, g.y, u.y), glu_act(act, g.z, u.z), glu_act(act, g.w, u.w));
-        return;
-    }
-    for (int i = e; i < min(e + 4, ff); i++) store_actv(o + i, glu_act(act, row[i], row[ff + i]));
-}
 
 template <typename TA>
 __global__ void __launch_bounds__(256) rms_cols_kernel(const float *__restrict__ x, int n, int ldx, const float *__restrict__ w, float eps, TA *__restrict__ out, int ld)
@@ -52,6 +37,7 @@ __global__ void __launch_bounds__(256) resid_norm_rows_kernel(const ResidNormPar
     __shared__ int s_slot[kMaxTop];
     __shared__ float s_w[kMaxTop];
     const int tid = threadIdx.x, W = p.width, len = W / p.groups;
+    const float inv_len = 1.f / (float)len;
     const size_t t = blockIdx.x;
     float *x = p.x + t * W;
     const bool v4 = W % 4 == 0 && len % 4 == 0;
@@ -98,7 +84,7 @@ __global__ void __launch_bounds__(256) resid_norm_rows_kernel(const ResidNormPar
         group_inv_rms(at, W, p.groups, p.eps, part, inv);
         if (v4) {
             for (int e = tid * 4; e < W; e += 1024) {
-                const float f = inv[e / len];
+                const float f = inv[group_of(e, inv_len)];
                 const float4 a = *reinterpret_cast<const float4 *>(row + e), w = *reinterpret_cast<const float4 *>(p.post_w + e);
                 float4 v = *reinterpret_cast<const float4 *>(x + e);
                 v.x += a.x * f * (w.x + p.offset); v.y += a.y * f * (w.y + p.offset); v.z += a.z * f * (w.z + p.offset); v.w += a.w * f * (w.w + p.offset);
@@ -106,7 +92,7 @@ __global__ void __launch_bounds__(256) resid_norm_rows_kernel(const ResidNormPar
                 *reinterpret_cast<float4 *>(row + e) = v;
             }
         } else {
-            for (int e = tid; e < W; e += 256) x[e] = row[e] = x[e] + row[e] * inv[e / len] * (p.post_w[e] + p.offset);
+            for (int e = tid; e < W; e += 256) x[e] = row[e] = x[e] + row[e] * inv[group_of(e, inv_len)] * (p.post_w[e] + p.offset);
         }
     } else {
         for (int e = tid; e < W; e += 256) row[e] = x[e];
@@ -117,12 +103,12 @@ __global__ void __launch_bounds__(256) resid_norm_rows_kernel(const ResidNormPar
     TA *o = out + t * p.ldo;
     if (v4 && p.ldo % 4 == 0) {
         for (int e = tid * 4; e < W; e += 1024) {
-            const float f = inv[e / len];
+            const float f = inv[group_of(e, inv_len)];
             const float4 a = *reinterpret_cast<const float4 *>(row + e), w = *reinterpret_cast<const float4 *>(p.norm_w + e);
             store_actv4(o + e, a.x * f * (w.x + p.offset), a.y * f * (w.y + p.offset), a.z * f * (w.z + p.offset), a.w * f * (w.w + p.offset));
         }
     } else {
-        for (int e = tid; e < W; e += 256) store_actv(o + e, row[e] * inv[e / len] * (p.norm_w[e] + p.offset));
+        for (int e = tid; e < W; e += 256) store_actv(o + e, row[e] * inv[group_of(e, inv_len)] * (p.norm_w[e] + p.offset));
     }
 }
 
@@ -148,14 +134,6 @@ tlb_status run_resid(const ResidNormParams &p, int T, void *out)
 }
 
 }  // namespace
-
-tlb_status launch_glu_rows(const float *z, int T, int ff, int ldz, int act, void *out, int ld, bool f32)
-{
-    const dim3 grid(T, (ff + 1023) / 1024);
-    if (f32) glu_rows_kernel<<<grid, 256, 0, ctx()->stream>>>(z, ff, ldz, act, (float *)out, ld);
-    else glu_rows_kernel<<<grid, 256, 0, ctx()->stream>>>(z, ff, ldz, act, (__nv_bfloat16 *)out, ld);
-    return launched("gated activation launch");
-}
 
 tlb_status launch_rms_cols(const float *x, int T, int n, int ldx, const float *w, float eps, void *out, int ld, bool f32)
 {
