@@ -123,9 +123,9 @@ def test_mixer_alone(name, f32):
 
 
 FFNS = {
-    "dense": dense(), "dense_1": dense(1), "dense_1030": dense(1030), "moe": moe(), "moe_no_groups": moe(groups=None), "moe_one_group": moe(groups=(1, 1)),
+    "dense": dense(), "dense_1": dense(1), "dense_1030": dense(1030), "dense_12200": dense(12200), "moe": moe(), "moe_no_groups": moe(groups=None), "moe_one_group": moe(groups=(1, 1)),
     "moe_groups_of_one": moe(6, 2, groups=(6, 4)), "moe_keeps_all": moe(8, 3, groups=(4, 4)), "moe_keeps_one": moe(14, 4, groups=(2, 1)), "moe_top_1": moe(7, 1, groups=None),
-    "moe_every_expert": moe(4, 4, groups=(2, 2)), "moe_one_expert": moe(1, 1, groups=None), "moe_no_shared": moe(shared=None), "moe_sizes": moe(40, 6, 260, (8, 3), 2.5, 300), "moe_ff_1": moe(5, 2, 1, None, 1.0, 1)}
+    "moe_every_expert": moe(4, 4, groups=(2, 2)), "moe_one_expert": moe(1, 1, groups=None), "moe_no_shared": moe(shared=None), "moe_sizes": moe(40, 6, 260, (8, 3), 2.5, 300), "moe_48_kB": moe(7, 6, 1500, (7, 6), 1.0, 3000), "moe_ff_1": moe(5, 2, 1, None, 1.0, 1)}
 
 
 @BOTH

@@ -6,15 +6,17 @@
 
 namespace tlb {
 
-__device__ __forceinline__ float sigmoidf(float x) { return 1.f / (1.f + expf(-x)); }
-__device__ __forceinline__ float siluf(float x) { return x / (1.f + expf(-x)); }
-// z / 2 (1 + tanh(c)) = z sigmoid(2 c)
-__device__ __forceinline__ float gelu_tanhf(float z)
+// __fdividef: two units in the last place, without the branch of the full division; a divisor near overflow gives zero, the limit
+__device__ __forceinline__ float sigmoidf(float x) { return __fdividef(1.f, 1.f + expf(-x)); }
+__device__ __forceinline__ float siluf(float x) { return __fdividef(x, 1.f + expf(-x)); }
+// Both gated activations are z sigmoid(z (a + b z^2)): SiLU with a = 1, b = 0; the tanh form of GELU, z / 2 (1 + tanh(c)) = z sigmoid(2 c).
+struct GluConst { float a, b; };
+__host__ __device__ inline GluConst glu_const(int act)
 {
-    constexpr float kRoot2 = 2.f * 0.79788456080286535588f;  // 2 sqrt(2 / pi)
-    return z / (1.f + expf(-kRoot2 * fmaf(0.044715f * z * z, z, z)));
+    const float root = 2.f * 0.79788456080286535588f;        // 2 sqrt(2 / pi)
+    return act == GLU_SILU ? GluConst{1.f, 0.f} : GluConst{root, 0.044715f * root};
 }
-__device__ __forceinline__ float glu_act(int act, float gate, float up) { return (act == GLU_SILU ? siluf(gate) : gelu_tanhf(gate)) * up; }
+__device__ __forceinline__ float glu_act(const GluConst &c, float z, float up) { return __fdividef(z, 1.f + expf(-z * fmaf(c.b * z, z, c.a))) * up; }
 // value that enters a gated recurrence without a normaliser: positive, continuous, slope one above zero
 __device__ __forceinline__ float gru_candidate(float u) { return u >= 0.f ? u + 0.5f : sigmoidf(u); }
 

@@ -47,7 +47,8 @@ struct DenseMvParams {
     const float *y, *y_gate, *post_w;
     float *h_out;
     float *act_out;
-    int glu, act, ldx;
+    int glu, ldx;
+    GluConst act;
     RouteDesc route;
     const float *logits;
     int *sel;
@@ -351,14 +352,15 @@ struct DenseTcParams {
     size_t block_stride;
     __half *out_h, *out_t;
     const int4 *tiles;
-    int glu, act, ld_act;
+    int glu, ld_act;
+    GluConst act;
     __nv_bfloat16 *act_out;
     uint32_t type_bits;                    // operand types in the instruction descriptor
 };
 
 // One CTA: 128 weight rows (lanes of the accumulator) x nt tokens (its columns).  Warps 0-3 write out (a warp's 32 lanes are 32
 // consecutive output features of one token: coalesced), warp 4 lane 0 issues TMA, warp 5 lane 0 the MMAs.  Every wait is bounded.
-__global__ void __launch_bounds__(kTcThreads, 1)
+__global__ void __launch_bounds__(kTcThreads, 2)
 dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ CUtensorMap xmap, const DenseTcParams p)
 {
     extern __shared__ uint8_t tc_smem[];
@@ -410,14 +412,16 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_cons
                 if (n0 + warp * 32 < p.glu) {
                     // lanes (0, 1), (2, 3) of four hold gates and ups of two units: the former take tokens 0 .. 15, the latter 16 .. 31
                     const bool hi = lane & 2;
-                    const float mine = bias, theirs = __shfl_xor_sync(0xffffffffu, bias, 2);
+                    const float theirs = __shfl_xor_sync(0xffffffffu, bias, 2);
+                    const GluConst act = p.act;
                     __nv_bfloat16 *da = p.act_out + (size_t)(t0 + c0) * p.ld_act + (row >> 2) * 2 + (row & 1);
 #pragma unroll
                     for (int i = 0; i < 16; i++) {
                         const float other = __uint_as_float(__shfl_xor_sync(0xffffffffu, hi ? v[i] : v[i + 16], 2)) + theirs;
-                        const float own = __uint_as_float(hi ? v[i + 16] : v[i]) + mine;
+                        const float own = __uint_as_float(hi ? v[i + 16] : v[i]) + bias;
                         const int t = hi ? i + 16 : i;
-                        if (row < p.glu && t0 + c0 + t < t_end) da[(size_t)t * p.ld_act] = __float2bfloat16_rn(hi ? glu_act(p.act, other, own) : glu_act(p.act, own, other));
+                        const float y = glu_act(act, hi ? other : own, hi ? own : other);
+                        if (row < p.glu && t0 + c0 + t < t_end) da[(size_t)t * p.ld_act] = __float2bfloat16_rn(y);
                     }
                 }
                 if (!in || row < p.glu) continue;
@@ -509,7 +513,8 @@ struct DenseF32Params {
     int per;
     size_t block_stride;
     const int4 *tiles;
-    int glu, act, ld_act;
+    int glu, ld_act;
+    GluConst act;
     float *act_out;
 };
 constexpr int kSgT = kF32GemmRows, kSgN = 64, kSgK = 16;
@@ -708,7 +713,7 @@ tlb_status run_matvec(const DenseMvParams &p, bool pdl)
 {
     Context *c = ctx();
     const size_t smem = ((size_t)p.nch * kMvChunk + (PRO == DPRO_EXPERT ? route_scratch_floats(p.route) : 0)) * sizeof(float);
-    static size_t allowed = 48 << 10;
+    static size_t allowed = 40 << 10;      // with the static part, under the 48 KB that need no asking
     if (smem > allowed) {
         TLB_CUDA(cudaFuncSetAttribute(dense_matvec_kernel<PRO, WK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         allowed = smem;
@@ -756,7 +761,7 @@ tlb_status launch_dense_matvec(const DenseMatvecJob &j)
     p.bias = j.w.bias; p.x = j.x; p.emb = j.emb; p.emb_ld = act_ld(j.w.k); p.token = j.token; p.x_out = j.x_out;
     p.norm_w = j.norm_w; p.norm_offset = j.norm_offset; p.eps = j.eps; p.poly = j.poly; p.out = j.out; p.resid_scale = j.resid_scale;
     p.softcap = j.softcap; p.groups = j.groups; p.y = j.y; p.y_gate = j.y_gate; p.post_w = j.post_w; p.h_out = j.h_out;
-    p.glu = j.w.glu; p.act = j.w.glu_act; p.act_out = j.act_out; p.ldx = j.ldx;
+    p.glu = j.w.glu; p.act = glu_const(j.w.glu_act); p.act_out = j.act_out; p.ldx = j.ldx;
     p.route = j.route; p.logits = j.logits; p.sel = j.sel; p.weight = j.weight;
     if (j.pro == DPRO_EXPERTS) {
         p.seg_nch = p.nch;
@@ -780,7 +785,7 @@ tlb_status launch_dense_gemm(const DenseGemmJob &j, bool f32)
     if (f32) {
         DenseF32Params p;
         p.softcap = j.softcap; p.per = per; p.block_stride = j.block_stride; p.tiles = j.tiles;
-        p.glu = j.w.glu; p.act = j.w.glu_act; p.ld_act = j.ld_act; p.act_out = (float *)j.act_out;
+        p.glu = j.w.glu; p.act = glu_const(j.w.glu_act); p.ld_act = j.ld_act; p.act_out = (float *)j.act_out;
         p.w = j.w.w; p.n = j.w.n; p.k = j.w.k; p.ld = j.w.ld; p.bias = j.w.bias; p.x = (const float *)j.x; p.resid_scale = j.resid_scale;
         p.ldx = j.ldx; p.T = j.T; p.ldo = j.ldo; p.out = j.out;
         dense_gemm_f32_kernel<<<dim3(j.tiles ? j.n_tiles : (j.T + kSgT - 1) / kSgT, (j.w.n + kSgN - 1) / kSgN), 256, 0, c->stream>>>(p);
@@ -789,14 +794,16 @@ tlb_status launch_dense_gemm(const DenseGemmJob &j, bool f32)
     DenseTcParams p;
     p.out = j.out; p.bias = j.w.bias; p.resid_scale = j.resid_scale; p.n = j.w.n; p.T = j.T; p.ldo = j.ldo;
     p.softcap = j.softcap; p.per = per; p.block_stride = j.block_stride; p.out_h = j.out_h; p.out_t = j.out_t; p.tiles = j.tiles;
-    p.glu = j.w.glu; p.act = j.w.glu_act; p.ld_act = j.ld_act; p.act_out = (__nv_bfloat16 *)j.act_out;
+    p.glu = j.w.glu; p.act = glu_const(j.w.glu_act); p.ld_act = j.ld_act; p.act_out = (__nv_bfloat16 *)j.act_out;
     p.type_bits = j.w.f16 ? 0u : (1u << 7) | (1u << 10);
-    p.nt = j.tiles ? j.tile_rows : (j.out_t ? 128 : std::min(256, (j.T + 31) / 32 * 32));
+    p.kt = (j.w.k + kTcK - 1) / kTcK;
+    // short sums, and experts' tiles: two CTAs share an SM, one's epilogue under the other's products
+    const bool pair = p.kt <= 16 || j.tiles;
+    p.nt = j.tiles ? j.tile_rows : (j.out_t ? 128 : std::min(pair ? 128 : 256, (j.T + 31) / 32 * 32));
     p.tmem_cols = 32;
     while (p.tmem_cols < (uint32_t)p.nt) p.tmem_cols *= 2;
-    p.kt = (j.w.k + kTcK - 1) / kTcK;
     const size_t stage = kTcWBytes + (size_t)p.nt * kTcK * 2;
-    p.stages = (int)std::min<size_t>(8, ((size_t)216 << 10) / stage);
+    p.stages = (int)std::min<size_t>(8, ((size_t)(pair ? 104 : 216) << 10) / stage);
     p.err = c->err_flag;
     CUtensorMap wmap, xmap;
     const CUtensorMapDataType type = j.w.f16 ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;

@@ -354,7 +354,7 @@ tlb_status run_decode(const MixAttnDecode &j)
     const int rep = a.H / a.KVH;
     const size_t smem = (size_t)(rep * a.ldk + 2 * rep * kDecKeys + 2 * rep + 4 + std::max(dec_red_floats<CT>(), rep * decode_splits(a) + 4 + 4 * kDecThreads)) * sizeof(float);
     if (smem > ctx()->smem_optin) return fail(TLB_ERR_SHAPE, "attention: %d query heads per KV head of size %d do not fit shared memory", rep, a.D);
-    static size_t allowed = 48 << 10;
+    static size_t allowed = 40 << 10;      // with the static part, under the 48 KB that need no asking
     if (smem > allowed) {
         TLB_CUDA(cudaFuncSetAttribute(mix_attn_decode_kernel<CT, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         allowed = smem;

@@ -468,23 +468,36 @@ __global__ void __launch_bounds__(kThreads) latent_value_kernel(const MixLatentR
 }
 
 // ================================================================ long portions
-// rotates the queries of a token in place (or, with q16, into f16 rows whose heads are padded to qd) and appends its cache row
-template <typename CT>
-__global__ void __launch_bounds__(kThreads) latent_prep_kernel(const MixLatent m, int seq, int pos0, int rope0, int rope_step, __half *__restrict__ q16, int qd)
+// rotates the queries of a token in place (or, with QD, into f16 rows whose heads are padded to QD) and appends its cache row
+template <typename CT, int QD>
+__global__ void __launch_bounds__(kThreads) latent_prep_kernel(const MixLatent m, int seq, int pos0, int rope0, int rope_step, __half *__restrict__ q16)
 {
+    constexpr int kPairs = QD ? QD / 2 : 1;
     __shared__ float part[kWarps], inv[1];
     const int t = blockIdx.x, rope = rope0 + t * rope_step, half = m.rot / 2, hd = m.D + m.RD;
     const float *c = m.rot_cos + (size_t)rope * half, *s = m.rot_sin + (size_t)rope * half;
     float *q = m.q + (size_t)t * m.ldq;
-    if (q16) {
-        __half2 *dst = reinterpret_cast<__half2 *>(q16 + (size_t)t * m.H * qd);
-        auto value = [&](const float *x, int d) { return d < m.D ? __ldcg(x + d) : (d < hd ? turned(x + m.D, d - m.D, m.rot, c, s) : 0.f); };
+    if (QD) {
+        __half2 *dst = reinterpret_cast<__half2 *>(q16 + (size_t)t * m.H * QD);
         auto clamp = [](float v) { return fminf(fmaxf(v, -65504.f), 65504.f); };
+        if (m.D % 2 == 0 && m.RD % 2 == 0 && m.ldq % 2 == 0 && (reinterpret_cast<uintptr_t>(m.q) & 7) == 0) {
 #pragma unroll 4
-        for (int i = threadIdx.x; i < m.H * qd / 2; i += kThreads) {
-            const int h = i / (qd / 2), d = (i - h * (qd / 2)) * 2;
-            const float *x = q + (size_t)h * hd;
-            dst[i] = __floats2half2_rn(clamp(value(x, d)), clamp(value(x, d + 1)));
+            for (int i = threadIdx.x; i < m.H * kPairs; i += kThreads) {
+                const int h = i / kPairs, d = (i - h * kPairs) * 2, r = d - m.D;
+                float2 v = d < hd ? __ldcg(reinterpret_cast<const float2 *>(q + (size_t)h * hd + d)) : make_float2(0.f, 0.f);
+                if (r >= 0 && r < m.rot) {
+                    const float cs = c[r >> 1], sn = s[r >> 1];
+                    v = make_float2(v.x * cs - v.y * sn, v.y * cs + v.x * sn);
+                }
+                dst[i] = __floats2half2_rn(clamp(v.x), clamp(v.y));
+            }
+        } else {
+            auto value = [&](const float *x, int d) { return d < m.D ? __ldcg(x + d) : (d < hd ? turned(x + m.D, d - m.D, m.rot, c, s) : 0.f); };
+            for (int i = threadIdx.x; i < m.H * kPairs; i += kThreads) {
+                const int h = i / kPairs, d = (i - h * kPairs) * 2;
+                const float *x = q + (size_t)h * hd;
+                dst[i] = __floats2half2_rn(clamp(value(x, d)), clamp(value(x, d + 1)));
+            }
         }
     } else {
         for (int i = threadIdx.x; i < m.H * half; i += kThreads) {
@@ -525,7 +538,7 @@ template <int PW>
 tlb_status run_attn_tc(const MixLatentRows &j, int splits)
 {
     const size_t smem = attn_tc_smem(j.m);
-    static size_t allowed = 48 << 10;
+    static size_t allowed = 40 << 10;      // with the static part, under the 48 KB that need no asking
     if (smem > allowed) {
         TLB_CUDA(cudaFuncSetAttribute(latent_attn_tc_kernel<PW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         allowed = smem;
@@ -544,7 +557,7 @@ tlb_status run_query(const MixLatentRows &j)
     int tc = 8;
     while (tc < 64 && tc < vecs && (vecs / tc) * m.H * tiles > 4 * ctx()->sm_count) tc *= 2;
     const size_t smem = ((size_t)(RT * m.D + 3) / 4 * 4 + (size_t)kThreads * RT * 8) * sizeof(float);
-    static size_t allowed = 48 << 10;
+    static size_t allowed = 40 << 10;      // with the static part, under the 48 KB that need no asking
     if (smem > allowed) {
         TLB_CUDA(cudaFuncSetAttribute(latent_query_kernel<CT, RT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         allowed = smem;
@@ -628,8 +641,10 @@ tlb_status launch_latent_prompt(const MixLatent &m, int seq, int T, int pos0, in
     void *keys = get((size_t)m.H * n_keys * ldk * es), *vals = get((size_t)m.H * (tc5 ? (size_t)128 * vt_ld : (size_t)n_keys * ldv) * es);
     __half *q16 = tc5 ? (__half *)get((size_t)T * m.H * qd * 2) : nullptr;
     if (!keys || !vals || (tc5 && !q16)) return done(TLB_ERR_ALLOC);
-    if (f32) latent_prep_kernel<float><<<T, kThreads, 0, c->stream>>>(m, seq, pos0, rope0, rope_step, nullptr, 0);
-    else latent_prep_kernel<__half><<<T, kThreads, 0, c->stream>>>(m, seq, pos0, rope0, rope_step, q16, qd);
+    if (f32) latent_prep_kernel<float, 0><<<T, kThreads, 0, c->stream>>>(m, seq, pos0, rope0, rope_step, nullptr);
+    else if (!tc5) latent_prep_kernel<__half, 0><<<T, kThreads, 0, c->stream>>>(m, seq, pos0, rope0, rope_step, nullptr);
+    else if (qd == 128) latent_prep_kernel<__half, 128><<<T, kThreads, 0, c->stream>>>(m, seq, pos0, rope0, rope_step, q16);
+    else latent_prep_kernel<__half, 192><<<T, kThreads, 0, c->stream>>>(m, seq, pos0, rope0, rope_step, q16);
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return done(cuda_fail(e, "latent preparation launch"));
     const char *cache = (const char *)m.cache + ((size_t)seq * m.seq_stride + (size_t)key_first * m.ld) * es;

@@ -76,7 +76,7 @@ int moe_tile_rows(const RouteDesc &r, int T, bool f32)
 {
     if (f32) return kF32GemmRows;
     const int mean = (int)((int64_t)T * r.top / r.experts);
-    return std::min(256, std::max(32, (mean + mean / 4 + 31) / 32 * 32));
+    return std::min(128, std::max(32, (mean + mean / 4 + 31) / 32 * 32));
 }
 
 int moe_max_tiles(const RouteDesc &r, int T, bool f32)

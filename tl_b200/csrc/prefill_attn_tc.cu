@@ -206,9 +206,20 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __gr
             if (MIX && p.gate) {
                 const float *gt = p.gate + (size_t)(q0 + warp * 32) * p.ld_gate + (size_t)h * p.DV;
                 const int nr = min(32, p.T - (q0 + warp * 32));
-                for (int c = lane; c < p.DV; c += 32) {
-#pragma unroll 16
-                    for (int r = 0; r < nr; r++) s_gate[r * kGatePitch + c] = sigmoidf(__ldg(gt + (size_t)r * p.ld_gate + c));
+                if (p.DV % 4 == 0 && p.ld_gate % 4 == 0 && (reinterpret_cast<uintptr_t>(p.gate) & 15) == 0) {
+#pragma unroll
+                    for (int r0 = 0; r0 < 32; r0 += 16) {
+                        float4 g[16];
+#pragma unroll
+                        for (int r = 0; r < 16; r++)
+                            g[r] = r0 + r < nr && lane * 4 < p.DV ? __ldcg(reinterpret_cast<const float4 *>(gt + (size_t)(r0 + r) * p.ld_gate) + lane) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+                        for (int r = 0; r < 16; r++)
+                            *reinterpret_cast<float4 *>(s_gate + (r0 + r) * kGatePitch + lane * 4) = make_float4(sigmoidf(g[r].x), sigmoidf(g[r].y), sigmoidf(g[r].z), sigmoidf(g[r].w));
+                    }
+                } else {
+                    for (int r = 0; r < nr; r++)
+                        for (int c = lane; c < p.DV; c += 32) s_gate[r * kGatePitch + c] = sigmoidf(gt[(size_t)r * p.ld_gate + c]);
                 }
                 __syncwarp();
             }
