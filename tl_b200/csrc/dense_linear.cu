@@ -447,7 +447,7 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_cons
                     for (int i = 0; i < 32; i++)
                         if (i < m) dh[(size_t)i * p.ldo] = __float2half_rn(fminf(fmaxf(__uint_as_float(v[i]) + bias, -65504.f), 65504.f));
                 } else if (p.softcap > 0.f) {
-#pragma unroll 4
+#pragma unroll
                     for (int i = 0; i < 32; i++)
                         if (i < m) dst[(size_t)i * p.ldo] = p.softcap * tanhf((__uint_as_float(v[i]) + bias) / p.softcap);
                 } else if (p.resid_scale) {
@@ -589,14 +589,14 @@ __device__ __forceinline__ void store_act4(__nv_bfloat16 *p, float a, float b, f
 }
 
 template <typename TA>
-__global__ void __launch_bounds__(256) norm_rows_kernel(const float *__restrict__ x, int width, const float *__restrict__ w, float offset, float eps,
+__global__ void __launch_bounds__(256) norm_rows_kernel(const float *__restrict__ x, int width, int ldx, const float *__restrict__ w, float offset, float eps,
                                                         TA *__restrict__ out, int ld)
 {
     __shared__ float red[8];
-    const float *row = x + (size_t)blockIdx.x * width;
+    const float *row = x + (size_t)blockIdx.x * ldx;
     TA *o = out + (size_t)blockIdx.x * ld;
     float ss[1] = {0.f};
-    if (width % 4 == 0 && width <= 256 * 4 * 8) {       // the row stays in registers: one pass over memory
+    if (width % 4 == 0 && ldx % 4 == 0 && width <= 256 * 4 * 8) {       // the row stays in registers: one pass over memory
         float4 v[8];
         const int n4 = width / 4;
 #pragma unroll
@@ -797,8 +797,8 @@ tlb_status launch_dense_gemm(const DenseGemmJob &j, bool f32)
     p.glu = j.w.glu; p.act = glu_const(j.w.glu_act); p.ld_act = j.ld_act; p.act_out = (__nv_bfloat16 *)j.act_out;
     p.type_bits = j.w.f16 ? 0u : (1u << 7) | (1u << 10);
     p.kt = (j.w.k + kTcK - 1) / kTcK;
-    // short sums, and experts' tiles: two CTAs share an SM, one's epilogue under the other's products
-    const bool pair = p.kt <= 16 || j.tiles;
+    // short sums, gated activations and experts' tiles: two CTAs share an SM, one's epilogue under the other's products
+    const bool pair = p.kt <= 16 || j.w.glu || j.tiles;
     p.nt = j.tiles ? j.tile_rows : (j.out_t ? 128 : std::min(pair ? 128 : 256, (j.T + 31) / 32 * 32));
     p.tmem_cols = 32;
     while (p.tmem_cols < (uint32_t)p.nt) p.tmem_cols *= 2;
@@ -820,10 +820,10 @@ tlb_status launch_dense_gemm(const DenseGemmJob &j, bool f32)
     return launched("GEMM launch");
 }
 
-tlb_status launch_norm_rows(const float *x, int T, int width, const float *w, float offset, float eps, void *out, int ld, bool f32)
+tlb_status launch_norm_rows(const float *x, int T, int width, int ldx, const float *w, float offset, float eps, void *out, int ld, bool f32)
 {
-    if (f32) norm_rows_kernel<<<T, 256, 0, ctx()->stream>>>(x, width, w, offset, eps, (float *)out, ld);
-    else norm_rows_kernel<<<T, 256, 0, ctx()->stream>>>(x, width, w, offset, eps, (__nv_bfloat16 *)out, ld);
+    if (f32) norm_rows_kernel<<<T, 256, 0, ctx()->stream>>>(x, width, ldx, w, offset, eps, (float *)out, ld);
+    else norm_rows_kernel<<<T, 256, 0, ctx()->stream>>>(x, width, ldx, w, offset, eps, (__nv_bfloat16 *)out, ld);
     return launched("norm launch");
 }
 

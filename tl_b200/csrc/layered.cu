@@ -536,7 +536,7 @@ tlb_status rows_norm(const LayeredModel *lm, const float *x, int T, const tlb_te
 {
     const ModelDesc &d = lm->desc;
     const int ld = act_ld(d.width);
-    if (d.norm_groups == 1) return launch_norm_rows(x, T, d.width, w->f32(), d.norm_offset, d.eps, out, ld, lm->cfg.f32);
+    if (d.norm_groups == 1) return launch_norm_rows(x, T, d.width, d.width, w->f32(), d.norm_offset, d.eps, out, ld, lm->cfg.f32);
     ResidNormJob j;
     j.x = const_cast<float *>(x); j.T = T; j.width = d.width; j.groups = d.norm_groups; j.offset = d.norm_offset; j.eps = d.eps; j.norm_w = w->f32(); j.out = out; j.ldo = ld;
     return launch_resid_norm_rows(j, lm->cfg.f32);
@@ -548,7 +548,7 @@ tlb_status rows_mixer(LayeredModel *lm, const Layer &L, RowBufs &b, const RowCtx
     const bool f32 = lm->cfg.f32;
     const MixerDesc &x = L.d->mix;
     if (x.q_rank) {
-        TLB_TRY(launch_rms_cols(b.proj, c.T, x.q_rank, lm->ldp, L.qnorm->f32(), lm->desc.eps, b.act, act_ld(x.q_rank), f32));
+        TLB_TRY(launch_norm_rows(b.proj, c.T, x.q_rank, lm->ldp, L.qnorm->f32(), 0.f, lm->desc.eps, b.act, act_ld(x.q_rank), f32));
         TLB_TRY(rows_gemm(lm, L.uq, b.act, act_ld(x.q_rank), c.T, b.q, lm->ldq, nullptr));
     }
     if (c.pos) return decode_mixer(lm, L, c.T, b.proj, b.q, b.qa, b.partial, c.pos, c.rope, b.act, lda, f32, false);

@@ -94,8 +94,8 @@ struct DenseGemmJob {
 tlb_status launch_dense_gemm(const DenseGemmJob &j, bool f32);
 constexpr int kF32GemmRows = 64;          // rows of a tile of the 32-bit GEMM
 
-// rows in the activation type, pitch ld
-tlb_status launch_norm_rows(const float *x, int T, int width, const float *w, float offset, float eps, void *out, int ld, bool f32);
+// rows in the activation type, pitch ld; x: the first `width` of every ldx numbers, 16-byte aligned
+tlb_status launch_norm_rows(const float *x, int T, int width, int ldx, const float *w, float offset, float eps, void *out, int ld, bool f32);
 tlb_status launch_poly_rows(const float *z, int T, int ff, int ldz, const float *coef, float eps, void *out, int ld, bool f32);
 tlb_status launch_embed_bf16(const int *tokens, const __nv_bfloat16 *table, int width, int ld, float *x, int T);
 tlb_status launch_gather_rows(const float *x, int width, const int *idx, int n, float *out);
@@ -104,7 +104,7 @@ tlb_status launch_pack_rows(const __nv_bfloat16 *src, int n, int k, __nv_bfloat1
 tlb_status launch_pack_glu_rows(const __nv_bfloat16 *src, int ff, int k, __nv_bfloat16 *dst, int ld, bool up);
 tlb_status launch_pack_rows_f16(const __nv_bfloat16 *src, int n, int k, void *dst, int ld);      // values as f16
 
-// ---------------------------------------------------------------- row_kernels.cu
+// ---------------------------------------------------------------- resid_rows.cu
 // What a mixture of experts leaves per token: y = sum over the choice of weight * part[slot] + sigmoid(shared_gate) * shared.
 struct MoeRows {
     int top = 0;
@@ -127,8 +127,6 @@ struct ResidNormJob {
     int ldo = 0;
 };
 tlb_status launch_resid_norm_rows(const ResidNormJob &j, bool f32);
-// out [T, ld] = rows of n values at x, each over its root mean square, times w
-tlb_status launch_rms_cols(const float *x, int T, int n, int ldx, const float *w, float eps, void *out, int ld, bool f32);
 
 // ---------------------------------------------------------------- moe.cu
 // The choice of T tokens and the order their rows take behind one another, expert by expert.

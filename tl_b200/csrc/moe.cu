@@ -27,14 +27,17 @@ __global__ void __launch_bounds__(128) route_rows_kernel(const RouteDesc r, cons
 // first row of every expert and the tiles; one CTA
 __global__ void __launch_bounds__(256) moe_tiles_kernel(int experts, int *__restrict__ count, int tile_rows, int4 *__restrict__ tiles, int max_tiles)
 {
-    extern __shared__ int s_first[];                       // [experts + 1] rows, [experts + 1] tiles
+    extern __shared__ int s_first[];                       // [experts + 1] counts, then first rows; [experts + 1] tiles
     int *s_tile = s_first + experts + 1;
+    for (int e = threadIdx.x; e < experts; e += 256) s_first[e] = count[e];
+    __syncthreads();
     if (threadIdx.x == 0) {
         int row = 0, tile = 0;
         for (int e = 0; e < experts; e++) {
+            const int n = s_first[e];
             s_first[e] = row; s_tile[e] = tile;
-            row += count[e];
-            tile += (count[e] + tile_rows - 1) / tile_rows;
+            row += n;
+            tile += (n + tile_rows - 1) / tile_rows;
         }
         s_first[experts] = row; s_tile[experts] = tile;
     }

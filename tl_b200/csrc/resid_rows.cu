@@ -1,5 +1,5 @@
-// Row kernels of layered models: norms of part of a row, and the residual step of designs that norm what a sublayer adds - gate,
-// norm in groups, addition and the next sublayer's norm in one pass over the row.
+// The residual step of designs that norm what a sublayer adds, over rows: gate, norm in groups, addition and the next sublayer's norm
+// in one pass; the sum over a token's experts comes in front where the sublayer is a mixture.
 #include <algorithm>
 
 #include "act.cuh"
@@ -8,15 +8,6 @@
 namespace tlb {
 
 namespace {
-
-template <typename TA>
-__global__ void __launch_bounds__(256) rms_cols_kernel(const float *__restrict__ x, int n, int ldx, const float *__restrict__ w, float eps, TA *__restrict__ out, int ld)
-{
-    __shared__ float part[8], inv[1];
-    const float *row = x + (size_t)blockIdx.x * ldx;
-    group_inv_rms([&](int e) { return row[e]; }, n, 1, eps, part, inv);
-    for (int e = threadIdx.x; e < n; e += 256) store_actv(out + (size_t)blockIdx.x * ld + e, row[e] * inv[0] * w[e]);
-}
 
 struct ResidNormParams {
     float *x;
@@ -134,13 +125,6 @@ tlb_status run_resid(const ResidNormParams &p, int T, void *out)
 }
 
 }  // namespace
-
-tlb_status launch_rms_cols(const float *x, int T, int n, int ldx, const float *w, float eps, void *out, int ld, bool f32)
-{
-    if (f32) rms_cols_kernel<<<T, 256, 0, ctx()->stream>>>(x, n, ldx, w, eps, (float *)out, ld);
-    else rms_cols_kernel<<<T, 256, 0, ctx()->stream>>>(x, n, ldx, w, eps, (__nv_bfloat16 *)out, ld);
-    return launched("norm launch");
-}
 
 tlb_status launch_resid_norm_rows(const ResidNormJob &j, bool f32)
 {
