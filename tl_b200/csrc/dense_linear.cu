@@ -2,8 +2,10 @@
 //
 //   dense_matvec_kernel   one activation row (decode): streams the weight once, f32 activation and accumulation.  The prologue
 //                         makes the activation in shared memory - RMS norm, PolyNorm (its three root mean squares), an embedding
-//                         row - and the finish adds the scaled result to the residual, so a layer is five launches.
-//   dense_gemm_tc_kernel  many rows, bf16 operands: tcgen05.mma, both tiles by TMA, f32 accumulator in tensor memory.
+//                         row, the residual step of a gated and normed sublayer, a router's choice - and the finish adds the
+//                         scaled result to the residual or turns gate and up into one activation.
+//   dense_gemm_tc_kernel  many rows, 16-bit operands: tcgen05.mma, both tiles by TMA, f32 accumulator in tensor memory; also over
+//                         row tiles of several stacked weights (experts).
 //   dense_gemm_f32_kernel many rows, f32 activations: plain f32 multiply-adds (no tensor core rounds the operands).
 #include <algorithm>
 

@@ -10,7 +10,7 @@ namespace tlb {
 
 namespace {
 
-constexpr int kGruWarps = 32, kGruRun = 4, kGruTile = kGruWarps * kGruRun;
+constexpr int kGruWarps = 16, kGruRun = 8, kGruTile = kGruWarps * kGruRun;
 
 template <typename TO>
 __global__ void __launch_bounds__(kGruWarps * 32) gru_scan_kernel(const MixGru m, int seq, int T, int pos0, TO *__restrict__ out, int ldo)
@@ -18,18 +18,17 @@ __global__ void __launch_bounds__(kGruWarps * 32) gru_scan_kernel(const MixGru m
     __shared__ float s_a[2][kGruWarps][32], s_b[2][kGruWarps][32];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, c = blockIdx.x * 32 + lane;
     const bool live = c < m.width;
-    const float *pz = m.proj + c, *pu = pz + m.width, *pg = pu + m.width;
+    const float *pz = m.proj + c;
     float state = live && pos0 > 0 ? m.state[(size_t)seq * m.width + c] : 0.f;
     float z[kGruRun], u[kGruRun], g[kGruRun];
     auto fetch = [&](int t0) {
+        const int n = live ? T - (t0 + warp * kGruRun) : 0;       // tokens of the run that exist
+        const float *row = pz + (size_t)(t0 + warp * kGruRun) * m.ldp;
 #pragma unroll
-        for (int i = 0; i < kGruRun; i++) {
-            const int t = t0 + warp * kGruRun + i;
-            const bool in = live && t < T;
-            const size_t at = (size_t)t * m.ldp;
-            z[i] = in ? pz[at] : -INFINITY;                 // past the end: z = 0, the state stays
-            u[i] = in ? pu[at] : 0.f;
-            g[i] = in ? pg[at] : 0.f;
+        for (int i = 0; i < kGruRun; i++, row += m.ldp) {
+            z[i] = i < n ? __ldcs(row) : -INFINITY;          // past the end: z = 0, the state stays
+            u[i] = i < n ? __ldcs(row + m.width) : 0.f;
+            g[i] = i < n ? __ldcs(row + 2 * m.width) : 0.f;
         }
     };
     fetch(0);
@@ -54,11 +53,12 @@ __global__ void __launch_bounds__(kGruWarps * 32) gru_scan_kernel(const MixGru m
             if (i == warp) mine = state;
             state = fmaf(s_a[b][i][lane], state, s_b[b][i][lane]);
         }
+        const int n = live ? T - (t0 + warp * kGruRun) : 0;
+        TO *dst = out + (size_t)(t0 + warp * kGruRun) * ldo + c;
 #pragma unroll
-        for (int i = 0; i < kGruRun; i++) {
+        for (int i = 0; i < kGruRun; i++, dst += ldo) {
             mine = fmaf(k[i], mine, v[i]);
-            const int t = t0 + warp * kGruRun + i;
-            if (live && t < T) store_actv(out + (size_t)t * ldo + c, mine * w[i]);
+            if (i < n) store_actv(dst, mine * w[i]);
         }
     }
     if (live && warp == 0) m.state[(size_t)seq * m.width + c] = state;

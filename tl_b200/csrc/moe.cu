@@ -52,7 +52,6 @@ __global__ void __launch_bounds__(256) moe_tiles_kernel(int experts, int *__rest
 }
 
 // one CTA per (token, choice): the row moves to its place, which becomes an index over all experts' rows
-template <int BYTES>
 __global__ void __launch_bounds__(128) moe_gather_kernel(int top, const int *__restrict__ sel, int *__restrict__ place, const int *__restrict__ first,
                                                          const char *__restrict__ act, size_t row_bytes, char *__restrict__ out)
 {
@@ -60,7 +59,7 @@ __global__ void __launch_bounds__(128) moe_gather_kernel(int top, const int *__r
     const int dst = first[sel[i]] + place[i];
     const uint4 *s = reinterpret_cast<const uint4 *>(act + (size_t)t * row_bytes);
     uint4 *d = reinterpret_cast<uint4 *>(out + (size_t)dst * row_bytes);
-    for (size_t k = threadIdx.x; k < row_bytes / BYTES; k += 128) d[k] = s[k];
+    for (size_t k = threadIdx.x; k < row_bytes / 16; k += 128) d[k] = s[k];
     __syncthreads();
     if (threadIdx.x == 0) place[i] = dst;
 }
@@ -99,7 +98,7 @@ tlb_status launch_moe_plan(const RouteDesc &r, const float *logits, int ldl, int
 
 tlb_status launch_moe_gather(const RouteDesc &r, const MoePlan &p, const void *act, int T, int ld, void *out, bool f32)
 {
-    moe_gather_kernel<16><<<T * r.top, 128, 0, ctx()->stream>>>(r.top, p.sel, p.place, p.count + r.experts, (const char *)act, (size_t)ld * (f32 ? 4 : 2), (char *)out);
+    moe_gather_kernel<<<T * r.top, 128, 0, ctx()->stream>>>(r.top, p.sel, p.place, p.count + r.experts, (const char *)act, (size_t)ld * (f32 ? 4 : 2), (char *)out);
     return launched("expert gather launch");
 }
 
