@@ -517,6 +517,16 @@ __global__ void __launch_bounds__(kThreads) latent_rot_kernel(const MixLatent m,
 {
     const int key = blockIdx.x, tail = ldk - m.D;
     const CT *src = cache + (size_t)key * m.ld + m.R;
+    constexpr int VE = 16 / sizeof(CT);
+    if (m.D % VE == 0 && m.R % VE == 0 && m.RD % VE == 0) {
+        const int nv = tail / VE;
+        for (int i = threadIdx.x; i < m.H * nv; i += kThreads) {
+            const int h = i / nv, v = i - h * nv;
+            *reinterpret_cast<uint4 *>(keys + ((size_t)h * n_keys + key) * ldk + m.D + v * VE) =
+                v * VE < m.RD ? *reinterpret_cast<const uint4 *>(src + v * VE) : make_uint4(0u, 0u, 0u, 0u);
+        }
+        return;
+    }
     for (int i = threadIdx.x; i < m.H * tail; i += kThreads) {
         const int h = i / tail, e = i - h * tail;
         keys[((size_t)h * n_keys + key) * ldk + m.D + e] = e < m.RD ? src[e] : (CT)0.f;
