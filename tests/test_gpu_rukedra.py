@@ -99,7 +99,7 @@ MIXERS = {
     "latent_factor_1": latent(scaling=dict(YARN, factor=1.0)), "latent_narrow_ramp": latent(scaling={"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}),
     "latent_tiny": latent(heads=1, dim=1, rot_dim=2, vdim=1, kv_rank=1, q_rank=1, window=6, scale=1.0), "latent_17_heads": latent(heads=17, dim=8, rot_dim=4, vdim=5, kv_rank=16, window=64),
     "latent_equal": latent(heads=4, dim=32, rot_dim=32, vdim=32, kv_rank=32, q_rank=32, window=33, scale=0.125),
-    "latent_80": latent(heads=2, dim=64, rot_dim=16, vdim=64, kv_rank=48, window=66, scale=0.1), "latent_rank_130": latent(heads=2, kv_rank=130, window=90),
+    "latent_80": latent(heads=2, dim=64, rot_dim=16, vdim=64, kv_rank=48, window=66, scale=0.1), "latent_84_odd": latent(heads=3, dim=70, rot_dim=14, vdim=66, kv_rank=47, q_rank=35, window=90, scale=0.1), "latent_rank_130": latent(heads=2, kv_rank=130, window=90),
     "direct": direct(), "direct_one_head": direct(heads=1), "direct_192": direct(heads=2, dim=128, rot_dim=64, vdim=128, kv_rank=200, scale=0.07),
     "direct_170": direct(heads=2, dim=130, rot_dim=40, vdim=100, kv_rank=88, scale=0.07), "direct_256": direct(heads=2, dim=200, rot_dim=56, vdim=150, kv_rank=64, scale=0.06),
     "direct_300": direct(heads=2, dim=280, rot_dim=20, vdim=270, kv_rank=40, scale=0.06), "direct_rank_300": direct(heads=3, kv_rank=300), "direct_rank_600": direct(heads=2, kv_rank=600, rot_dim=10),
@@ -120,6 +120,17 @@ def test_mixer_alone(name, f32):
     assert close(decode(d, t[139:], 139), want[139:], f32)
     assert close(decode(m.dec(f32), t[:24], 0), want[:24], f32)
     assert close(run_portions(m.dec(f32), t[:90], [2, 7, 30]), want[:90], f32)
+
+
+@BOTH
+@pytest.mark.parametrize("sizes", [dict(dim=64, rot_dim=16, vdim=64, kv_rank=48), dict(dim=128, rot_dim=60, vdim=101, kv_rank=72), dict(dim=12, rot_dim=10, vdim=9, kv_rank=20)], ids=["80", "188", "22"])
+def test_long_portions_behind_a_window(sizes, f32):
+    """Portions whose window starts well behind the first cache row."""
+    m = Model(config([(latent(heads=2, window=66, scale=0.1, **sizes), None)]), seed=6)
+    t = toks(460)
+    want = m.ref(t)
+    for portions in ([200, 130, 65], [129, 70], [300, 100, 2]):
+        assert close(run_portions(m.dec(f32, max_seq=460), t, portions), want, f32), portions
 
 
 FFNS = {
@@ -151,6 +162,16 @@ def test_norms_gates_and_soft_cap(width, groups, vocab, eps, cap, f32):
     m.plain.forward(t, m.plain.new_state(), layers)
     x = layers[-1][-1]
     assert np.allclose(d.hidden(), x, atol=(1e-4 if f32 else 6e-2) * np.max(np.abs(x)))
+
+
+@BOTH
+def test_a_width_beyond_the_registers_of_a_launch(f32):
+    m = Model(config([(gru(16), None), 0], width=4224, groups=3, vocab=40), seed=5)
+    t = toks(14, 40)
+    want = m.ref(t)
+    d = m.dec(f32)
+    assert close(d.prefill_logits(t[:9]), want[:9], f32)
+    assert close(decode(d, t[9:], 9), want[9:], f32)
 
 
 def test_the_gate_and_the_norms_matter():
